@@ -315,3 +315,50 @@ LRM_API int lrm_tanh_columns(const void* src, int in_dtype, long long stride, vo
     return LRM_BAD_ARGUMENT;
   return 0;
 }
+
+// The stream leaves through `out` in the activation type (with the float32 slices of a product that
+// belong to it added in slice order) and is replaced by `base`: what a product that rewrites the whole
+// stream, x <- W x + base, needs before it adds its sums in place.
+template <typename A>
+__global__ void stream_swap_kernel(float* x, const float* base, const float* partials, int n_partials, A* __restrict__ out,
+                                   size_t n) {
+  pdl_trigger();
+  pdl_wait();
+  const size_t idx = blockIdx.x * static_cast<size_t>(blockDim.x) + threadIdx.x;
+  if (idx >= n) return;
+  float v = x[idx];
+  for (int p = 0; p < n_partials; ++p) v += partials[p * n + idx];
+  out[idx] = from_f32<A>(v);
+  x[idx] = base[idx];
+}
+
+LRM_API int lrm_stream_swap(float* x, const float* base, const float* partials, int n_partials, void* out, int dtype,
+                            long long n, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (x == nullptr || base == nullptr || out == nullptr || n_partials < 0 || (n_partials > 0 && partials == nullptr))
+    return LRM_BAD_ARGUMENT;
+  if (dtype == LRM_F32)
+    LRM_LAUNCH(stream_swap_kernel<float>, blocks_for(n), 256, 0, stream, x, base, partials, n_partials,
+               static_cast<float*>(out), static_cast<size_t>(n));
+  else if (dtype == LRM_BF16)
+    LRM_LAUNCH(stream_swap_kernel<__nv_bfloat16>, blocks_for(n), 256, 0, stream, x, base, partials, n_partials,
+               static_cast<__nv_bfloat16*>(out), static_cast<size_t>(n));
+  else
+    return LRM_BAD_ARGUMENT;
+  return 0;
+}
+
+// x = cap tanh(x / cap) in place.
+__global__ void softcap_kernel(float* x, float cap, size_t n) {
+  pdl_trigger();
+  pdl_wait();
+  const size_t idx = blockIdx.x * static_cast<size_t>(blockDim.x) + threadIdx.x;
+  if (idx < n) x[idx] = cap * tanhf(x[idx] / cap);
+}
+
+LRM_API int lrm_softcap_inplace(float* x, float cap, long long n, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (x == nullptr || !(cap > 0.f)) return LRM_BAD_ARGUMENT;
+  LRM_LAUNCH(softcap_kernel, blocks_for(n), 256, 0, stream, x, cap, static_cast<size_t>(n));
+  return 0;
+}

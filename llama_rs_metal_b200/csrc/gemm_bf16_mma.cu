@@ -54,13 +54,17 @@ __device__ __forceinline__ void load_tile(__nv_bfloat16 (*dst)[BK + PAD],
 __global__ __launch_bounds__(128) void gemm_bf16_mma_kernel(const __nv_bfloat16* __restrict__ X,
                                                             const __nv_bfloat16* __restrict__ W,
                                                             void* __restrict__ C, int M, int N,
-                                                            int K, int mode, int vector_ok) {
+                                                            int K, int mode, int vector_ok, int group_cols,
+                                                            int group_rows) {
   __shared__ __align__(16) __nv_bfloat16 Xs[BM][BK + PAD];
   __shared__ __align__(16) __nv_bfloat16 Ws[BN][BK + PAD];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int g = lane >> 2, t = lane & 3;
   const int wm = (warp >> 1) * 32, wn = (warp & 1) * 32;
   const int m0 = blockIdx.y * BM, n0 = blockIdx.x * BN;
+  // grouped inputs: columns [i group_cols, (i + 1) group_cols) multiply the input that begins i group_rows
+  // rows into X
+  if (group_cols > 0) X += static_cast<size_t>(n0 / group_cols) * group_rows * K;
   float acc[2][4][4];
 #pragma unroll
   for (int i = 0; i < 2; ++i)
@@ -137,9 +141,11 @@ __global__ __launch_bounds__(128) void gemm_bf16_mma_kernel(const __nv_bfloat16*
 }
 }  // namespace
 
-LRM_API int lrm_gemm_bf16_mma(const void* X, const void* W, void* C, int M, int N, int K, int mode,
-                              cudaStream_t stream) {
+// group_cols > 0 (a multiple of 64): several inputs `group_rows` rows apart in X.
+LRM_API int lrm_gemm_bf16_mma_grouped(const void* X, const void* W, void* C, int M, int N, int K, int mode,
+                                      int group_cols, int group_rows, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
+  if (group_cols < 0 || group_cols % BN || (group_cols > 0 && group_rows < M)) return LRM_BAD_ARGUMENT;
   if (K <= 0 || mode < 0 || mode > 3) return LRM_BAD_ARGUMENT;
   if (mode == 3 && N % 16 != 0) return LRM_BAD_ARGUMENT;
   const dim3 grid((N + BN - 1) / BN, (M + BM - 1) / BM);
@@ -148,7 +154,12 @@ LRM_API int lrm_gemm_bf16_mma(const void* X, const void* W, void* C, int M, int 
                        (reinterpret_cast<uintptr_t>(W) % 16 == 0) && (K % 8 == 0);
   gemm_bf16_mma_kernel<<<grid, 128, 0, stream>>>(static_cast<const __nv_bfloat16*>(X),
                                                  static_cast<const __nv_bfloat16*>(W), C, M, N, K,
-                                                 mode, aligned ? 1 : 0);
+                                                 mode, aligned ? 1 : 0, group_cols, group_rows);
   LRM_LAUNCH_CHECK();
   return 0;
+}
+
+LRM_API int lrm_gemm_bf16_mma(const void* X, const void* W, void* C, int M, int N, int K, int mode,
+                              cudaStream_t stream) {
+  return lrm_gemm_bf16_mma_grouped(X, W, C, M, N, K, mode, 0, 0, stream);
 }

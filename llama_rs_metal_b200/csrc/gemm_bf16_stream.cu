@@ -19,6 +19,10 @@
 // norm kernel does it in its own pass). No atomics: the result does not depend on which CTA
 // finishes first.
 //
+// Grouped inputs (GROUPED): output columns [i cols, (i + 1) cols) multiply the rows of input i, which
+// begins `rows` rows after input i - 1 in X: one launch for the products of several inputs of equal
+// shape with the rows of one stacked W. A variant of its own: the plain kernel's registers are counted.
+//
 // Epilogues: 0 store bf16, 1 store f32, 2 add into f32 in place, 3 SiLU gate
 // (rows alternate in blocks of 8 gate / 8 up rows, so a 16-row tile holds 8
 // gated pairs; out is [M, N/2] bf16), 4 store f32 partials per K slice, 5 token choice: the
@@ -71,11 +75,16 @@ struct PickArgs {
   unsigned long long seed;
 };
 
+// Output columns per input and rows of X between inputs (GROUPED).
+struct Grouped {
+  int cols, rows;
+};
+
 // MINB: CTAs per SM the register budget must allow (a single wave for the usual sizes).
-template <int NT, int WARPS, int MINB>
+template <int NT, int WARPS, int MINB, bool GROUPED>
 __global__ __launch_bounds__(WARPS * 32, MINB) void gemm_bf16_stream_kernel(
     const __nv_bfloat16* __restrict__ X, const __nv_bfloat16* __restrict__ W, void* __restrict__ out,
-    int M, int N, int K_total, int mode, int k_per_split, PickArgs pick) {
+    int M, int N, int K_total, int mode, int k_per_split, PickArgs pick, Grouped grouped) {
   extern __shared__ float red[];  // [WARPS][NT][32 lanes][4]
   pdl_trigger();  // the next kernel may be scheduled at once (its CTAs fetch their first weights while
                   // this kernel streams); it waits for this one where it must
@@ -83,6 +92,8 @@ __global__ __launch_bounds__(WARPS * 32, MINB) void gemm_bf16_stream_kernel(
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int g = lane >> 2, t = lane & 3;
   const int n0 = blockIdx.x * 16;
+  if (GROUPED) __builtin_assume(mode >= 0 && mode <= 1);
+  if (GROUPED) X += static_cast<size_t>(n0 / grouped.cols) * grouped.rows * K_total;
   const int k_lo = blockIdx.y * k_per_split;              // this CTA's slice of K: [k_lo, K)
   const int K = min(K_total, k_lo + k_per_split);
   // epilogue 4: this slice's partial product goes to its own [M, N] plane of `out`
@@ -237,11 +248,11 @@ __global__ __launch_bounds__(WARPS * 32, MINB) void gemm_bf16_stream_kernel(
   }
 }
 
-template <int NT, int WARPS, int MINB>
+template <int NT, int WARPS, int MINB, bool GROUPED = false>
 int launch_variant(const void* X, const void* W, void* out, int M, int N, int K, int mode, int splits,
-                   const PickArgs& pick, cudaStream_t stream) {
+                   const PickArgs& pick, cudaStream_t stream, const Grouped& grouped = Grouped{0, 0}) {
   constexpr int smem = WARPS * NT * 32 * 4 * static_cast<int>(sizeof(float));
-  auto kernel = gemm_bf16_stream_kernel<NT, WARPS, MINB>;
+  auto kernel = gemm_bf16_stream_kernel<NT, WARPS, MINB, GROUPED>;
   if (smem > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return static_cast<int>(e);
@@ -250,7 +261,7 @@ int launch_variant(const void* X, const void* W, void* out, int M, int N, int K,
   const int k_per_split = ((K + splits - 1) / splits + kChunk - 1) / kChunk * kChunk;
   const dim3 grid((N + 15) / 16, (K + k_per_split - 1) / k_per_split);
   LRM_LAUNCH(kernel, grid, WARPS * 32, smem, stream, static_cast<const __nv_bfloat16*>(X),
-             static_cast<const __nv_bfloat16*>(W), out, M, N, K, mode, k_per_split, pick);
+             static_cast<const __nv_bfloat16*>(W), out, M, N, K, mode, k_per_split, pick, grouped);
   return 0;
 }
 
@@ -281,6 +292,16 @@ int launch_rows(const void* X, const void* W, void* out, int M, int N, int K, in
   if (M <= 16) return launch_stream<2>(X, W, out, M, N, K, mode, warps, splits, pick, stream);
   if (M <= 32) return launch_stream<4>(X, W, out, M, N, K, mode, warps, splits, pick, stream);
   return launch_stream<8>(X, W, out, M, N, K, mode, warps < 8 ? warps : 8, splits, pick, stream);
+}
+
+template <int NT>
+int launch_grouped(const void* X, const void* W, void* out, int M, int N, int K, int mode, const Grouped& grouped,
+                   cudaStream_t stream) {
+  constexpr int kWarpsPerSm = NT <= 2 ? 32 : 16;
+  // a stack of several matrices has tiles enough: few warps per CTA unless it is small
+  if ((N + 15) / 16 >= 148 * 4 || K <= 512)
+    return launch_variant<NT, 4, kWarpsPerSm / 4, true>(X, W, out, M, N, K, mode, 1, PickArgs{}, stream, grouped);
+  return launch_variant<NT, 8, kWarpsPerSm / 8, true>(X, W, out, M, N, K, mode, 1, PickArgs{}, stream, grouped);
 }
 
 }  // namespace
@@ -325,6 +346,21 @@ LRM_API int lrm_gemm_bf16_stream_shaped(const void* X, const void* W, void* out,
   if (reinterpret_cast<uintptr_t>(X) % 16 || reinterpret_cast<uintptr_t>(W) % 16) return LRM_UNSUPPORTED;
   splits = mode == 4 ? pick_splits(N, K, splits) : 1;
   return launch_rows(X, W, out, M, N, K, mode, warps, splits, PickArgs{}, stream);
+}
+
+// Several inputs in one launch: X holds them `group_rows` rows apart, out [M, N] (mode 0 or 1), column n
+// from input n / group_cols. group_cols a multiple of 16.
+LRM_API int lrm_gemm_bf16_stream_grouped(const void* X, const void* W, void* out, int M, int N, int K, int mode,
+                                         int group_cols, int group_rows, cudaStream_t stream) {
+  if (M <= 0 || N <= 0) return 0;
+  if (!lrm_gemm_bf16_stream_supports(M, N, K)) return LRM_UNSUPPORTED;
+  if ((mode != 0 && mode != 1) || group_cols <= 0 || group_cols % 16 || group_rows < M) return LRM_BAD_ARGUMENT;
+  if (reinterpret_cast<uintptr_t>(X) % 16 || reinterpret_cast<uintptr_t>(W) % 16) return LRM_UNSUPPORTED;
+  const Grouped grouped{group_cols, group_rows};
+  if (M <= 8) return launch_grouped<1>(X, W, out, M, N, K, mode, grouped, stream);
+  if (M <= 16) return launch_grouped<2>(X, W, out, M, N, K, mode, grouped, stream);
+  if (M <= 32) return launch_grouped<4>(X, W, out, M, N, K, mode, grouped, stream);
+  return launch_grouped<8>(X, W, out, M, N, K, mode, grouped, stream);
 }
 
 // The head product with the token choice in its epilogue: ids[m] = the chosen vocabulary row for

@@ -24,6 +24,10 @@
 // This is how a product with few rows and few columns (decode at batch 17-64: O and down
 // projections) still fills the machine, with a result that does not depend on timing.
 //
+// Grouped inputs (group_cols > 0, a multiple of the tile's width): output columns [i group_cols,
+// (i + 1) group_cols) multiply the rows of input i, which begins i group_rows rows into X: one launch
+// makes the products of several inputs of equal shape with the rows of one stacked W.
+//
 // Every wait on an mbarrier is bounded: after kSpinLimit polls the thread
 // records where it gave up in `status` and the CTA winds down (waiting, again
 // bounded, for its own copies in flight, then freeing its tensor memory).
@@ -50,7 +54,7 @@ template <int BN, int STAGES, int MT>
 __global__ __launch_bounds__(kUmmaThreads, 1) void gemm_bf16_umma_kernel(
     const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
     void* __restrict__ out, int M, int N, int K, int mode, int kb_per_split, int splits,
-    int* __restrict__ status, const QkvArgs qkv) {
+    int* __restrict__ status, const QkvArgs qkv, int group_cols, int group_rows) {
   constexpr uint32_t A_BYTES = MT * BM * BK * 2, B_BYTES = BN * BK * 2, STAGE_BYTES = A_BYTES + B_BYTES;
   constexpr uint32_t SET = MT * BN;                      // columns of one set of accumulators
   constexpr uint32_t NBUF = 2 * SET <= 512 ? 2 : 1;      // sets that fit in tensor memory
@@ -108,6 +112,7 @@ __global__ __launch_bounds__(kUmmaThreads, 1) void gemm_bf16_umma_kernel(
         const int m0 = (item % m_tiles) * MT * BM, n0 = ((item / m_tiles) % n_tiles) * BN;
         const int kb_begin = (item / (m_tiles * n_tiles)) * kb_per_split;
         const int num_kb = min(k_blocks - kb_begin, kb_per_split);
+        const int x0 = m0 + (group_cols > 0 ? n0 / group_cols * group_rows : 0);  // the tile's first row of X
         for (int kb = 0; kb < num_kb; ++kb, ++it) {
           const int s = it % STAGES;
           const uint32_t round = it / STAGES;
@@ -119,7 +124,7 @@ __global__ __launch_bounds__(kUmmaThreads, 1) void gemm_bf16_umma_kernel(
 #pragma unroll
           for (int i = 0; i < MT; ++i)  // 128 rows of X per accumulator (rows beyond M read as zero)
             tma_load_2d(tiles + s * STAGE_BYTES + i * BM * BK * 2, &map_x, full + s, (kb_begin + kb) * BK,
-                        m0 + i * BM);
+                        x0 + i * BM);
           tma_load_2d(tiles + s * STAGE_BYTES + A_BYTES, &map_w, full + s, (kb_begin + kb) * BK, n0);
         }
       }
@@ -214,7 +219,8 @@ __global__ __launch_bounds__(kUmmaThreads, 1) void gemm_bf16_umma_kernel(
 // ------------------------------------------------------------------------- host side
 template <int BN, int STAGES, int MT = 1>
 int launch_umma(const void* X, const void* W, void* out, int M, int x_rows, int N, int K, int mode, int splits,
-                int* status, cudaStream_t stream, const QkvArgs& qkv = QkvArgs{}) {
+                int* status, cudaStream_t stream, const QkvArgs& qkv = QkvArgs{}, int group_cols = 0,
+                int group_rows = 0) {
   CUtensorMap map_x, map_w;
   if (!make_map_bf16(&map_x, X, x_rows, K, BM) || !make_map_bf16(&map_w, W, N, K, BN)) return LRM_UNSUPPORTED;
   constexpr int smem = STAGES * (MT * BM * BK * 2 + BN * BK * 2) + 1024 + 256;
@@ -234,7 +240,7 @@ int launch_umma(const void* X, const void* W, void* out, int M, int x_rows, int 
   }
   const int grid = static_cast<int>(items < sm_count ? items : sm_count);
   LRM_LAUNCH(kernel, dim3(grid), kUmmaThreads, smem, stream, map_x, map_w, out, M, N, K, mode, kb_per_split, real_splits,
-             status, qkv);
+             status, qkv, group_cols, group_rows);
   return 0;
 }
 
@@ -276,6 +282,26 @@ LRM_API int lrm_gemm_bf16_umma_rows(const void* X, const void* W, void* out, int
   if (tile == 2) return launch_umma<256, 3, 2>(X, W, out, M, x_rows, N, K, mode, splits, status, stream);
   if (tile == 1) return launch_umma<256, 4>(X, W, out, M, x_rows, N, K, mode, splits, status, stream);
   return launch_umma<128, 6>(X, W, out, M, x_rows, N, K, mode, splits, status, stream);
+}
+
+// Several inputs of M rows each in one launch (mode 0 or 1): input i begins i * group_rows rows into X
+// (x_rows rows in all) and makes columns [i group_cols, (i + 1) group_cols); group_cols must be a multiple
+// of the tile's width.
+LRM_API int lrm_gemm_bf16_umma_grouped(const void* X, const void* W, void* out, int M, int x_rows, int N, int K,
+                                       int mode, int tile, int group_cols, int group_rows, int* status,
+                                       cudaStream_t stream) {
+  if (M <= 0 || N <= 0) return 0;
+  if (!lrm_gemm_bf16_umma_supports(M, N, K)) return LRM_UNSUPPORTED;
+  const int width = tile == 0 ? 128 : tile == 3 ? 192 : 256;
+  if ((mode != 0 && mode != 1) || status == nullptr || tile < 0 || tile > 3 || group_cols <= 0 || group_cols % width ||
+      group_rows < M || x_rows < M + (N - 1) / group_cols * group_rows)
+    return LRM_BAD_ARGUMENT;
+  if (reinterpret_cast<uintptr_t>(X) % 16 || reinterpret_cast<uintptr_t>(W) % 16) return LRM_UNSUPPORTED;
+  const QkvArgs none{};
+  if (tile == 3) return launch_umma<192, 5>(X, W, out, M, x_rows, N, K, mode, 1, status, stream, none, group_cols, group_rows);
+  if (tile == 2) return launch_umma<256, 3, 2>(X, W, out, M, x_rows, N, K, mode, 1, status, stream, none, group_cols, group_rows);
+  if (tile == 1) return launch_umma<256, 4>(X, W, out, M, x_rows, N, K, mode, 1, status, stream, none, group_cols, group_rows);
+  return launch_umma<128, 6>(X, W, out, M, x_rows, N, K, mode, 1, status, stream, none, group_cols, group_rows);
 }
 
 // Epilogue 5: X . W^T is a prompt's fused q|k|v projection; it is rotated and stored as rope_store.cu

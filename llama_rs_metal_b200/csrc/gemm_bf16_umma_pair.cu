@@ -94,7 +94,8 @@ __device__ __forceinline__ void umma_bf16_pair(uint32_t tmem_d, uint64_t desc_a,
 template <int BN, int STAGES>
 __global__ __launch_bounds__(kPairThreads, 1) void gemm_bf16_umma_pair_kernel(
     const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
-    void* __restrict__ out, int M, int N, int K, int mode, int* __restrict__ status, const QkvArgs qkv) {
+    void* __restrict__ out, int M, int N, int K, int mode, int* __restrict__ status, const QkvArgs qkv,
+    int group_cols, int group_rows) {
   constexpr uint32_t A_BYTES = PM * PK * 2, B_BYTES = (BN / 2) * PK * 2, STAGE_BYTES = A_BYTES + B_BYTES;
   constexpr uint32_t ALLOC = 512, SET = 256;  // two sets of accumulators, 256 columns apart
   static_assert(BN % 32 == 0 && BN >= 64 && BN <= 256, "BN / 2 rows of W per CTA, a multiple of 16");
@@ -148,6 +149,7 @@ __global__ __launch_bounds__(kPairThreads, 1) void gemm_bf16_umma_pair_kernel(
       for (int item = pair; item < items && !*bail; item += pairs) {
         const int m0 = (item % m_tiles) * 2 * PM + static_cast<int>(rank) * PM;
         const int n0 = (item / m_tiles) * BN + static_cast<int>(rank) * (BN / 2);
+        const int x0 = m0 + (group_cols > 0 ? n0 / group_cols * group_rows : 0);  // grouped inputs, as in gemm_bf16_umma.cu
         for (int kb = 0; kb < k_blocks; ++kb, ++it) {
           const int s = it % STAGES;
           const uint32_t round = it / STAGES;
@@ -157,7 +159,7 @@ __global__ __launch_bounds__(kPairThreads, 1) void gemm_bf16_umma_pair_kernel(
           }
           if (leader) mbar_expect_tx(full + s, 2 * STAGE_BYTES);  // both CTAs' copies
           const uint32_t bar = map_to_rank(smem_u32(full + s), 0);
-          tma_load_2d_pair(tiles + s * STAGE_BYTES, &map_x, bar, kb * PK, m0);
+          tma_load_2d_pair(tiles + s * STAGE_BYTES, &map_x, bar, kb * PK, x0);
           tma_load_2d_pair(tiles + s * STAGE_BYTES + A_BYTES, &map_w, bar, kb * PK, n0);
         }
       }
@@ -279,11 +281,12 @@ template <int BN, int STAGES> int resident_pairs() {
 
 template <int BN, int STAGES>
 int launch_pair(const void* X, const void* W, void* out, int M, int N, int K, int mode, int* status,
-                cudaStream_t stream, const QkvArgs& qkv = QkvArgs{}) {
+                cudaStream_t stream, const QkvArgs& qkv = QkvArgs{}, int x_rows = 0, int group_cols = 0,
+                int group_rows = 0) {
   const int room = resident_pairs<BN, STAGES>();
   if (room <= 0) return LRM_UNSUPPORTED;
   CUtensorMap map_x, map_w;
-  if (!make_map_bf16(&map_x, X, M, K, PM) || !make_map_bf16(&map_w, W, N, K, BN / 2)) return LRM_UNSUPPORTED;
+  if (!make_map_bf16(&map_x, X, x_rows > 0 ? x_rows : M, K, PM) || !make_map_bf16(&map_w, W, N, K, BN / 2)) return LRM_UNSUPPORTED;
   const long long items = static_cast<long long>((N + BN - 1) / BN) * ((M + 2 * PM - 1) / (2 * PM));
   const int pairs = static_cast<int>(items < room ? items : room);
   cudaLaunchConfig_t config = {};
@@ -291,7 +294,7 @@ int launch_pair(const void* X, const void* W, void* out, int M, int N, int K, in
   int code = pair_config<BN, STAGES>(config, attributes, 2 * pairs, stream);
   if (code != 0) return code;
   cudaError_t e = cudaLaunchKernelEx(&config, gemm_bf16_umma_pair_kernel<BN, STAGES>, map_x, map_w, out, M, N, K,
-                                     mode, status, qkv);
+                                     mode, status, qkv, group_cols, group_rows);
   return e == cudaSuccess ? 0 : static_cast<int>(e);
 }
 
@@ -315,6 +318,19 @@ LRM_API int lrm_gemm_bf16_umma_pair(const void* X, const void* W, void* out, int
   if (mode < 0 || mode > 3 || (mode == 3 && N % 16 != 0) || status == nullptr) return LRM_BAD_ARGUMENT;
   if (reinterpret_cast<uintptr_t>(X) % 16 || reinterpret_cast<uintptr_t>(W) % 16) return LRM_UNSUPPORTED;
   return launch_pair<256, 6>(X, W, out, M, N, K, mode, status, stream);
+}
+
+// Several inputs in one launch, as lrm_gemm_bf16_umma_grouped; group_cols a multiple of 256.
+LRM_API int lrm_gemm_bf16_umma_pair_grouped(const void* X, const void* W, void* out, int M, int x_rows, int N, int K,
+                                            int mode, int group_cols, int group_rows, int* status,
+                                            cudaStream_t stream) {
+  if (M <= 0 || N <= 0) return 0;
+  if (K < 8 || K % 8 != 0 || encode_tiled() == nullptr) return LRM_UNSUPPORTED;
+  if ((mode != 0 && mode != 1) || status == nullptr || group_cols <= 0 || group_cols % 256 || group_rows < M ||
+      x_rows < M + (N - 1) / group_cols * group_rows)
+    return LRM_BAD_ARGUMENT;
+  if (reinterpret_cast<uintptr_t>(X) % 16 || reinterpret_cast<uintptr_t>(W) % 16) return LRM_UNSUPPORTED;
+  return launch_pair<256, 6>(X, W, out, M, N, K, mode, status, stream, QkvArgs{}, x_rows, group_cols, group_rows);
 }
 
 // Epilogue 5 on pairs of SMs (see lrm_gemm_bf16_umma_qkv): head sizes 64 and 128.

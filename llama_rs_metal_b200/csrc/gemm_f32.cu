@@ -15,11 +15,14 @@ constexpr int BM = 64, BN = 64, BK = 16;
 __global__ __launch_bounds__(256) void gemm_f32_kernel(const float* __restrict__ X,
                                                        const float* __restrict__ W,
                                                        float* __restrict__ C, int M, int N, int K,
-                                                       int mode) {
+                                                       int mode, int group_cols, int group_rows) {
   __shared__ float Xs[BK][BM + 4];
   __shared__ float Ws[BK][BN + 4];
   const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
   const int m0 = blockIdx.y * BM, n0 = blockIdx.x * BN;
+  // grouped inputs: columns [i group_cols, (i + 1) group_cols) multiply the input that begins i group_rows
+  // rows into X
+  if (group_cols > 0) X += static_cast<size_t>(n0 / group_cols) * group_rows * K;
   float acc[4][4];
 #pragma unroll
   for (int i = 0; i < 4; ++i)
@@ -65,13 +68,20 @@ __global__ __launch_bounds__(256) void gemm_f32_kernel(const float* __restrict__
 }
 }  // namespace
 
-LRM_API int lrm_gemm_f32(const float* X, const float* W, float* C, int M, int N, int K, int mode,
-                         cudaStream_t stream) {
+// group_cols > 0 (a multiple of 64): several inputs `group_rows` rows apart in X.
+LRM_API int lrm_gemm_f32_grouped(const float* X, const float* W, float* C, int M, int N, int K, int mode,
+                                 int group_cols, int group_rows, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
+  if (group_cols < 0 || group_cols % BN || (group_cols > 0 && group_rows < M)) return LRM_BAD_ARGUMENT;
   if (K <= 0 || (mode != 0 && mode != 1)) return LRM_BAD_ARGUMENT;
   const dim3 grid((N + BN - 1) / BN, (M + BM - 1) / BM);
   if (grid.y > 65535) return LRM_UNSUPPORTED;
-  gemm_f32_kernel<<<grid, 256, 0, stream>>>(X, W, C, M, N, K, mode);
+  gemm_f32_kernel<<<grid, 256, 0, stream>>>(X, W, C, M, N, K, mode, group_cols, group_rows);
   LRM_LAUNCH_CHECK();
   return 0;
+}
+
+LRM_API int lrm_gemm_f32(const float* X, const float* W, float* C, int M, int N, int K, int mode,
+                         cudaStream_t stream) {
+  return lrm_gemm_f32_grouped(X, W, C, M, N, K, mode, 0, 0, stream);
 }

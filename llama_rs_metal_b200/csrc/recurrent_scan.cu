@@ -4,13 +4,16 @@
 //   plain decay (retention):   S <- a S + k v^T                      o = S^T q
 //   decay per token:           S <- a_t S + k v^T                    o = S^T q
 //   gated delta rule:          S <- diag(g) S;  u = b (v - S^T k);   S <- S + k u^T;   o = S^T q
+//   delta rule, head decay:    S <- a_t S;  u = b (v - S^T k);   S <- S + k u^T;   o = S^T q
 //   generalized delta rule:    S <- diag(g) S + e (c^T S) + k v^T   (both terms read the old S)   o = S^T q
+//   bonus for the newest:      o = (S + diag(m) k v^T)^T q;   S <- diag(g) S + k v^T   (read before the write)
 //
 // with a one decay per head (or, per token, one per head and token: state-space and matrix-memory
 // mixers, whose step size or input gate the caller has multiplied into v), g one decay per head
 // and key channel and token, b one step size per head and token; in the generalized rule c is the
 // direction that is read (a unit key) and e what is written back along it (minus a removal rate
-// per key channel times that direction), both per head, key channel and token. Everything here is float32: the inputs are prepared in float32 by the kernels
+// per key channel times that direction), both per head, key channel and token; m is one factor per
+// head and key channel that the current token's own contribution has in the read-out. Everything here is float32: the inputs are prepared in float32 by the kernels
 // below (rotation, short convolutions, unit norms, decays), the state lives in float32 in the
 // cache's state storage, one matrix per slot and head, and is carried from step to step.
 //
@@ -48,22 +51,30 @@ __device__ __forceinline__ void scan_cp_async(float* dst, const float* src, bool
 // MODE 0: one decay per head (head_decay); 1: the gated delta rule (g, beta); 2: one decay per head
 // and token (in `beta`'s place, [T, H]); 3: the generalized delta rule (g, and the two more rows
 // `look` = c and `put` = e per token, [T, H, d]): with t_j = sum_i c_i S_ij over the old state,
-// S_ij <- g_i S_ij + e_i t_j + k_i v_j and o_j = sum_i g_i S_ij q_i + t_j (e . q) + v_j (k . q).
+// S_ij <- g_i S_ij + e_i t_j + k_i v_j and o_j = sum_i g_i S_ij q_i + t_j (e . q) + v_j (k . q);
+// 4: the read-out before the write with a bonus (g, and `look` = m [H, d], the same for every token):
+// o_j = sum_i S_ij q_i + v_j sum_i m_i k_i q_i, then S_ij <- g_i S_ij + k_i v_j: nothing a token adds to
+// the state waits for a sum over it; 5: the delta rule with one decay per head and token (`beta`
+// [T, H] step sizes, `put` [T, H] decays).
+// q and k rows of a token are q_stride floats after those of the token before, v rows v_stride.
 template <int ROWS, int MODE>
 __global__ __launch_bounds__(kScanThreads) void linear_scan_kernel(
     const float* __restrict__ q, const float* __restrict__ k, const float* __restrict__ v,
     const float* __restrict__ g, const float* __restrict__ head_decay, const float* __restrict__ beta,
     const float* __restrict__ look, const float* __restrict__ put,
     float* __restrict__ state, float* __restrict__ out, const int* __restrict__ cu_seqlens,
-    const int* __restrict__ slots, int H, int KH, int d, int dv, int P, int chunk) {
+    const int* __restrict__ slots, int H, int KH, int d, int dv, int P, int chunk, long long q_stride,
+    long long v_stride, int wide_rows) {
   extern __shared__ __align__(16) float smem[];
-  constexpr bool DELTA = MODE == 1;
+  constexpr bool DELTA = MODE == 1 || MODE == 5;
   constexpr bool GEN = MODE == 3;
-  constexpr int NR = DELTA ? 3 : GEN ? 5 : 2;          // rows of d floats a token brings
+  constexpr bool BONUS = MODE == 4;
+  constexpr bool ROW_DECAY = MODE == 1 || MODE == 3 || MODE == 4;  // a row g of decays per token
+  constexpr int NR = GEN ? 5 : ROW_DECAY ? 3 : 2;      // rows of d floats a token brings
   constexpr int RS = ROWS + 4;
   const int TS = P * RS, COLS = kScanThreads / P;
   const int VS = (COLS + 3) & ~3;                       // v of a token, padded to whole 16 bytes
-  const int TOKEN = NR * TS + VS + 4;                   // q | k | (g) | (look | put) | v | beta
+  const int TOKEN = NR * TS + VS + 4;                   // q | k | (g) | (look | put) | v | beta, decay
   const int STAGE = chunk * TOKEN;
 
   const int tid = threadIdx.x, pidx = tid % P, jl = tid / P;
@@ -80,8 +91,16 @@ __global__ __launch_bounds__(kScanThreads) void linear_scan_kernel(
     S[i] = (mine != nullptr && row < d && j < dv) ? mine[static_cast<size_t>(row) * dv + j] : 0.f;
   }
   const float a = MODE == 0 ? head_decay[h] : 1.f;
+  float bonus[BONUS ? ROWS : 1];
+  if constexpr (BONUS) {
+#pragma unroll
+    for (int i = 0; i < ROWS; ++i) {
+      const int row = pidx * ROWS + i;
+      bonus[i] = row < d ? look[h * d + row] : 0.f;
+    }
+  }
   // 16-byte copies where every row of the inputs starts on a 16-byte boundary
-  const bool wide = d % 4 == 0 && dv % 4 == 0 && COLS % 4 == 0;
+  const bool wide = wide_rows && COLS % 4 == 0;
   const int step = wide ? 4 : 1;
 
   auto issue = [&](int c0, int stage) {
@@ -93,9 +112,9 @@ __global__ __launch_bounds__(kScanThreads) void linear_scan_kernel(
       const size_t tok = static_cast<size_t>(start + c0 + c);
       const bool in = r < d;
       float* dst = base + c * TOKEN + (r / ROWS) * RS + r % ROWS;
-      scan_cp_async(dst, q + (tok * KH + kh) * d + (in ? r : 0), in, wide);
-      scan_cp_async(dst + TS, k + (tok * KH + kh) * d + (in ? r : 0), in, wide);
-      if (DELTA || GEN) scan_cp_async(dst + 2 * TS, g + (tok * H + h) * d + (in ? r : 0), in, wide);
+      scan_cp_async(dst, q + tok * q_stride + kh * d + (in ? r : 0), in, wide);
+      scan_cp_async(dst + TS, k + tok * q_stride + kh * d + (in ? r : 0), in, wide);
+      if (ROW_DECAY) scan_cp_async(dst + 2 * TS, g + (tok * H + h) * d + (in ? r : 0), in, wide);
       if (GEN) {
         scan_cp_async(dst + 3 * TS, look + (tok * H + h) * d + (in ? r : 0), in, wide);
         scan_cp_async(dst + 4 * TS, put + (tok * H + h) * d + (in ? r : 0), in, wide);
@@ -106,12 +125,16 @@ __global__ __launch_bounds__(kScanThreads) void linear_scan_kernel(
       const int c = idx / v_per_token, cl = (idx % v_per_token) * step, col = blockIdx.x * COLS + cl;
       const size_t tok = static_cast<size_t>(start + c0 + c);
       const bool in = col < dv;
-      scan_cp_async(base + c * TOKEN + NR * TS + cl, v + (tok * H + h) * dv + (in ? col : 0), in, wide);
+      scan_cp_async(base + c * TOKEN + NR * TS + cl, v + tok * v_stride + h * dv + (in ? col : 0), in, wide);
     }
-    if (MODE == 1 || MODE == 2)
-      for (int c = tid; c < cn; c += kScanThreads)
+    if (MODE == 1 || MODE == 2 || MODE == 5)
+      for (int c = tid; c < cn; c += kScanThreads) {
         scan_cp_async(base + c * TOKEN + NR * TS + VS, beta + static_cast<size_t>(start + c0 + c) * H + h,
                       true, false);
+        if (MODE == 5)
+          scan_cp_async(base + c * TOKEN + NR * TS + VS + 1, put + static_cast<size_t>(start + c0 + c) * H + h,
+                        true, false);
+      }
     asm volatile("cp.async.commit_group;\n" ::);
   };
 
@@ -126,12 +149,12 @@ __global__ __launch_bounds__(kScanThreads) void linear_scan_kernel(
     }
     __syncthreads();
     const float* base = smem + (it & 1) * STAGE;
-#pragma unroll 2
+#pragma unroll (BONUS ? 4 : 2)
     for (int c = 0; c < cn; ++c) {
       const float* qc = base + c * TOKEN + pidx * RS;
       const float* kc = qc + TS;
       const float* gc = kc + TS;
-      const float at = MODE == 2 ? base[c * TOKEN + 2 * TS + VS] : a;
+      const float at = MODE == 2 ? base[c * TOKEN + 2 * TS + VS] : MODE == 5 ? base[c * TOKEN + 2 * TS + VS + 1] : a;
       float kr[ROWS];
       float er[GEN ? ROWS : 1];
       float r0 = 0.f, r1 = 0.f, s0 = 0.f, s1 = 0.f, kq0 = 0.f, kq1 = 0.f, eq0 = 0.f, eq1 = 0.f;
@@ -140,7 +163,7 @@ __global__ __launch_bounds__(kScanThreads) void linear_scan_kernel(
         const float4 k4 = *reinterpret_cast<const float4*>(kc + i);
         const float4 q4 = *reinterpret_cast<const float4*>(qc + i);
         float4 g4 = make_float4(at, at, at, at);
-        if (DELTA || GEN) g4 = *reinterpret_cast<const float4*>(gc + i);
+        if (ROW_DECAY) g4 = *reinterpret_cast<const float4*>(gc + i);
         kr[i] = k4.x, kr[i + 1] = k4.y, kr[i + 2] = k4.z, kr[i + 3] = k4.w;
         if constexpr (GEN) {  // what the old state holds along `look`, before the decay
           const float4 c4 = *reinterpret_cast<const float4*>(gc + TS + i);
@@ -150,6 +173,14 @@ __global__ __launch_bounds__(kScanThreads) void linear_scan_kernel(
           er[i] = e4.x, er[i + 1] = e4.y, er[i + 2] = e4.z, er[i + 3] = e4.w;
           eq0 = fmaf(e4.x, q4.x, eq0), eq1 = fmaf(e4.y, q4.y, eq1);
           eq0 = fmaf(e4.z, q4.z, eq0), eq1 = fmaf(e4.w, q4.w, eq1);
+        }
+        if constexpr (BONUS) {  // the old state is read, then decayed
+          s0 = fmaf(S[i], q4.x, s0), s1 = fmaf(S[i + 1], q4.y, s1);
+          s0 = fmaf(S[i + 2], q4.z, s0), s1 = fmaf(S[i + 3], q4.w, s1);
+          kq0 = fmaf(k4.x * bonus[i], q4.x, kq0), kq1 = fmaf(k4.y * bonus[i + 1], q4.y, kq1);
+          kq0 = fmaf(k4.z * bonus[i + 2], q4.z, kq0), kq1 = fmaf(k4.w * bonus[i + 3], q4.w, kq1);
+          S[i] *= g4.x, S[i + 1] *= g4.y, S[i + 2] *= g4.z, S[i + 3] *= g4.w;
+          continue;
         }
         S[i] *= g4.x, S[i + 1] *= g4.y, S[i + 2] *= g4.z, S[i + 3] *= g4.w;
         if (DELTA) {
@@ -169,7 +200,7 @@ __global__ __launch_bounds__(kScanThreads) void linear_scan_kernel(
         kq += __shfl_xor_sync(0xffffffffu, kq, o);
       }
       const float vj = base[c * TOKEN + NR * TS + jl];
-      const float u = DELTA ? base[c * TOKEN + 3 * TS + VS] * (vj - r) : vj;
+      const float u = DELTA ? base[c * TOKEN + NR * TS + VS] * (vj - r) : vj;
 #pragma unroll
       for (int i = 0; i < ROWS; ++i) S[i] = fmaf(kr[i], u, S[i]);
       if constexpr (GEN) {
@@ -191,11 +222,16 @@ __global__ __launch_bounds__(kScanThreads) void linear_scan_kernel(
   }
 }
 
+// How far apart a token's q and k rows, and its v row, are from those of the token before (0: packed).
+struct RowStrides {
+  long long q = 0, v = 0;
+};
+
 template <int ROWS, int MODE>
 int launch_scan(const float* q, const float* k, const float* v, const float* g, const float* head_decay,
                 const float* beta, const float* look, const float* put, float* state, float* out, const int* cu_seqlens, const int* slots,
-                int seqs, int H, int KH, int d, int dv, int P, cudaStream_t stream) {
-  constexpr int NR = MODE == 1 ? 3 : MODE == 3 ? 5 : 2;
+                int seqs, int H, int KH, int d, int dv, int P, const RowStrides& rows, cudaStream_t stream) {
+  constexpr int NR = MODE == 3 ? 5 : MODE == 1 || MODE == 4 ? 3 : 2;
   const int COLS = kScanThreads / P, TS = P * (ROWS + 4), VS = (COLS + 3) & ~3;
   int chunk = kChunk;
   while (chunk > 1 && sizeof(float) * 2 * chunk * (static_cast<size_t>(NR) * TS + VS + 4) > 200 * 1024) chunk >>= 1;
@@ -208,9 +244,14 @@ int launch_scan(const float* q, const float* k, const float* v, const float* g, 
     if (e != cudaSuccess) return static_cast<int>(e);
     raised = true;
   }
+  const long long q_stride = rows.q > 0 ? rows.q : static_cast<long long>(KH) * d;
+  const long long v_stride = rows.v > 0 ? rows.v : static_cast<long long>(H) * dv;
+  auto aligned = [](const float* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+  const int wide = d % 4 == 0 && dv % 4 == 0 && q_stride % 4 == 0 && v_stride % 4 == 0 && aligned(q) && aligned(k) &&
+                   aligned(v) && aligned(g) && (MODE != 3 || (aligned(look) && aligned(put)));
   const dim3 grid((dv + COLS - 1) / COLS, H, seqs);
   LRM_LAUNCH((linear_scan_kernel<ROWS, MODE>), grid, kScanThreads, bytes, stream, q, k, v, g, head_decay, beta,
-             look, put, state, out, cu_seqlens, slots, H, KH, d, dv, P, chunk);
+             look, put, state, out, cu_seqlens, slots, H, KH, d, dv, P, chunk, q_stride, v_stride, wide);
   return 0;
 }
 
@@ -231,7 +272,7 @@ void scan_shape(int d, int* rows, int* parts, int most_rows) {
 template <int MODE>
 int dispatch_scan(const float* q, const float* k, const float* v, const float* g, const float* head_decay,
                   const float* beta, const float* look, const float* put, float* state, float* out, const int* cu_seqlens, const int* slots,
-                  int seqs, int H, int KH, int d, int dv, cudaStream_t stream) {
+                  int seqs, int H, int KH, int d, int dv, cudaStream_t stream, const RowStrides& rows = RowStrides{}) {
   int R, P;
   scan_shape(d, &R, &P, g_scan_rows);
   if (MODE == 3 && g_scan_rows > 8) {
@@ -245,7 +286,7 @@ int dispatch_scan(const float* q, const float* k, const float* v, const float* g
 #define LRM_SCAN_CASE(N)                                                                             \
   case N:                                                                                            \
     return launch_scan<N, MODE>(q, k, v, g, head_decay, beta, look, put, state, out, cu_seqlens, slots, seqs, H, \
-                                 KH, d, dv, P, stream)
+                                 KH, d, dv, P, rows, stream)
   switch (R) {
     LRM_SCAN_CASE(4);
     LRM_SCAN_CASE(8);
@@ -267,7 +308,8 @@ template <typename A, typename G>
 __global__ void head_norm_gate_kernel(const float* __restrict__ o, int o_stride, const float* __restrict__ weight,
                                       int w_stride, const float* __restrict__ floor, float den_eps,
                                       const G* __restrict__ gate, long long gate_stride, int gate_act,
-                                      A* __restrict__ out, int H, int dv, float eps, float out_scale) {
+                                      A* __restrict__ out, long long out_stride, int H, int dv, float eps,
+                                      float out_scale) {
   __shared__ float scratch[32];
   pdl_trigger();
   pdl_wait();
@@ -290,7 +332,7 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, int o_stride,
       const float sig = 1.0f / (1.0f + expf(-z));
       y *= gate_act == 1 ? z * sig : sig;
     }
-    out[(static_cast<size_t>(t) * H + h) * dv + j] = from_f32<A>(y * out_scale);
+    out[static_cast<size_t>(t) * out_stride + h * dv + j] = from_f32<A>(y * out_scale);
   }
 }
 
@@ -485,20 +527,51 @@ LRM_API int lrm_general_delta_scan(const float* q, const float* k, const float* 
                           stream);
 }
 
+// The read-out before the write, with a bonus for the current token: q, k at [t * q_stride + h * d], v at
+// [t * v_stride + h * dv] (strides in floats; columns of a wider activation), g float32 [T, H, d], bonus
+// float32 [H, d]: o = (S + diag(bonus) k v^T)^T q, then S <- diag(g) S + k v^T. out float32 [T, H, dv].
+LRM_API int lrm_bonus_state_scan(const float* q, const float* k, long long q_stride, const float* v,
+                                 long long v_stride, const float* g, const float* bonus, float* state, float* out,
+                                 const int* cu_seqlens, const int* slots, int seqs, int H, int d, int dv,
+                                 cudaStream_t stream) {
+  if (seqs <= 0) return 0;
+  if (H <= 0 || d <= 0 || dv <= 0 || seqs > 65535 || H > 65535) return LRM_BAD_ARGUMENT;
+  if (g == nullptr || bonus == nullptr || q_stride < static_cast<long long>(H) * d || v_stride < static_cast<long long>(H) * dv)
+    return LRM_BAD_ARGUMENT;
+  if (d > 2048) return LRM_UNSUPPORTED;
+  return dispatch_scan<4>(q, k, v, g, nullptr, nullptr, bonus, nullptr, state, out, cu_seqlens, slots, seqs, H, H, d,
+                          dv, stream, RowStrides{q_stride, v_stride});
+}
+
+// The delta rule with one decay per head and token: q, k float32 [T, KH, d], v [T, H, dv], decay and beta
+// float32 [T, H]: S <- decay S;  S <- S + k (beta (v - S^T k))^T;  o = S^T q.
+LRM_API int lrm_head_decay_delta_scan(const float* q, const float* k, const float* v, const float* decay,
+                                      const float* beta, float* state, float* out, const int* cu_seqlens,
+                                      const int* slots, int seqs, int H, int KH, int d, int dv, cudaStream_t stream) {
+  if (seqs <= 0) return 0;
+  if (H <= 0 || KH <= 0 || H % KH || d <= 0 || dv <= 0 || seqs > 65535 || H > 65535) return LRM_BAD_ARGUMENT;
+  if (decay == nullptr || beta == nullptr) return LRM_BAD_ARGUMENT;
+  if (d > 2048) return LRM_UNSUPPORTED;
+  return dispatch_scan<5>(q, k, v, nullptr, nullptr, beta, nullptr, decay, state, out, cu_seqlens, slots, seqs, H, KH, d,
+                          dv, stream);
+}
+
 // `gate` (type gate_dtype, may be null) is read at gate[t * gate_stride + h * dv + j]; o at
-// o[(t * H + h) * o_stride + j]; weight at weight[h * w_stride + j]; floor (may be null) at [t * H + h].
+// o[(t * H + h) * o_stride + j]; weight at weight[h * w_stride + j]; floor (may be null) at [t * H + h];
+// the result goes to out[t * out_stride + h * dv + j].
 LRM_API int lrm_head_norm_gate(const float* o, int o_stride, const float* weight, int w_stride, const float* floor,
                                float den_eps, const void* gate, int gate_dtype, long long gate_stride, int gate_act,
                                void* out, int dtype, int tokens, int H, int dv, float eps, float out_scale,
-                               cudaStream_t stream) {
+                               long long out_stride, cudaStream_t stream) {
   if (tokens <= 0) return 0;
+  if (out_stride < static_cast<long long>(H) * dv) return LRM_BAD_ARGUMENT;
   if (H <= 0 || H > 65535 || dv <= 0 || (gate != nullptr && gate_act != 1 && gate_act != 2)) return LRM_BAD_ARGUMENT;
   if (o_stride < dv || (floor != nullptr && o_stride <= dv) || (w_stride != 0 && w_stride != dv)) return LRM_BAD_ARGUMENT;
   const int threads = dv >= 256 ? 256 : ((dv + 31) / 32) * 32;
   const dim3 grid(tokens, H);
 #define LRM_HEAD_NORM(AT, GT)                                                                              \
   LRM_LAUNCH((head_norm_gate_kernel<AT, GT>), grid, threads, 0, stream, o, o_stride, weight, w_stride, floor,    \
-             den_eps, static_cast<const GT*>(gate), gate_stride, gate_act, static_cast<AT*>(out), H, dv, eps,     \
+             den_eps, static_cast<const GT*>(gate), gate_stride, gate_act, static_cast<AT*>(out), out_stride, H, dv, eps, \
              out_scale)
   if (dtype == LRM_F32 && gate_dtype == LRM_F32)
     LRM_HEAD_NORM(float, float);

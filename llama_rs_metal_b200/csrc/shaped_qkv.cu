@@ -1,31 +1,39 @@
 // The split of a step's fused q|k|v projection for attention layers that shape their queries and
 // keys on the way: one CTA per token takes the projection row [q_heads * d | kv_heads * d |
-// kv_heads * dv] through, in this order and each only if asked for,
+// kv_heads * dv] (rows may be further apart than that: columns behind it belong to someone else)
+// through, in this order and each only if asked for,
 //   1. the projections' biases (float32 [row]);
 //   2. a short causal convolution over time per channel (taps [n, row], the last row the current
 //      token's, no bias, zeros before the sequence's start); inputs before the step's first token
 //      come from the sequence's tail [n - 1, row] of unbiased projections in the state storage,
 //      the bias added here where the input's position is not before the start;
 //   3. an RMS norm over the whole query part and one over the whole key part, with weights;
-//   4. a rotation by position of the first `rotary` dimensions of every query and key head,
+//   4. an RMS norm over every query head and every key head, with one weight of size d for all
+//      query heads and one for all key heads;
+//   5. a rotation by position of the first `rotary` dimensions of every query and key head,
 //      dimension i paired with i + rotary/2 (pairing 0) or 2i with 2i + 1 (pairing 1), angle =
 //      position * inv_freq[i] formed in double precision;
-//   5. the division of every query and key head by its root mean square (no weight),
+//   6. the division of every query and key head by its root mean square (no weight),
 // and writes q, k, v in the activation type: q packed, k and v packed (when asked for) and into
 // the paged cache at dest_rows[t] (see qkv_store.cu for the layout). Everything between the
 // projection and the rounding at the end is float32. Reads of the projection go through plain
 // pointers: it is the output of the kernel before.
+//
+// Layers without a convolution, a row norm and a division behind the rotation (steps 1, 4 and 5 at
+// most) run a second kernel: a warp takes a head from its projection to its stores in registers,
+// with no barrier after the table of cosines and sines.
 #include "common.cuh"
 
 namespace {
 
 template <typename S, typename A>
-__global__ void shaped_qkv_kernel(const S* proj, const float* __restrict__ bias, const float* __restrict__ taps, int n,
+__global__ void shaped_qkv_kernel(const S* proj, long long stride, const float* __restrict__ bias, const float* __restrict__ taps, int n,
                                   const float* tails, const int* __restrict__ cu_seqlens,
                                   const int* __restrict__ seq_of_token, const int* __restrict__ slots,
                                   const int* __restrict__ positions, const float* __restrict__ q_norm,
                                   const float* __restrict__ k_norm, float row_eps,
-                                  const double* __restrict__ inv_freq, int rotary, int pairing, int head_norm,
+                                  const float* __restrict__ q_head_w, const float* __restrict__ k_head_w,
+                                  float head_w_eps, const double* __restrict__ inv_freq, int rotary, int pairing, int head_norm,
                                   float head_eps, A* __restrict__ q_out, A* __restrict__ k_out,
                                   A* __restrict__ v_out, A* __restrict__ k_pages, A* __restrict__ v_pages,
                                   const int* __restrict__ dest_rows, int q_heads, int kv_heads, int d, int dv,
@@ -46,7 +54,7 @@ __global__ void shaped_qkv_kernel(const S* proj, const float* __restrict__ bias,
     cs[half + i] = static_cast<float>(sn);
   }
   pdl_wait();
-  const S* src = proj + static_cast<size_t>(t) * width;
+  const S* src = proj + static_cast<size_t>(t) * stride;
   if (taps == nullptr || n <= 1) {
     for (int c = threadIdx.x; c < width; c += blockDim.x) {
       float x = to_f32(src[c]) + (bias != nullptr ? bias[c] : 0.f);
@@ -70,7 +78,7 @@ __global__ void shaped_qkv_kernel(const S* proj, const float* __restrict__ bias,
       for (int back = n - 1; back >= 0; --back) {  // oldest input first
         if (pos - back < 0) continue;              // before the sequence's start: zero
         const int at = local - back;
-        const S* from_step = at >= 0 ? proj + static_cast<size_t>(t - back) * width : nullptr;
+        const S* from_step = at >= 0 ? proj + static_cast<size_t>(t - back) * stride : nullptr;
         const float* from_tail = (at < 0 && tail != nullptr) ? tail + static_cast<size_t>(n - 1 + at) * width : nullptr;
         const float* tap = taps + static_cast<size_t>(n - 1 - back) * width;
 #pragma unroll
@@ -101,6 +109,18 @@ __global__ void shaped_qkv_kernel(const S* proj, const float* __restrict__ bias,
     const float inv_k = nk > 0 ? 1.0f / sqrtf(total_k / static_cast<float>(nk) + row_eps) : 0.f;
     for (int c = threadIdx.x; c < nq + nk; c += blockDim.x)
       row[c] = c < nq ? row[c] * inv_q * q_norm[c] : row[c] * inv_k * k_norm[c - nq];
+    __syncthreads();
+  }
+  if (q_head_w != nullptr) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+    for (int hd = warp; hd < q_heads + kv_heads; hd += warps) {
+      float* head = row + hd * d;
+      const float* w = hd < q_heads ? q_head_w : k_head_w;
+      float ss = 0.f;
+      for (int i = lane; i < d; i += 32) ss = fmaf(head[i], head[i], ss);
+      const float inv = 1.0f / sqrtf(warp_sum(ss) / static_cast<float>(d) + head_w_eps);
+      for (int i = lane; i < d; i += 32) head[i] = (head[i] * inv) * w[i];
+    }
     __syncthreads();
   }
   if (half > 0) {
@@ -145,15 +165,110 @@ __global__ void shaped_qkv_kernel(const S* proj, const float* __restrict__ bias,
   }
 }
 
+// gridDim.y CTAs per token share its heads, one warp per head at a time; lane l holds elements VEC l .. of every group of
+// 32 VEC (VEC 2 where d, dv, the row pitch and all addresses allow pairs).
+constexpr int kHeadPer = 8;  // elements of a head one lane holds at most: heads of up to 256
+
+template <typename S, typename A, int VEC>
+__global__ void shaped_heads_kernel(const S* proj, long long stride, const float* __restrict__ bias,
+                                    const int* __restrict__ positions, const float* __restrict__ q_head_w,
+                                    const float* __restrict__ k_head_w, float head_w_eps,
+                                    const double* __restrict__ inv_freq, int rotary, int pairing,
+                                    A* __restrict__ q_out, A* __restrict__ k_out, A* __restrict__ v_out,
+                                    A* __restrict__ k_pages, A* __restrict__ v_pages,
+                                    const int* __restrict__ dest_rows, int q_heads, int kv_heads, int d, int dv,
+                                    int page_size) {
+  extern __shared__ float cs[];  // [rotary / 2] cosines, then as many sines
+  const int half = rotary / 2;
+  pdl_trigger();
+  const int t = blockIdx.x, pos = positions[t];
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    double sn, c;
+    sincos(static_cast<double>(pos) * inv_freq[i], &sn, &c);
+    cs[i] = static_cast<float>(c);
+    cs[half + i] = static_cast<float>(sn);
+  }
+  const int dest = k_pages != nullptr ? dest_rows[t] : -1;
+  const size_t page = dest >= 0 ? static_cast<size_t>(dest / page_size) : 0;
+  const int in_page = dest >= 0 ? dest % page_size : 0;
+  __syncthreads();
+  pdl_wait();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+  const S* row = proj + static_cast<size_t>(t) * stride;
+  for (int hd = blockIdx.y * warps + warp; hd < q_heads + 2 * kv_heads; hd += warps * gridDim.y) {
+    const bool is_q = hd < q_heads, is_v = hd >= q_heads + kv_heads;
+    const int kh = is_q ? 0 : hd - q_heads - (is_v ? kv_heads : 0);
+    const int n = is_v ? dv : d;
+    const int first = is_v ? (q_heads + kv_heads) * d + kh * dv : hd * d;  // column in the row
+    const S* src = row + first;
+    const float* add = bias != nullptr ? bias + first : nullptr;
+    const float* w = is_v ? nullptr : is_q ? q_head_w : k_head_w;
+    float x[kHeadPer];
+#pragma unroll
+    for (int g = 0; g < kHeadPer / VEC; ++g) {
+      const int i = (g * 32 + lane) * VEC;
+#pragma unroll
+      for (int e = 0; e < VEC; ++e)
+        x[g * VEC + e] = i + e < n ? to_f32(src[i + e]) + (add != nullptr ? add[i + e] : 0.f) : 0.f;
+    }
+    float inv = 1.f;
+    if (w != nullptr) {
+      float ss = 0.f;
+#pragma unroll
+      for (int u = 0; u < kHeadPer; ++u) ss = fmaf(x[u], x[u], ss);
+      inv = 1.0f / sqrtf(warp_sum(ss) / static_cast<float>(d) + head_w_eps);
+    }
+    A* packed = is_q ? q_out + (static_cast<size_t>(t) * q_heads + hd) * d
+                : is_v ? (v_out != nullptr ? v_out + (static_cast<size_t>(t) * kv_heads + kh) * dv : nullptr)
+                       : (k_out != nullptr ? k_out + (static_cast<size_t>(t) * kv_heads + kh) * d : nullptr);
+    A* cached = (is_q || dest < 0) ? nullptr
+                : (is_v ? v_pages : k_pages) + ((page * kv_heads + kh) * page_size + in_page) * n;
+#pragma unroll
+    for (int g = 0; g < kHeadPer / VEC; ++g) {
+      const int i = (g * 32 + lane) * VEC;
+      if (i >= n) continue;
+      A y[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        const int c = i + e;
+        float v = w != nullptr ? (x[g * VEC + e] * inv) * w[c] : x[g * VEC + e];
+        if (!is_v && c < rotary) {
+          // this element's pair: the partner is read again (it is in L1) and shaped alike
+          const int pair = pairing == 0 ? (c < half ? c : c - half) : c >> 1;
+          const bool leads = pairing == 0 ? c < half : (c & 1) == 0;
+          const int other = pairing == 0 ? (leads ? c + half : c - half) : (leads ? c + 1 : c - 1);
+          float p = to_f32(src[other]) + (add != nullptr ? add[other] : 0.f);
+          if (w != nullptr) p = (p * inv) * w[other];
+          const float co = cs[pair], sn = cs[half + pair];
+          v = leads ? fmaf(v, co, -__fmul_rn(p, sn)) : fmaf(v, co, __fmul_rn(p, sn));
+        }
+        y[e] = from_f32<A>(v);
+      }
+#pragma unroll
+      for (int target = 0; target < 2; ++target) {
+        A* dst = target == 0 ? packed : cached;
+        if (dst == nullptr) continue;
+        if constexpr (VEC == 2 && sizeof(A) == 2) {
+          *reinterpret_cast<uint32_t*>(dst + i) = *reinterpret_cast<const uint32_t*>(y);
+        } else {
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) dst[i + e] = y[e];
+        }
+      }
+    }
+  }
+}
+
 }  // namespace
 
-// proj: [tokens, q_heads * d + kv_heads * (d + dv)] float32 or bfloat16 (in_dtype); outputs of
-// out_dtype. bias, taps (float32 [n, row]; + tails, cu_seqlens, seq_of_token, slots), q_norm + k_norm, inv_freq
-// (double [rotary / 2]) may each be null: that step is then left out. kv_heads 0: queries only.
-LRM_API int lrm_shaped_qkv_store(const void* proj, int in_dtype, const float* bias, const float* taps, int n,
+// proj: [tokens, stride], of whose columns the first q_heads * d + kv_heads * (d + dv) are the row;
+// float32 or bfloat16 (in_dtype); outputs of out_dtype. bias, taps (float32 [n, row]; + tails, cu_seqlens, seq_of_token, slots), q_norm + k_norm, q_head_w
+// + k_head_w (float32 [d] each), inv_freq (double [rotary / 2]) may each be null: that step is then left out. kv_heads 0: queries only.
+LRM_API int lrm_shaped_qkv_store(const void* proj, int in_dtype, long long stride, const float* bias, const float* taps, int n,
                                  const float* tails, const int* cu_seqlens, const int* seq_of_token,
                                  const int* slots, const int* positions, const float* q_norm, const float* k_norm,
-                                 float row_eps, const double* inv_freq, int rotary, int pairing, int head_norm,
+                                 float row_eps, const float* q_head_w, const float* k_head_w, float head_w_eps,
+                                 const double* inv_freq, int rotary, int pairing, int head_norm,
                                  float head_eps, void* q_out, void* k_out, void* v_out, void* k_pages, void* v_pages,
                                  const int* dest_rows, int out_dtype, int tokens, int q_heads, int kv_heads, int d,
                                  int dv, int page_size, cudaStream_t stream) {
@@ -167,7 +282,33 @@ LRM_API int lrm_shaped_qkv_store(const void* proj, int in_dtype, const float* bi
   if (taps != nullptr && n > 1 && (tails == nullptr || cu_seqlens == nullptr || seq_of_token == nullptr || slots == nullptr))
     return LRM_BAD_ARGUMENT;
   if (k_pages != nullptr && dest_rows == nullptr) return LRM_BAD_ARGUMENT;
+  if ((q_head_w == nullptr) != (k_head_w == nullptr)) return LRM_BAD_ARGUMENT;
   const int width = q_heads * d + kv_heads * (d + dv);
+  if (stride < width) return LRM_BAD_ARGUMENT;
+  if (taps == nullptr && q_norm == nullptr && !head_norm && d <= 32 * kHeadPer && dv <= 32 * kHeadPer) {
+    const int heads = q_heads + 2 * kv_heads;
+    const int threads = 32 * (heads < 4 ? heads : heads >= 16 ? 8 : 4);
+    // few tokens: a warp per head; many: a CTA per token, which makes its table of angles once
+    const dim3 grid(tokens, tokens < 148 ? (heads * 32 + threads - 1) / threads : 1);
+    const size_t in_pair = in_dtype == LRM_F32 ? 8 : 4;
+    const bool pairs = d % 2 == 0 && dv % 2 == 0 && stride % 2 == 0 && reinterpret_cast<uintptr_t>(proj) % in_pair == 0;
+#define LRM_HEADS(ST, AT, V)                                                                                        \
+  LRM_LAUNCH((shaped_heads_kernel<ST, AT, V>), grid, threads, sizeof(float) * rotary, stream, static_cast<const ST*>(proj), \
+             stride, bias, positions, q_head_w, k_head_w, head_w_eps, inv_freq, rotary, pairing, static_cast<AT*>(q_out), \
+             static_cast<AT*>(k_out), static_cast<AT*>(v_out), static_cast<AT*>(k_pages), static_cast<AT*>(v_pages), \
+             dest_rows, q_heads, kv_heads, d, dv, page_size)
+    if (in_dtype == LRM_F32 && out_dtype == LRM_F32) {
+      if (pairs) LRM_HEADS(float, float, 2); else LRM_HEADS(float, float, 1);
+    } else if (in_dtype == LRM_F32 && out_dtype == LRM_BF16) {
+      if (pairs) LRM_HEADS(float, __nv_bfloat16, 2); else LRM_HEADS(float, __nv_bfloat16, 1);
+    } else if (in_dtype == LRM_BF16 && out_dtype == LRM_BF16) {
+      if (pairs) LRM_HEADS(__nv_bfloat16, __nv_bfloat16, 2); else LRM_HEADS(__nv_bfloat16, __nv_bfloat16, 1);
+    } else {
+      return LRM_BAD_ARGUMENT;
+    }
+#undef LRM_HEADS
+    return 0;
+  }
   const size_t bytes = sizeof(float) * (static_cast<size_t>(width) + rotary);
   if (bytes > 200 * 1024) return LRM_UNSUPPORTED;
 #define LRM_SHAPED(ST, AT)                                                                                      \
@@ -179,8 +320,8 @@ LRM_API int lrm_shaped_qkv_store(const void* proj, int in_dtype, const float* bi
       if (e != cudaSuccess) return static_cast<int>(e);                                                         \
       raised = true;                                                                                            \
     }                                                                                                           \
-    LRM_LAUNCH((shaped_qkv_kernel<ST, AT>), tokens, width >= 2048 ? 512 : 256, bytes, stream, static_cast<const ST*>(proj), bias, taps, n, \
-               tails, cu_seqlens, seq_of_token, slots, positions, q_norm, k_norm, row_eps, inv_freq, rotary,    \
+    LRM_LAUNCH((shaped_qkv_kernel<ST, AT>), tokens, width >= 2048 ? 512 : 256, bytes, stream, static_cast<const ST*>(proj), stride, bias, taps, n, \
+               tails, cu_seqlens, seq_of_token, slots, positions, q_norm, k_norm, row_eps, q_head_w, k_head_w, head_w_eps, inv_freq, rotary, \
                pairing, head_norm, head_eps, static_cast<AT*>(q_out), static_cast<AT*>(k_out),                  \
                static_cast<AT*>(v_out), static_cast<AT*>(k_pages), static_cast<AT*>(v_pages), dest_rows, q_heads, \
                kv_heads, d, dv, page_size);                                                                     \

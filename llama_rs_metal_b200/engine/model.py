@@ -58,6 +58,10 @@ class DecoderModel:
         self.embedding: Optional[torch.Tensor] = None
         self.stream_offsets: Optional[torch.Tensor] = None  # float32 [rows, hidden]
         self.head: Optional[LinearWeight] = None
+        # the two halves of the plan's stream_join matrix: W [x; x0] = W_x x + W_0 x0, of which the second
+        # term is the same for every pass of a step
+        self.join_stream: Optional[LinearWeight] = None
+        self.join_embedding: Optional[LinearWeight] = None
         self.unexpected_tensors: tuple = ()  # stored names the loader skipped (set by the loader's caller)
         self._check_schedule()
 
@@ -71,6 +75,8 @@ class DecoderModel:
                 rows = self.plan.stream_offsets[1] if self.plan.stream_offsets is not None else 0
                 if not 0 <= entry.add_offset < rows:
                     raise InvalidError(f"schedule entry {position} adds offset {entry.add_offset} of {rows}")
+            if entry.join_embedding and self.plan.stream_join is None:
+                raise InvalidError(f"schedule entry {position} joins the embedding, the plan has no matrix for it")
             if entry.writes_cache:
                 if entry.cache in writers:
                     raise InvalidError(f"cache entry {entry.cache} is written by two schedule entries")
@@ -104,6 +110,8 @@ class DecoderModel:
             specs[plan.head_name] = TensorSpec((plan.vocab_size, plan.hidden_size))
         if plan.stream_offsets is not None:
             specs[plan.stream_offsets[0]] = TensorSpec((plan.stream_offsets[1], plan.hidden_size))
+        if plan.stream_join is not None:
+            specs[plan.stream_join] = TensorSpec((plan.hidden_size, 2 * plan.hidden_size))
         for block, names, own_names in zip(self.blocks, self._names, self._block_names):
             for role, mapping in names.items():
                 part_specs = getattr(block, role).tensors()
@@ -124,6 +132,9 @@ class DecoderModel:
         self.head = LinearWeight(head)
         if self.plan.stream_offsets is not None:  # added to the float32 stream: kept in float32
             self.stream_offsets = tensors[self.plan.stream_offsets[0]].to(torch.float32).contiguous()
+        if self.plan.stream_join is not None:
+            both, h = tensors[self.plan.stream_join], self.plan.hidden_size
+            self.join_stream, self.join_embedding = LinearWeight(both[:, :h]), LinearWeight(both[:, h:])
         for block, names, own_names in zip(self.blocks, self._names, self._block_names):
             for role, mapping in names.items():
                 getattr(block, role).bind({own: tensors[full] for own, full in mapping.items()}, rt)
@@ -139,6 +150,8 @@ class DecoderModel:
         logits = self.head(x, out_dtype=torch.float32)
         if self.plan.logit_scale is not None:
             ops.scale_(logits, self.plan.logit_scale)
+        if self.plan.logit_softcap is not None:
+            ops.softcap_(logits, self.plan.logit_softcap)
         return logits
 
     def forward_pick(self, ctx, cache, temperature=None, seed: int = 0, keys=None) -> torch.Tensor:
@@ -150,14 +163,16 @@ class DecoderModel:
         x = self._hidden_of_wanted_rows(ctx, cache)
         if x is None:
             return torch.empty((0,), dtype=torch.int32, device=self.runtime.device)
-        scale = self.plan.logit_scale
-        if scale is not None and scale <= 0:
+        scale, cap = self.plan.logit_scale, self.plan.logit_softcap
+        if scale is not None and (scale <= 0 or cap is not None):
             logits = ops.scale_(self.head(x, out_dtype=torch.float32), scale)
+            if cap is not None:
+                ops.softcap_(logits, cap)
             return ops.argmax_rows(logits) if temperature is None else \
                 ops.sample_gumbel_rows(logits, temperature, seed, keys)
         if temperature is not None and scale is not None:
             temperature = temperature / scale  # (s z) / T = z / (T / s)
-        return self.head.pick(x, temperature, seed, keys)
+        return self.head.pick(x, temperature, seed, keys, softcap=cap)
 
     def _hidden_of_wanted_rows(self, ctx, cache) -> Optional[torch.Tensor]:
         """Embedding, the scheduled blocks and the final norm on the wanted rows; None when no
@@ -172,6 +187,9 @@ class DecoderModel:
         wanted = ctx.wanted_rows.numel() > 0
         schedule = plan.schedule
         embedded = hidden.clone() if any(entry.add_embedding for entry in schedule) else None
+        joined = None  # W_0 x0 of the stream's join, made once
+        if any(entry.join_embedding for entry in schedule):
+            joined = self.join_embedding(ops.cast(hidden, self.runtime.dtype), out_dtype=torch.float32)
         for i, entry in enumerate(schedule):
             ctx.entry = entry
             view = cache.view(entry.cache) if cache is not None else None
@@ -182,10 +200,18 @@ class DecoderModel:
                 # a block may hand the next one its stream already passed through that block's
                 # first norm (nothing may be added to the stream in between)
                 ctx.next_entry_norm = following.entry_norm \
-                    if schedule[i + 1].add_offset is None and not schedule[i + 1].add_embedding else None
+                    if schedule[i + 1].add_offset is None and not schedule[i + 1].add_embedding \
+                    and not schedule[i + 1].join_embedding else None
+                # a join takes pending sums along with the stream it reads
+                ctx.next_folds_pending |= schedule[i + 1].join_embedding
             else:
                 ctx.next_folds_pending = wanted and self.final_norm.folds_pending
                 ctx.next_entry_norm = None
+            if entry.join_embedding:
+                # x <- W_x x + W_0 x0: the stream leaves in the activation type and is replaced by the second
+                # term, into which the product of the first is added
+                x = ops.stream_swap_(hidden, joined, self.runtime.dtype, ctx.take_pending())
+                hidden = self.join_stream(x, epilogue=ops.ADD, out=hidden)
             if entry.add_embedding:
                 hidden = ops.add_(ctx.settle(hidden), embedded)
             if entry.add_offset is not None:

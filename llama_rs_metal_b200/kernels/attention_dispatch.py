@@ -11,6 +11,8 @@ cache write, attention and the merge of the splits as one cluster kernel
 sequences stores its keys first and attends over the cache (row-wise, or the tiled
 extend kernel in bfloat16). bfloat16 attention over one key head whose rows also hold the
 values (latent attention's cache) runs csrc/attention_shared_keys.cu in every phase.
+Attention without a softmax (a key's weight is the sigmoid of its score) has kernels of its own in
+csrc/attention_sigmoid.cu: tiled in bfloat16 for head sizes 32, 64, 96 and 128, row-wise otherwise.
 
 `attend` is the one call a mixer makes: it takes the step's projection and picks
 rotation, cache write and attention kernels for the step's phase and geometry.
@@ -33,6 +35,7 @@ force_warp_level = False  # tests keep prompts off the tcgen05 kernel to cover t
 force_unfused_decode = False  # tests keep decode steps on the separate rotation / attention / merge kernels
 force_cluster_size = None  # tests fix the CTAs per cluster of the fused decode kernel
 force_shared_key_splits = None  # tests fix the splits of the shared-key kernel's decode step
+force_sigmoid_ranks = None  # tests fix the CTAs per cluster of the sigmoid decode kernel
 prefill_kernel = None  # tests pin the tcgen05 prompt kernel: "pingpong" or "single" (None: the rule in prefill())
 
 
@@ -74,6 +77,8 @@ class Shaping:
     inv_freq, rotary, adjacent_pairs: a rotation of each head's first `rotary` dimensions, angle =
         position * inv_freq[i] (float64 [rotary / 2]); dimension i pairs with i + rotary / 2, or 2i
         with 2i + 1.
+    head_weights: (q weight, k weight), an RMS norm over every query and every key head ahead of the
+        rotation, one weight of the head size each (eps `head_weight_eps`).
     head_norm_eps: each query and key head is divided by its root mean square afterwards.
     """
 
@@ -81,6 +86,8 @@ class Shaping:
     tails: Optional[object] = None
     row_norm: Optional[tuple] = None
     row_eps: float = 0.0
+    head_weights: Optional[tuple] = None
+    head_weight_eps: float = 0.0
     inv_freq: Optional[torch.Tensor] = None
     rotary: int = 0
     adjacent_pairs: bool = False
@@ -278,6 +285,45 @@ def extend(q, kv, out, cu_seqlens, seq_of_token, positions, slots, kv_lens, max_
           "attention_paged_rowwise")
 
 
+def sigmoid(q, k, v, kv, kv_heads: int, dv: int, out, out_stride: int, offset, gate, gate_stride: int, scale: float,
+            window: int, out_scale: float, max_seq_len: int, max_kv_len: int, cu_seqlens, seq_of_token, positions, slots,
+            kv_lens) -> None:
+    """Attention with sigmoid weights (csrc/attention_sigmoid.cu): packed keys k, v, or the cache view kv
+    (one query per sequence where cu_seqlens is None). `out` and `gate` are pointers at first columns."""
+    T, Hq, d = q.shape
+    lib = library.load()
+    paged = kv is not None
+    tail = (ctypes.c_float(scale), window, _ptr(offset), gate, ctypes.c_longlong(gate_stride), ctypes.c_float(out_scale))
+    pages = (_ptr(kv.page_table), kv.page_table.shape[1]) if paged else (None, 0)
+    keys, values = (kv.k, kv.v) if paged else (k, v)
+    page_size = kv.page_size if paged else 64
+    if (not force_rowwise and q.dtype == torch.bfloat16 and lib.lrm_attention_sigmoid_supports(d, dv, page_size)
+            and out_stride % 2 == 0 and all(t.data_ptr() % 16 == 0 for t in (q, keys, values)) and out.value % 4 == 0):
+        if paged and cu_seqlens is None:
+            # the CTAs of a cluster share a sequence's pages; about two CTAs per SM, no CTA without a page
+            seen = min(max_kv_len, abs(window) + 63) if window else max_kv_len
+            clusters = T * kv_heads * -(-(Hq // kv_heads) // 16)
+            ranks = max(1, min(8, -(-seen // 64), -(-2 * SM_COUNT // clusters)))
+            if force_sigmoid_ranks is not None:
+                ranks = force_sigmoid_ranks
+            _done(lib.lrm_attention_sigmoid_decode(_ptr(q), _ptr(keys), _ptr(values), out, ctypes.c_longlong(out_stride),
+                                                   *pages, _ptr(slots), _ptr(kv_lens), T, Hq, kv_heads, d, *tail, ranks,
+                                                   _stream()), "attention_sigmoid_decode")
+            return
+        _done(lib.lrm_attention_sigmoid_tiled(_ptr(q), _ptr(keys), _ptr(values), out, ctypes.c_longlong(out_stride),
+                                              _ptr(cu_seqlens), *pages, _ptr(slots if paged else None),
+                                              _ptr(kv_lens if paged else None), cu_seqlens.numel() - 1, max_seq_len, Hq,
+                                              kv_heads, d, *tail, _stream()), "attention_sigmoid_tiled")
+        return
+    one_each = paged and cu_seqlens is None
+    _done(lib.lrm_attention_sigmoid_rowwise(_ptr(q), _ptr(keys), _ptr(values), out, _code(q.dtype),
+                                            ctypes.c_longlong(out_stride), _ptr(cu_seqlens),
+                                            _ptr(None if one_each else seq_of_token),
+                                            _ptr(None if one_each or not paged else positions), *pages,
+                                            _ptr(slots if paged else None), _ptr(kv_lens if paged else None), T, Hq,
+                                            kv_heads, d, dv, page_size, *tail, _stream()), "attention_sigmoid_rowwise")
+
+
 _cluster_room = {}
 
 
@@ -367,7 +413,7 @@ def decode_fused(qkv, positions, inv_freq, rotary: int, kv, dest_rows, out, slot
 def attend(projected, *, q_heads: int, kv_heads: int, head_dim: int, rotary, ctx, cache, writes_cache: bool,
            cache_entry: int, scale: float, window, projection=None, value_dim=None, bias=None, slopes=None,
            out_scale: float = 1.0, extras=None, values_are_keys: bool = False, shaping: Optional[Shaping] = None,
-           chunk: Optional[int] = None):
+           chunk: Optional[int] = None, sigmoid_weights=None):
     """A layer's attention for one step: position rotation, cache write and attention, with the
     kernels chosen here for the step's phase, dtype and geometry. -> mixed heads [T, q_heads * d].
 
@@ -389,6 +435,8 @@ def attend(projected, *, q_heads: int, kv_heads: int, head_dim: int, rotary, ctx
         stays None) and takes the projection in float32. chunk: positions form chunks of this many,
         counted from position 0, and a query sees only the keys of its own chunk (`window` is then
         what the cache keeps, and the kernels are told the chunk as a negative window).
+    sigmoid_weights: an ops.SigmoidWeights (with a `shaping`): no softmax, see there; the result may then
+        go to columns of a tensor it names.
     """
     from . import ops
     inv_freq, width = rotary if rotary is not None else (None, 0)
@@ -416,7 +464,7 @@ def attend(projected, *, q_heads: int, kv_heads: int, head_dim: int, rotary, ctx
                 projected, q_heads, kv_heads if writes_cache else 0, head_dim, dv, ctx.positions, ctx.runtime.dtype,
                 bias=bias, taps=s.taps, tails=s.tails.state if s.tails is not None else None,
                 cu_seqlens=ctx.cu_seqlens, seq_of_token=ctx.seq_of_token, slots=ctx.slots, row_norm=s.row_norm,
-                row_eps=s.row_eps, inv_freq=s.inv_freq, rotary=s.rotary, adjacent_pairs=s.adjacent_pairs,
+                row_eps=s.row_eps, head_weights=s.head_weights, head_weight_eps=s.head_weight_eps, inv_freq=s.inv_freq, rotary=s.rotary, adjacent_pairs=s.adjacent_pairs,
                 head_norm_eps=s.head_norm_eps, **stored)
         else:
             q, k, v = ops.qkv_bias_store(projected, bias, q_heads, kv_heads if writes_cache else 0, head_dim, dv,
@@ -425,6 +473,13 @@ def attend(projected, *, q_heads: int, kv_heads: int, head_dim: int, rotary, ctx
             if writes_cache:
                 ctx.fresh_kv[cache_entry] = (k, k if values_are_keys else v)
             k, v = ctx.fresh_kv[cache_entry]
+        if sigmoid_weights is not None:
+            where = dict(k=k, v=v) if prefill_phase else dict(kv=cache, slots=ctx.slots, kv_lens=ctx.kv_lens,
+                                                              max_kv_len=ctx.max_kv_len)
+            if phase != "decode":
+                where.update(cu_seqlens=ctx.cu_seqlens, seq_of_token=ctx.seq_of_token, positions=ctx.positions)
+            return ops.attention_sigmoid(q, sigmoid_weights, scale, window, out_scale, ctx.max_seq_len, **where)
+        if prefill_phase:
             return ops.attention_prefill(q, k, v, ctx.cu_seqlens, ctx.seq_of_token, ctx.max_seq_len, scale, window,
                                          slopes, out_scale, extras)
         if phase == "decode":

@@ -305,3 +305,36 @@ def gemm_bf16(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, mode: in
         return
     _done(lib.lrm_gemm_bf16_mma(_ptr(x), _ptr(weight), _ptr(out), M, N, K, mode, _stream()),
           "gemm_bf16_mma")
+
+
+def gemm_bf16_grouped(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, group_cols: int) -> None:
+    """float32 out [T, N] from the inputs x [G, T, K] and one stacked weight [N, K]: columns i * group_cols
+    .. of out belong to x[i]. The kernels of gemm_bf16 with a row offset into x per column tile."""
+    G, T, K = x.shape
+    N = weight.shape[0]
+    lib = library.load()
+    aligned = not force_tiled and x.data_ptr() % 16 == 0 and weight.data_ptr() % 16 == 0
+    stream_ok = aligned and bool(lib.lrm_gemm_bf16_stream_supports(T, N, K))
+    umma_ok = aligned and bool(lib.lrm_gemm_bf16_umma_supports(T, N, K))
+    if stream_ok and umma_ok and T > STREAM_ROWS and not force_stream:
+        stream_ok = not _few_rows_plan(T, N, K, 1)[0]
+    if stream_ok:
+        _done(lib.lrm_gemm_bf16_stream_grouped(_ptr(x), _ptr(weight), _ptr(out), T, N, K, 1, group_cols, T, _stream()),
+              "gemm_bf16_stream_grouped")
+        return
+    if umma_ok:
+        tile = tile_choice(T, N, K, 1, pair_room() if T > 64 else 0)
+        width = {0: 128, 1: 256, 2: 256, 3: 192, PAIR: 256}[tile]
+        if group_cols % width:
+            tile = 1 if group_cols % 256 == 0 else 0
+        mark_status_dirty()
+        if tile == PAIR:
+            _done(lib.lrm_gemm_bf16_umma_pair_grouped(_ptr(x), _ptr(weight), _ptr(out), T, G * T, N, K, 1, group_cols, T,
+                                                      _ptr(_status_word(x.device)), _stream()),
+                  "gemm_bf16_umma_pair_grouped")
+        else:
+            _done(lib.lrm_gemm_bf16_umma_grouped(_ptr(x), _ptr(weight), _ptr(out), T, G * T, N, K, 1, tile, group_cols, T,
+                                                 _ptr(_status_word(x.device)), _stream()), "gemm_bf16_umma_grouped")
+        return
+    _done(lib.lrm_gemm_bf16_mma_grouped(_ptr(x), _ptr(weight), _ptr(out), T, N, K, 1, group_cols, T, _stream()),
+          "gemm_bf16_mma_grouped")

@@ -148,38 +148,99 @@ def rms_norm_add_(stream: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, e
     return out
 
 
-def layer_norm(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, eps: float, out_dtype: torch.dtype,
-               rows: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """(x - mean) / sqrt(variance + eps) * weight + bias over float32 rows [T, h] (all, or those `rows`
-    names); weight and bias float32 [h]. -> [T or len(rows), h] in `out_dtype`."""
+def _check_norm(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], partials: Optional[torch.Tensor],
+                what: str):
+    """Shared checks of the layer norms; -> (planes to add, elements between them)."""
     _check(x, "x", torch.float32, 2)
-    _check(weight, "weight", torch.float32, 1)
-    _check(bias, "bias", torch.float32, 1)
+    for name, t in (("weight", weight), ("bias", bias)):
+        if name == "weight" or t is not None:
+            _check(t, name, torch.float32, 1)
+            if t.numel() != x.shape[1]:
+                raise InvalidError(f"{what}: {name} must have one entry per column")
+    if partials is None:
+        return 0, 0
+    _check(partials, "partials", torch.float32, 3)
+    if tuple(partials.shape[1:]) != tuple(x.shape):
+        raise InvalidError(f"{what}: partials must be [n, T, h]")
+    return partials.shape[0], x.numel()
+
+
+def layer_norm(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], eps: float, out_dtype: torch.dtype,
+               rows: Optional[torch.Tensor] = None, partials: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """(x - mean) / sqrt(variance + eps) * weight [+ bias] over float32 rows [T, h] (all, or those `rows`
+    names); weight and bias float32 [h]. `partials` float32 [n, T, h]: slices that are first added into
+    the rows (and written back, unless rows are gathered). -> [T or len(rows), h] in `out_dtype`."""
+    n_partials, stride = _check_norm(x, weight, bias, partials, "layer_norm")
     hidden = x.shape[1]
-    if weight.numel() != hidden or bias.numel() != hidden:
-        raise InvalidError("layer_norm: weight and bias must have one entry per column")
     n_rows = x.shape[0]
     if rows is not None:
         _check(rows, "rows", torch.int32, 1)
         n_rows = rows.numel()
     out = _activation(n_rows, hidden, out_dtype, x.device)
     _done(_lib().lrm_layer_norm(_ptr(x), _ptr(weight), _ptr(bias), _ptr(out), _code(out_dtype), _ptr(rows), n_rows,
-                                hidden, ctypes.c_float(eps), _stream()), "layer_norm")
+                                hidden, ctypes.c_float(eps), _ptr(partials), n_partials, ctypes.c_longlong(stride),
+                                _stream()), "layer_norm")
     return out
 
 
-def layer_norm_add_(stream: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, eps: float,
-                    mult: float = 1.0, cast_dtype: Optional[torch.dtype] = None) -> Optional[torch.Tensor]:
+def _check_taps(taps: torch.Tensor, tails: Optional[torch.Tensor], width: int, what: str) -> int:
+    """Taps float32 [n, width] and, for n > 1, tails float32 [slots, n - 1, width]; -> n."""
+    _check(taps, "taps", torch.float32, 2)
+    n = taps.shape[0]
+    if taps.shape[1] != width:
+        raise InvalidError(f"{what}: one tap per channel in every row of taps")
+    if n > 1:
+        _check(tails, "tails", torch.float32, 3)
+        if tuple(tails.shape[1:]) != (n - 1, width):
+            raise InvalidError(f"{what}: tails must be [slots, taps - 1, channels]")
+    return n
+
+
+def layer_norm_conv(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], eps: float,
+                    out_dtype: torch.dtype, taps: torch.Tensor, tails: torch.Tensor, slots: torch.Tensor,
+                    partials: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """input_conv(layer_norm(x)) for a step of one token per sequence, in one pass: row b of x [B, h] is
+    sequence b's token; taps float32 [n, h] with n > 1, tails float32 [slots, n - 1, h]."""
+    n_partials, stride = _check_norm(x, weight, bias, partials, "layer_norm_conv")
+    B, hidden = x.shape
+    n = _check_taps(taps, tails, hidden, "layer_norm_conv")
+    _check(slots, "slots", torch.int32, 1)
+    if n < 2 or slots.numel() != B:
+        raise InvalidError("layer_norm_conv: several taps, and one sequence per row")
+    out = _activation(B, hidden, out_dtype, x.device)
+    _done(_lib().lrm_layer_norm_conv(_ptr(x), _ptr(weight), _ptr(bias), _ptr(out), _code(out_dtype), _ptr(partials),
+                                     n_partials, ctypes.c_longlong(stride), _ptr(taps), n, _ptr(tails), _ptr(slots), B,
+                                     hidden, ctypes.c_float(eps), _stream()), "layer_norm_conv")
+    return out
+
+
+def input_conv(h: torch.Tensor, taps: torch.Tensor, tails: Optional[torch.Tensor], cu_seqlens: torch.Tensor,
+               seq_of_token: torch.Tensor, slots: torch.Tensor) -> torch.Tensor:
+    """h + conv(h), a causal convolution over time per channel: h [T, W] packed sequences, taps float32
+    [n, W] (the last row the current token's); rows before a sequence's first token of the step come
+    from `tails` float32 [slots, n - 1, W] (zeros at its start), which the kernel moves on."""
+    _check(h, "h", dims=2)
+    T, W = h.shape
+    n = _check_taps(taps, tails, W, "input_conv")
+    for name, t in (("cu_seqlens", cu_seqlens), ("seq_of_token", seq_of_token), ("slots", slots)):
+        _check(t, name, torch.int32, 1)
+    out = _activation(T, W, h.dtype, h.device)
+    _done(_lib().lrm_input_conv(_ptr(h), _code(h.dtype), _ptr(taps), n, _ptr(tails if n > 1 else None), _ptr(out),
+                                _ptr(cu_seqlens), _ptr(seq_of_token), _ptr(slots), T, W, _stream()), "input_conv")
+    return out
+
+
+def layer_norm_add_(stream: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor],
+                    eps: float, mult: float = 1.0, cast_dtype: Optional[torch.dtype] = None) -> Optional[torch.Tensor]:
     """stream += mult * layer_norm(y), in place (both float32 [T, h]: a norm behind a sublayer). With
     `cast_dtype` the updated rows are also returned in that type, for a sublayer that reads the
     stream itself."""
     _check(stream, "stream", torch.float32, 2)
     _check(y, "y", torch.float32, 2)
-    _check(weight, "weight", torch.float32, 1)
-    _check(bias, "bias", torch.float32, 1)
+    _check_norm(stream, weight, bias, None, "layer_norm_add_")
     T, hidden = stream.shape
-    if tuple(y.shape) != (T, hidden) or weight.numel() != hidden or bias.numel() != hidden:
-        raise InvalidError("layer_norm_add_: y must match the stream, weight and bias its rows")
+    if tuple(y.shape) != (T, hidden):
+        raise InvalidError("layer_norm_add_: y must match the stream")
     out = _activation(T, hidden, cast_dtype, stream.device) if cast_dtype is not None else None
     _done(_lib().lrm_layer_norm_add(_ptr(stream), _ptr(y), _ptr(weight), _ptr(bias), ctypes.c_float(mult), _ptr(out),
                                     _code(cast_dtype or torch.float32), T, hidden, ctypes.c_float(eps), _stream()),
@@ -248,6 +309,31 @@ def linear(x: torch.Tensor, weight: torch.Tensor, epilogue: str = STORE,
     return out
 
 
+GROUP_MULTIPLE = 128  # a grouped product's columns per input are a multiple of this: whole tiles of one input
+
+
+def linear_grouped(x: torch.Tensor, weight: torch.Tensor, group_cols: int) -> torch.Tensor:
+    """Several products in one launch: x [G, T, K] (G inputs), weight [N, K], the matrices of all inputs one
+    above the other: columns i * group_cols .. (i + 1) * group_cols of the result are x[i] . (those rows
+    of weight)^T. group_cols a multiple of GROUP_MULTIPLE; the last input may have fewer. -> float32 [T, N]."""
+    _check(x, "x", dims=3)
+    _check(weight, "weight", dims=2)
+    G, T, K = x.shape
+    N = weight.shape[0]
+    if weight.shape[1] != K or weight.dtype != x.dtype:
+        raise InvalidError("linear_grouped: inputs and matrices do not agree")
+    if group_cols <= 0 or group_cols % GROUP_MULTIPLE or not (G - 1) * group_cols < N <= G * group_cols:
+        raise InvalidError("linear_grouped: whole tiles per input, and rows of weight for every input")
+    out = torch.empty((T, N), dtype=torch.float32, device=x.device)
+    if x.dtype == torch.float32:
+        _done(_lib().lrm_gemm_f32_grouped(_ptr(x), _ptr(weight), _ptr(out), T, N, K, 0, group_cols, T, _stream()),
+              "gemm_f32_grouped")
+        return out
+    from . import gemm_dispatch
+    gemm_dispatch.gemm_bf16_grouped(x, weight, out, group_cols)
+    return out
+
+
 def linear_slices(x: torch.Tensor, weight: torch.Tensor) -> Optional[torch.Tensor]:
     """x . weight^T as float32 partial products over K slices [slices, M, N] (their sum in plane
     order is the product), or None when this product is not cut. Only narrow bfloat16 products
@@ -279,6 +365,33 @@ def scale_(x: torch.Tensor, factor: float) -> torch.Tensor:
     _done(_lib().lrm_scale_inplace(_ptr(x), ctypes.c_float(factor), ctypes.c_longlong(x.numel()), _stream()),
           "scale_")
     return x
+
+
+def softcap_(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """x = cap * tanh(x / cap) in place (float32)."""
+    _check(x, "x", torch.float32)
+    _done(_lib().lrm_softcap_inplace(_ptr(x), ctypes.c_float(cap), ctypes.c_longlong(x.numel()), _stream()), "softcap_")
+    return x
+
+
+def stream_swap_(x: torch.Tensor, base: torch.Tensor, dtype: torch.dtype,
+                 partials: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """The stream x (float32 [T, h], plus the slices `partials` [n, T, h] that belong to it) in the
+    activation type `dtype`; x itself becomes `base` (float32 [T, h])."""
+    _check(x, "x", torch.float32, 2)
+    _check(base, "base", torch.float32, 2)
+    if base.shape != x.shape:
+        raise InvalidError("stream_swap_: base must match the stream")
+    n = 0
+    if partials is not None:
+        _check(partials, "partials", torch.float32, 3)
+        if tuple(partials.shape[1:]) != tuple(x.shape):
+            raise InvalidError("stream_swap_: partials must be [n, T, h]")
+        n = partials.shape[0]
+    out = _activation(x.shape[0], x.shape[1], dtype, x.device)
+    _done(_lib().lrm_stream_swap(_ptr(x), _ptr(base), _ptr(partials), n, _ptr(out), _code(dtype),
+                                 ctypes.c_longlong(x.numel()), _stream()), "stream_swap_")
+    return out
 
 
 def silu_mul(gate_up: torch.Tensor, block: int) -> torch.Tensor:
@@ -554,22 +667,23 @@ def shaped_qkv_store(qkv: torch.Tensor, q_heads: int, kv_heads: int, head_dim: i
                      taps: Optional[torch.Tensor] = None, tails: Optional[torch.Tensor] = None,
                      cu_seqlens: Optional[torch.Tensor] = None, seq_of_token: Optional[torch.Tensor] = None,
                      slots: Optional[torch.Tensor] = None, row_norm=None, row_eps: float = 0.0,
-                     inv_freq: Optional[torch.Tensor] = None, rotary: int = 0, adjacent_pairs: bool = False,
+                     head_weights=None, head_weight_eps: float = 0.0, inv_freq: Optional[torch.Tensor] = None, rotary: int = 0, adjacent_pairs: bool = False,
                      head_norm_eps: Optional[float] = None, kv=None, dest_rows: Optional[torch.Tensor] = None,
                      keep_packed: bool = True):
-    """Split a fused [T, Hq*d + Hk*d + Hk*dv] projection (float32, or `out_dtype`) whose queries and
-    keys are shaped on the way, each step only if asked for and in this order: `bias` (float32
+    """Split a fused [T, Hq*d + Hk*d + Hk*dv (+ more)] projection (float32, or `out_dtype`; columns behind
+    the row are left alone) whose queries and keys are shaped on the way, each step only if asked for and in this order: `bias` (float32
     [row]); a causal convolution per channel (`taps` float32 [n, row], the last row the current
     token's, with the sequences' `tails`
     float32 [slots, n - 1, row] of unbiased projections, rewritten afterwards); an RMS norm over all
-    query columns and one over all key columns (`row_norm` = (q weight, k weight), `row_eps`); the
-    rotation of each head's first `rotary` dimensions by `inv_freq` (float64 [rotary/2]; split halves,
+    query columns and one over all key columns (`row_norm` = (q weight, k weight), `row_eps`); an RMS
+    norm over every query and every key head (`head_weights` = (q weight, k weight), float32 [d] each,
+    `head_weight_eps`); the rotation of each head's first `rotary` dimensions by `inv_freq` (float64 [rotary/2]; split halves,
     or neighbours with `adjacent_pairs`); each head divided by its root mean square
     (`head_norm_eps`). Returns (q [T,Hq,d], k, v) like qkv_bias_store, and writes the cache view."""
     _check(qkv, "qkv", dims=2)
     T = qkv.shape[0]
     width = q_heads * head_dim + kv_heads * (head_dim + value_dim)
-    if qkv.shape[1] != width:
+    if qkv.shape[1] < width:
         raise InvalidError("shaped_qkv_store: qkv width does not match the head geometry")
     _check(positions, "positions", torch.int32, 1)
     if bias is not None:
@@ -600,6 +714,13 @@ def shaped_qkv_store(qkv: torch.Tensor, q_heads: int, kv_heads: int, head_dim: i
                 raise InvalidError("shaped_qkv_store: the key norm's weight covers all key columns")
         else:
             k_norm = None
+    q_head = k_head = None
+    if head_weights is not None:
+        q_head, k_head = head_weights
+        for name, t in (("q head norm", q_head), ("k head norm", k_head)):
+            _check(t, name, torch.float32, 1)
+            if t.numel() != head_dim:
+                raise InvalidError(f"shaped_qkv_store: the {name}'s weight has one entry per head dimension")
     if rotary:
         _check(inv_freq, "inv_freq", torch.float64, 1)
         if inv_freq.numel() != rotary // 2 or rotary % 2 or rotary > head_dim:
@@ -622,10 +743,11 @@ def shaped_qkv_store(qkv: torch.Tensor, q_heads: int, kv_heads: int, head_dim: i
                 or (value_dim and tuple(v_pages.shape[1:]) != (kv_heads, page_size, value_dim))):
             raise InvalidError("shaped_qkv_store: cache pages do not match the head geometry")
     _done(_lib().lrm_shaped_qkv_store(
-        _ptr(qkv), _code(qkv.dtype), _ptr(bias), _ptr(taps), n, _ptr(tails if n > 1 else None),
+        _ptr(qkv), _code(qkv.dtype), ctypes.c_longlong(qkv.shape[1]), _ptr(bias), _ptr(taps), n,
+        _ptr(tails if n > 1 else None),
         _ptr(cu_seqlens if n > 1 else None), _ptr(seq_of_token if n > 1 else None), _ptr(slots if n > 1 else None),
-        _ptr(positions), _ptr(q_norm), _ptr(k_norm), ctypes.c_float(row_eps), _ptr(inv_freq if rotary else None),
-        rotary, int(bool(adjacent_pairs)), int(head_norm_eps is not None),
+        _ptr(positions), _ptr(q_norm), _ptr(k_norm), ctypes.c_float(row_eps), _ptr(q_head), _ptr(k_head),
+        ctypes.c_float(head_weight_eps), _ptr(inv_freq if rotary else None), rotary, int(bool(adjacent_pairs)), int(head_norm_eps is not None),
         ctypes.c_float(head_norm_eps if head_norm_eps is not None else 0.0), _ptr(q), _ptr(k), _ptr(v),
         _ptr(k_pages), _ptr(v_pages), _ptr(dest_rows if k_pages is not None else None), _code(out_dtype), T, q_heads,
         kv_heads, head_dim, value_dim, page_size, _stream()), "shaped_qkv_store")
@@ -793,6 +915,126 @@ def general_delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: tor
     _done(_lib().lrm_general_delta_scan(_ptr(q), _ptr(k), _ptr(v), _ptr(g), _ptr(look), _ptr(put), _ptr(state),
                                         _ptr(out), _ptr(cu_seqlens), _ptr(slots), slots.numel(), H, d, dv, _stream()),
           "general_delta_scan")
+    return out
+
+
+def _check_scan(state: torch.Tensor, cu_seqlens: torch.Tensor, slots: torch.Tensor, shape, what: str) -> None:
+    _check(state, "state", torch.float32, 4)
+    _check(cu_seqlens, "cu_seqlens", torch.int32, 1)
+    _check(slots, "slots", torch.int32, 1)
+    if tuple(state.shape[1:]) != tuple(shape):
+        raise InvalidError(f"{what}: state must be [slots, heads, head_dim, value_dim]")
+
+
+def bonus_state_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, g: torch.Tensor, bonus: torch.Tensor,
+                     state: torch.Tensor, cu_seqlens: torch.Tensor, slots: torch.Tensor, value_dim: int) -> torch.Tensor:
+    """A state that is read before it is written: o = (S + diag(bonus) k v^T)^T q, then S <- diag(g) S + k v^T
+    (float32 [slots, H, d, dv], updated in place). q, k [H*d] and v [H*dv] are the columns at q_off, k_off
+    and v_off of a float32 activation proj [T, W]; g float32 [T, H*d]; bonus float32 [H, d]. -> o [T,H,dv]."""
+    _check(proj, "proj", torch.float32, 2)
+    _check(g, "g", torch.float32, 2)
+    _check(bonus, "bonus", torch.float32, 2)
+    T, W = proj.shape
+    H, d = bonus.shape
+    _check_scan(state, cu_seqlens, slots, (H, d, value_dim), "bonus_state_scan")
+    if tuple(g.shape) != (T, H * d) or max(q_off, k_off) + H * d > W or v_off + H * value_dim > W:
+        raise InvalidError("bonus_state_scan: shapes do not agree")
+    out = _f32((T, H, value_dim), proj.device)
+    _done(_lib().lrm_bonus_state_scan(_column_ptr(proj, q_off), _column_ptr(proj, k_off), ctypes.c_longlong(W),
+                                      _column_ptr(proj, v_off), ctypes.c_longlong(W), _ptr(g), _ptr(bonus), _ptr(state),
+                                      _ptr(out), _ptr(cu_seqlens), _ptr(slots), slots.numel(), H, d, value_dim,
+                                      _stream()), "bonus_state_scan")
+    return out
+
+
+def head_decay_delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, step: torch.Tensor,
+                          state: torch.Tensor, cu_seqlens: torch.Tensor, slots: torch.Tensor) -> torch.Tensor:
+    """The delta rule with one decay per head and token on the per-sequence, per-head state (float32
+    [slots, H, d, dv], updated in place): S <- decay S; S <- S + k (step (v - S^T k))^T; o = S^T q. q, k
+    float32 [T,KH,d] (head h reads head h // (H/KH)), v [T,H,dv], decay and step [T,H]. -> o [T,H,dv]."""
+    for name, t, dims in (("q", q, 3), ("k", k, 3), ("v", v, 3), ("decay", decay, 2), ("step", step, 2)):
+        _check(t, name, torch.float32, dims)
+    T, KH, d = q.shape
+    H, dv = v.shape[1], v.shape[2]
+    _check_scan(state, cu_seqlens, slots, (H, d, dv), "head_decay_delta_scan")
+    if k.shape != q.shape or v.shape[0] != T or H % KH or tuple(decay.shape) != (T, H) or tuple(step.shape) != (T, H):
+        raise InvalidError("head_decay_delta_scan: shapes do not agree")
+    out = _f32((T, H, dv), q.device)
+    _done(_lib().lrm_head_decay_delta_scan(_ptr(q), _ptr(k), _ptr(v), _ptr(decay), _ptr(step), _ptr(state), _ptr(out),
+                                           _ptr(cu_seqlens), _ptr(slots), slots.numel(), H, KH, d, dv, _stream()),
+          "head_decay_delta_scan")
+    return out
+
+
+def head_decay_delta_prepare(proj: torch.Tensor, conv_off: int, b_off: int, a_off: int, dt_bias: torch.Tensor,
+                             rate: torch.Tensor, taps: torch.Tensor, tails: Optional[torch.Tensor],
+                             cu_seqlens: torch.Tensor, seq_of_token: torch.Tensor, slots: torch.Tensor, heads: int,
+                             kv_heads: int, head_dim: int, value_dim: int, unit_eps: float, q_scale: float,
+                             one_each: bool = False):
+    """Inputs of the delta rule with one decay per head from a fused projection [T, W]: the columns
+    conv_off .. (q | k | v channels) pass a short causal convolution (taps float32 [n, C]; inputs before
+    the step come from, and afterwards go to, `tails` float32 [slots, n-1, C]) and SiLU; q and k become
+    unit vectors per head (q also times q_scale); step = sigmoid of the H columns at b_off; decay =
+    exp(-rate_h softplus(a_h + dt_bias_h)) of those at a_off. `one_each`: the step brings one token per
+    sequence. -> q, k [T,G,d], v [T,H,dv], decay, step [T,H], all float32."""
+    _check(proj, "proj", dims=2)
+    T, W = proj.shape
+    C = 2 * kv_heads * head_dim + heads * value_dim
+    for name, t in (("dt_bias", dt_bias), ("rate", rate)):
+        _check(t, name, torch.float32, 1)
+        if t.numel() != heads:
+            raise InvalidError(f"head_decay_delta_prepare: one entry of {name} per head")
+    n = _check_taps(taps, tails, C, "head_decay_delta_prepare")
+    for name, t in (("cu_seqlens", cu_seqlens), ("seq_of_token", seq_of_token), ("slots", slots)):
+        _check(t, name, torch.int32, 1)
+    if conv_off + C > W or max(a_off, b_off) + heads > W or (one_each and slots.numel() != T):
+        raise InvalidError("head_decay_delta_prepare: columns outside the projection")
+    dev = proj.device
+    q, k = _f32((T, kv_heads, head_dim), dev), _f32((T, kv_heads, head_dim), dev)
+    v, decay, step = _f32((T, heads, value_dim), dev), _f32((T, heads), dev), _f32((T, heads), dev)
+    _done(_lib().lrm_head_decay_delta_prepare(
+        _ptr(proj), _code(proj.dtype), ctypes.c_longlong(W), conv_off, b_off, a_off, _ptr(dt_bias), _ptr(rate), _ptr(taps),
+        n, _ptr(tails if n > 1 else None), _ptr(cu_seqlens), _ptr(seq_of_token), _ptr(slots), _ptr(q), _ptr(k), _ptr(v),
+        _ptr(decay), _ptr(step), T, heads, kv_heads, head_dim, value_dim, ctypes.c_float(unit_eps),
+        ctypes.c_float(q_scale), int(one_each), _stream()), "head_decay_delta_prepare")
+    if n > 1 and not one_each:
+        conv_tail_update_(proj, conv_off, C, n, tails, cu_seqlens, slots)
+    return q, k, v, decay, step
+
+
+def token_mixes(h: torch.Tensor, mix: torch.Tensor, last: torch.Tensor, cu_seqlens: torch.Tensor,
+                seq_of_token: torch.Tensor, slots: torch.Tensor) -> torch.Tensor:
+    """Several token shifts in one pass: out[s, t] = h[t] + (h[t-1] - h[t]) * mix[s], mix float32 [S, W]; `last`
+    as for token_shift (read for a sequence's first token, and rewritten). -> [S, T, W] in h's type."""
+    _check(h, "h", dims=2)
+    _check(mix, "mix", torch.float32, 2)
+    _check(last, "last", torch.float32, 3)
+    T, W = h.shape
+    if mix.shape[1] != W or tuple(last.shape[1:]) != (1, W):
+        raise InvalidError("token_mixes: shapes do not agree")
+    for name, t in (("cu_seqlens", cu_seqlens), ("seq_of_token", seq_of_token), ("slots", slots)):
+        _check(t, name, torch.int32, 1)
+    out = torch.empty((mix.shape[0], T, W), dtype=h.dtype, device=h.device)
+    _done(_lib().lrm_token_mixes(_ptr(h), _code(h.dtype), _ptr(mix), mix.shape[0], _ptr(last), _ptr(out),
+                                 ctypes.c_longlong(T * W), _ptr(cu_seqlens), _ptr(seq_of_token), _ptr(slots), T, W,
+                                 _stream()), "token_mixes")
+    return out
+
+
+def decay_product(proj: torch.Tensor, column: int, weight: torch.Tensor, bias: torch.Tensor) -> torch.Tensor:
+    """exp(-exp(weight . tanh(z) + bias)) with z the columns column .. column + K of a float32 activation
+    proj [T, W], weight [N, K] (float32: true 32-bit; bfloat16: tanh rounded to it), bias float32 [N].
+    -> float32 [T, N]."""
+    _check(proj, "proj", torch.float32, 2)
+    _check(weight, "weight", dims=2)
+    _check(bias, "bias", torch.float32, 1)
+    T, W = proj.shape
+    N, K = weight.shape
+    if column < 0 or column + K > W or bias.numel() != N:
+        raise InvalidError("decay_product: shapes do not agree")
+    out = _f32((T, N), proj.device)
+    _done(_lib().lrm_decay_product(_column_ptr(proj, column), ctypes.c_longlong(W), _ptr(weight), _code(weight.dtype),
+                                   _ptr(bias), _ptr(out), T, N, K, _stream()), "decay_product")
     return out
 
 
@@ -1087,16 +1329,28 @@ def latent_prepare(proj: torch.Tensor, q_column: int, q_weight: Optional[torch.T
 GATE_SILU, GATE_SIGMOID = 1, 2
 
 
+def _output_columns(out: Optional[torch.Tensor], column: int, rows: int, width: int, dtype: torch.dtype, device):
+    """(tensor, pointer) a kernel writes [rows, width] to: a new activation, or columns column .. of `out`."""
+    if out is None:
+        out = _activation(rows, width, dtype, device)
+        return out, _ptr(out)
+    _check(out, "out", dtype, 2)
+    if out.shape[0] != rows or column < 0 or column + width > out.shape[1]:
+        raise InvalidError("output columns outside the given tensor")
+    return out, _column_ptr(out, column)
+
+
 def head_norm_gate(o: torch.Tensor, eps: float, out_dtype: torch.dtype, weight: Optional[torch.Tensor] = None,
                    gate: Optional[torch.Tensor] = None, gate_column: int = 0, gate_act: int = GATE_SILU,
                    out_scale: float = 1.0, value_dim: Optional[int] = None, floor: Optional[torch.Tensor] = None,
-                   floor_eps: float = 0.0) -> torch.Tensor:
+                   floor_eps: float = 0.0, out: Optional[torch.Tensor] = None, out_column: int = 0) -> torch.Tensor:
     """Per token and head: o / sqrt(mean(o^2) + eps) [* weight] [* act(gate)] * out_scale, o float32
     [T,H,dv] -> [T, H*dv] in `out_dtype`. `gate` is a [T, W] activation whose columns gate_column ..
     gate_column + H*dv hold the gate's pre-activation; act: GATE_SILU or GATE_SIGMOID. `weight`
     float32 [dv] (shared by the heads) or [H*dv]. `value_dim` < o.shape[2]: only the first value_dim
     columns of a head are values. With `floor` float32 [T,H] a head is first divided by
-    max(|o[value_dim]|, floor) + floor_eps: column value_dim is then a normalizer's read-out."""
+    max(|o[value_dim]|, floor) + floor_eps: column value_dim is then a normalizer's read-out. With `out`
+    ([T, W], out_dtype) the result goes to its columns out_column .. instead of a tensor of its own."""
     _check(o, "o", torch.float32, 3)
     T, H, o_stride = o.shape
     dv = o_stride if value_dim is None else value_dim
@@ -1120,11 +1374,11 @@ def head_norm_gate(o: torch.Tensor, eps: float, out_dtype: torch.dtype, weight: 
         if gate.shape[0] != T or gate_column + H * dv > gate.shape[1]:
             raise InvalidError("head_norm_gate: gate columns outside the activation")
         gate_ptr, stride = _column_ptr(gate, gate_column), gate.shape[1]
-    out = _activation(T, H * dv, out_dtype, o.device)
+    out, out_ptr = _output_columns(out, out_column, T, H * dv, out_dtype, o.device)
     _done(_lib().lrm_head_norm_gate(_ptr(o), o_stride, _ptr(weight), w_stride, _ptr(floor), ctypes.c_float(floor_eps),
-                                    gate_ptr, gate_code, ctypes.c_longlong(stride), gate_act, _ptr(out),
+                                    gate_ptr, gate_code, ctypes.c_longlong(stride), gate_act, out_ptr,
                                     _code(out_dtype), T, H, dv, ctypes.c_float(eps), ctypes.c_float(out_scale),
-                                    _stream()), "head_norm_gate")
+                                    ctypes.c_longlong(out.shape[1]), _stream()), "head_norm_gate")
     return out
 
 
@@ -1403,6 +1657,68 @@ def attention_extend(q: torch.Tensor, kv, cu_seqlens: torch.Tensor, seq_of_token
     _check_extras(extras, Hq)
     attention_dispatch.extend(q, kv, out, cu_seqlens, seq_of_token, positions, slots, kv_lens, max_seq_len,
                               scale, window or 0, slopes, out_scale, extras)
+    return out
+
+
+@dataclass(frozen=True)
+class SigmoidWeights:
+    """Attention without a softmax: a visible key's weight is sigmoid(score + offset_h), not normalized
+    over the keys. offset float32 [query heads]; gate (tensor float32 [T, W], column): the result is
+    multiplied by sigmoid of those columns; out (tensor [T, W'], column): where the result goes (None: a
+    tensor of its own)."""
+
+    offset: torch.Tensor
+    gate: Optional[Tuple[torch.Tensor, int]] = None
+    out: Optional[Tuple[torch.Tensor, int]] = None
+
+
+def attention_sigmoid(q: torch.Tensor, weights: SigmoidWeights, scale: float, window: Optional[int], out_scale: float,
+                      max_seq_len: int, k: Optional[torch.Tensor] = None, v: Optional[torch.Tensor] = None, kv=None,
+                      cu_seqlens: Optional[torch.Tensor] = None, seq_of_token: Optional[torch.Tensor] = None,
+                      positions: Optional[torch.Tensor] = None, slots: Optional[torch.Tensor] = None,
+                      kv_lens: Optional[torch.Tensor] = None, max_kv_len: int = 0) -> torch.Tensor:
+    """sum over the visible keys of sigmoid(scale q.k + offset_h) v [* sigmoid(gate)] * out_scale -> [T, Hq*dv].
+    With k, v (packed [T, Hk, d | dv], sequences from position 0: cu_seqlens, seq_of_token) a prompt; with
+    the cache view `kv` one query per sequence (slots, kv_lens), or, where cu_seqlens, seq_of_token and
+    positions are given too, a portion per sequence whose keys the cache already holds."""
+    _check(q, "q", dims=3)
+    T, Hq, d = q.shape
+    _check(weights.offset, "offset", torch.float32, 1)
+    if weights.offset.numel() != Hq:
+        raise InvalidError("attention_sigmoid: one offset per query head")
+    if kv is None:
+        _check(k, "k", q.dtype, 3)
+        _check(v, "v", q.dtype, 3)
+        heads, dv = k.shape[1], v.shape[2]
+        if k.shape[0] != T or k.shape[2] != d or k.shape[:2] != v.shape[:2] or Hq % heads:
+            raise InvalidError("attention_sigmoid: q, k, v shapes do not agree")
+    else:
+        _check(kv.k, "k pages", q.dtype, 4)
+        _check(kv.v, "v pages", q.dtype, 4)
+        _check(kv.page_table, "page table", torch.int32, 2)
+        heads, dv = kv.kv_heads, _value_dim(kv)
+        if tuple(kv.k.shape[1:]) != (heads, kv.page_size, d) or Hq % heads:
+            raise InvalidError("attention_sigmoid: cache pages do not match the query geometry")
+        for name, t in (("slots", slots), ("kv_lens", kv_lens)):
+            _check(t, name, torch.int32, 1)
+    if kv is None or cu_seqlens is not None:
+        _check(cu_seqlens, "cu_seqlens", torch.int32, 1)
+        _check(seq_of_token, "seq_of_token", torch.int32, 1)
+    elif slots.numel() != T:
+        raise InvalidError("attention_sigmoid: one query per sequence")
+    gate, gate_stride = ctypes.c_void_p(0), 0
+    if weights.gate is not None:
+        tensor, column = weights.gate
+        _check(tensor, "gate", torch.float32, 2)
+        if tensor.shape[0] != T or column < 0 or column + Hq * dv > tensor.shape[1]:
+            raise InvalidError("attention_sigmoid: gate columns outside the activation")
+        gate, gate_stride = _column_ptr(tensor, column), tensor.shape[1]
+    given, column = weights.out if weights.out is not None else (None, 0)
+    out, out_ptr = _output_columns(given, column, T, Hq * dv, q.dtype, q.device)
+    from . import attention_dispatch
+    attention_dispatch.sigmoid(q, k, v, kv, heads, dv, out_ptr, out.shape[1], weights.offset, gate, gate_stride, scale,
+                               window or 0, out_scale, max_seq_len, max_kv_len, cu_seqlens, seq_of_token, positions,
+                               slots, kv_lens)
     return out
 
 

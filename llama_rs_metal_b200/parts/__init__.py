@@ -5,8 +5,8 @@ from .norm import LayerNorm, RMSNorm, StreamCast
 from .rope import DistancePenalty, RotaryEmbedding
 from .attention import Attention
 from .mlp import GatedMLP, PlainMLP
-from .recurrent import (GatedDeltaRule, GatedLinearRecurrence, GeneralizedDeltaRule, MatrixMemory, Retention,
-                        StateSpaceDuality)
+from .recurrent import (GatedDeltaRule, GatedLinearRecurrence, GeneralizedDeltaRule, HeadDecayDeltaRule, MatrixMemory,
+                        Retention, StateSpaceDuality, TimeMix)
 from .latent import LatentAttention
 from .parallel import ParallelMixer
 from .moe import MixtureOfExperts
@@ -19,4 +19,4 @@ __all__ = ["Block", "CompositeRequest", "FeedForward", "KeyValueRequest", "Layer
            "GatedLinearRecurrence", "LatentAttention",
            "ParallelMixer", "MixtureOfExperts", "PreNormBlock", "PreNormMixerBlock", "SandwichNormBlock",
            "SandwichNormMixerBlock", "LayerNorm", "StreamCast", "PlainMLP", "StateSpaceDuality", "MatrixMemory",
-           "PostNormBlock", "PostNormMixerBlock", "GeneralizedDeltaRule", "ScaledPreNormBlock", "ScaledPreNormMixerBlock"]
+           "PostNormBlock", "PostNormMixerBlock", "GeneralizedDeltaRule", "HeadDecayDeltaRule", "TimeMix", "ScaledPreNormBlock", "ScaledPreNormMixerBlock"]

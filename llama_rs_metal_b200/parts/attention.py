@@ -43,8 +43,16 @@ class Attention(Mixer):
     sequence are kept as state beside its keys and values); `row_norm_eps`, an RMS norm with weights
     over the whole query row and the whole key row before the rotation (`q_norm.weight`,
     `k_norm.weight`); `head_norm_eps`, each query and key head divided by its root mean square after
-    the rotation, no weight. `chunk`: positions form chunks of this many counted from position 0 and a
+    the rotation, no weight; `head_weight_eps`, an RMS norm over each query and key head ahead of the
+    rotation with one weight of the head size for all query heads and one for all key heads
+    (`q_head_norm.weight`, `k_head_norm.weight`). `chunk`: positions form chunks of this many counted from position 0 and a
     query sees the keys of its own chunk only; the cache then keeps a window of `chunk` keys.
+
+    `weights` "sigmoid": no softmax. A visible key's weight is sigmoid(score + `score_offset`[head]) (a stored
+    tensor, one number per query head), not normalized over the keys (csrc/attention_sigmoid.cu; the layer takes
+    the shaped split). `gate` (with sigmoid weights): the heads are multiplied element by element by
+    sigmoid(W_g x) ahead of the output projection (tensor `g_proj.weight`); it rides in the fused projection
+    and the attention kernels apply it where they write.
     """
 
     def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int,
@@ -53,7 +61,10 @@ class Attention(Mixer):
                  output_scale: float = 1.0, values_are_keys: bool = False, sinks: bool = False,
                  query_temperature: Optional[Sequence[float]] = None, conv_taps: int = 0,
                  row_norm_eps: Optional[float] = None, head_norm_eps: Optional[float] = None,
-                 chunk: Optional[int] = None):
+                 chunk: Optional[int] = None, weights: str = "softmax", gate: bool = False,
+                 head_weight_eps: Optional[float] = None):
+        if weights not in ("softmax", "sigmoid"):
+            raise UnsupportedError(f"attention weights {weights!r}")
         if num_heads <= 0 or num_kv_heads <= 0 or num_heads % num_kv_heads:
             raise InvalidError("attention heads must be a multiple of key/value heads")
         self.values_are_keys, self.has_sinks = bool(values_are_keys), bool(sinks)
@@ -72,7 +83,13 @@ class Attention(Mixer):
         self.chunk = int(chunk) if chunk else None
         if self.conv_taps < 0 or (self.chunk is not None and (self.chunk <= 0 or window is not None)):
             raise InvalidError("attention: taps cannot be negative, and a chunked layer has no window besides")
-        self.shaped = bool(self.conv_taps) or self.row_norm_eps is not None or self.head_norm_eps is not None
+        self.sigmoid, self.gate = weights == "sigmoid", bool(gate)
+        self.head_weight_eps = None if head_weight_eps is None else float(head_weight_eps)
+        self.shaped = bool(self.conv_taps) or any(e is not None for e in (self.row_norm_eps, self.head_norm_eps,
+                                                                          self.head_weight_eps)) or self.sigmoid
+        if self.gate and not self.sigmoid:
+            raise InvalidError("an output gate is built together with sigmoid weights only")
+        self.head_weights = self.score_offset = None
         if self.shaped and (values_are_keys or sinks or query_temperature is not None):
             raise InvalidError("shaped queries and keys are not built together with sinks, a query temperature or keys as values")
         self.taps = self.row_norm = None
@@ -110,6 +127,12 @@ class Attention(Mixer):
                         "v_conv.weight": TensorSpec((v, self.conv_taps))})
         if self.row_norm_eps is not None:
             out.update({"q_norm.weight": TensorSpec((q,)), "k_norm.weight": TensorSpec((kv,))})
+        if self.head_weight_eps is not None:
+            out.update({"q_head_norm.weight": TensorSpec((self.head_dim,)), "k_head_norm.weight": TensorSpec((self.head_dim,))})
+        if self.sigmoid:
+            out["score_offset"] = TensorSpec((self.num_heads,))
+        if self.gate:
+            out["g_proj.weight"] = TensorSpec((mixed, h))
         if self.position is not None:
             out.update({"position." + n: s for n, s in self.position.tensors().items()})
         return out
@@ -127,6 +150,8 @@ class Attention(Mixer):
             q_weight = q_weight.view(self.num_heads, self.head_dim, -1)[:, index].reshape(q_weight.shape)
             k_weight = k_weight.view(self.num_kv_heads, self.head_dim, -1)[:, index].reshape(k_weight.shape)
         rows = [q_weight, k_weight] if self.values_are_keys else [q_weight, k_weight, weights["v_proj.weight"]]
+        if self.gate:  # behind q | k | v
+            rows.append(weights["g_proj.weight"])
         fused = torch.cat(rows, dim=0).contiguous()
         if self.has_sinks or self.query_temperature is not None:
             from ..kernels.attention_dispatch import Extras
@@ -149,6 +174,10 @@ class Attention(Mixer):
         if self.row_norm_eps is not None:
             self.row_norm = (weights["q_norm.weight"].to(torch.float32).contiguous(),
                              weights["k_norm.weight"].to(torch.float32).contiguous())
+        if self.head_weight_eps is not None:
+            self.head_weights = tuple(weights[n + "_head_norm.weight"].to(torch.float32).contiguous() for n in "qk")
+        if self.sigmoid:
+            self.score_offset = weights["score_offset"].to(torch.float32).contiguous()
         if self.shaped and self.position is not None and self.position.rotary_table() is None:
             raise InvalidError("a shaped attention layer rotates by a rotary table or not at all")
 
@@ -165,7 +194,11 @@ class Attention(Mixer):
             return CompositeRequest((keys, StateRequest((self.conv_taps - 1, self.projected_width), torch.float32)))
         return keys
 
-    def _shaped_forward(self, x, ctx, cache, residual):
+    @property
+    def mixed_width(self) -> Optional[int]:
+        return self.num_heads * self.value_dim if self.sigmoid else None
+
+    def mix(self, x, ctx, cache, out=None, column=0):
         """Projection in float32, then bias, convolution, norms and rotation in one kernel that also
         splits and stores, then attention under the window or the chunk."""
         from ..kernels.attention_dispatch import Shaping
@@ -178,17 +211,24 @@ class Attention(Mixer):
             rotary, adjacent = self.position.rotary_dim, self.position.adjacent_pairs
             inv_freq = self.position.inv_freq64
         shaping = Shaping(taps=self.taps, tails=tails, row_norm=self.row_norm, row_eps=self.row_norm_eps or 0.0,
+                          head_weights=self.head_weights, head_weight_eps=self.head_weight_eps or 0.0,
                           inv_freq=inv_freq, rotary=rotary, adjacent_pairs=adjacent, head_norm_eps=self.head_norm_eps)
-        mixed = ops.attend(self.qkv(x, out_dtype=torch.float32), q_heads=self.num_heads, kv_heads=self.num_kv_heads,
-                           head_dim=self.head_dim, rotary=None, ctx=ctx, cache=keys, writes_cache=True,
-                           cache_entry=entry.cache, scale=self.scale, window=self.chunk or self.window,
-                           value_dim=self.value_dim, bias=self.bias, out_scale=self.output_scale, shaping=shaping,
-                           chunk=self.chunk)
-        return self.out(mixed, epilogue=ops.ADD, out=residual, ctx=ctx)
+        projected = self.qkv(x, out_dtype=torch.float32)
+        sigmoid = None
+        if self.sigmoid:
+            sigmoid = ops.SigmoidWeights(self.score_offset, (projected, self.projected_width) if self.gate else None,
+                                         (out, column) if out is not None else None)
+        elif out is not None:
+            raise UnsupportedError("softmax attention writes a tensor of its own")
+        return ops.attend(projected, q_heads=self.num_heads, kv_heads=self.num_kv_heads,
+                          head_dim=self.head_dim, rotary=None, ctx=ctx, cache=keys, writes_cache=True,
+                          cache_entry=entry.cache, scale=self.scale, window=self.chunk or self.window,
+                          value_dim=self.value_dim, bias=self.bias, out_scale=self.output_scale, shaping=shaping,
+                          chunk=self.chunk, sigmoid_weights=sigmoid)
 
     def forward(self, x, ctx, cache, residual):
         if self.shaped:
-            return self._shaped_forward(x, ctx, cache, residual)
+            return self.out(self.mix(x, ctx, cache), epilogue=ops.ADD, out=residual, ctx=ctx)
         entry = ctx.entry
         weight = self.qkv if entry.writes_cache else self.q_only
         rotary = self.position.rotary_table() if self.position is not None else None

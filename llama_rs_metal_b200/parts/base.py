@@ -94,6 +94,9 @@ class ScheduleEntry:
     # the embedding's output (the stream as it was before the first entry) is added to the stream
     # right before this entry runs, ahead of `add_offset`
     add_embedding: bool = False
+    # right before this entry runs the stream x is replaced by W [x; x0], x0 being the embedding's
+    # output and W the plan's `stream_join` matrix
+    join_embedding: bool = False
 
 
 @dataclass(frozen=True)
@@ -113,6 +116,10 @@ class ModelPlan:
     # (checkpoint name, rows) of a [rows, hidden] table of vectors that schedule entries add to
     # the residual stream (ScheduleEntry.add_offset), or None
     stream_offsets: Optional[Tuple[str, int]] = None
+    # checkpoint name of the [hidden, 2 hidden] matrix of ScheduleEntry.join_embedding (columns of the
+    # stream first), or None
+    stream_join: Optional[str] = None
+    logit_softcap: Optional[float] = None    # logits become cap * tanh(logits / cap) (None: as they are)
 
 
 # --------------------------------------------------------------------------- cache requests
@@ -179,6 +186,13 @@ class Norm(Part):
         """float32 residual [T,h] -> normalized activations [T,h] (or [len(rows),h])."""
         raise NotImplementedError
 
+    def forward_conv(self, hidden: torch.Tensor, ctx, taps: torch.Tensor, tails: Optional[torch.Tensor]) -> torch.Tensor:
+        """h + conv(h) for h = forward(hidden): a causal convolution over time per channel behind the norm
+        (taps float32 [n, width], the last row the current token's), whose inputs before the step come
+        from `tails` (float32 [slots, n - 1, width], moved on; None for a single tap)."""
+        from ..kernels import ops
+        return ops.input_conv(self.forward(hidden, ctx), taps, tails, ctx.cu_seqlens, ctx.seq_of_token, ctx.slots)
+
     def add_into(self, hidden: torch.Tensor, y: torch.Tensor, ctx, mult: float = 1.0,
                  then: Optional["Norm"] = None) -> Optional[torch.Tensor]:
         """hidden += mult * norm(y) for a sublayer's float32 output y [T,h] (a norm behind the
@@ -213,6 +227,15 @@ class PositionEncoding(Part):
 
 
 class Mixer(Part):
+    # A mixer whose output is one product `out` (a LinearWeight) over a row of mixed heads of this many
+    # columns, and that can make that row without the product (mix()); None for other mixers.
+    mixed_width: Optional[int] = None
+
+    def mix(self, x: torch.Tensor, ctx, cache, out: Optional[torch.Tensor] = None, column: int = 0) -> torch.Tensor:
+        """The mixed heads ahead of the output product, [T, mixed_width] in the activation type: a new
+        tensor, or columns column .. of `out`, which is returned."""
+        raise NotImplementedError
+
     def cache_request(self):
         """KeyValueRequest, StateRequest, CompositeRequest or None."""
         return None

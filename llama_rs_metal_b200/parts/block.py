@@ -15,20 +15,60 @@ from .norm import StreamCast
 STREAM_ITSELF = StreamCast()  # what a block whose sublayers read the stream itself has for an entry norm
 
 
-@register_block("pre_norm")
-class PreNormBlock(Block):
-    """hidden += mixer(norm(hidden)); hidden += feed_forward(norm(hidden))
-    (crates/model-runtime/src/execute.rs:24,196-199,236)."""
+class _PreNormBlock(Block):
+    """Pre-norm sublayers. With `input_taps` n > 0 a mixer reads h + conv(h) instead of its norm's output
+    h: a causal convolution over time per channel (tensor `input_conv`, [hidden_size, n], the last
+    column the current token's, no bias); the last n - 1 rows h of every sequence are state of the
+    layer, kept beside the mixer's own."""
 
     graph_safe = True
+
+    def __init__(self, hidden_size: int = 0, input_taps: int = 0, **parts):
+        super().__init__(**parts)
+        self.hidden_size, self.input_taps = int(hidden_size), int(input_taps)
+        if self.input_taps < 0 or (self.input_taps and self.hidden_size <= 0):
+            raise InvalidError("an input convolution has positive taps and the layer's width")
+        self.taps: Optional[torch.Tensor] = None
 
     @property
     def folds_pending_on_entry(self) -> bool:
         return self.mixer_norm.folds_pending
 
+    def tensors(self) -> Dict[str, TensorSpec]:
+        return {"input_conv": TensorSpec((self.hidden_size, self.input_taps))} if self.input_taps else {}
+
+    def bind(self, weights, runtime) -> None:
+        if self.input_taps:
+            # [taps, width]: the kernels read one tap of many channels at a time
+            self.taps = weights["input_conv"].to(torch.float32).t().contiguous()
+
+    def cache_request(self):
+        request = self.mixer.cache_request()
+        if self.input_taps <= 1:
+            return request
+        return CompositeRequest((request, StateRequest((self.input_taps - 1, self.hidden_size), torch.float32)))
+
+    def _mixer_input(self, hidden, ctx, cache):
+        """(what the mixer reads, the mixer's part of the layer's cache)."""
+        if not self.input_taps:
+            return self.mixer_norm.forward(hidden, ctx), cache
+        tails = None
+        if self.input_taps > 1:
+            if cache is None or not ctx.entry.writes_cache:
+                raise InvalidError("a layer with an input convolution keeps state of its own")
+            cache, last = cache
+            tails = last.state
+        return self.mixer_norm.forward_conv(hidden, ctx, self.taps, tails), cache
+
+
+@register_block("pre_norm")
+class PreNormBlock(_PreNormBlock):
+    """hidden += mixer(norm(hidden)); hidden += feed_forward(norm(hidden))
+    (crates/model-runtime/src/execute.rs:24,196-199,236)."""
+
     def forward(self, hidden, ctx, cache):
         after = ctx.next_folds_pending  # what comes after this block (the model says)
-        x = self.mixer_norm.forward(hidden, ctx)
+        x, cache = self._mixer_input(hidden, ctx, cache)
         # the mixer's output goes straight into the second norm: if that norm adds pending
         # partial sums itself, the mixer's last product may leave its K slices unadded
         ctx.may_defer = self.feed_forward_norm.folds_pending
@@ -42,19 +82,14 @@ class PreNormBlock(Block):
 
 
 @register_block("pre_norm_mixer")
-class PreNormMixerBlock(Block):
+class PreNormMixerBlock(_PreNormBlock):
     """hidden += mixer(norm(hidden)): a layer without a feed-forward."""
 
-    graph_safe = True
     roles = {"mixer": "mixer", "mixer_norm": "norm"}
-
-    @property
-    def folds_pending_on_entry(self) -> bool:
-        return self.mixer_norm.folds_pending
 
     def forward(self, hidden, ctx, cache):
         after = ctx.next_folds_pending
-        x = self.mixer_norm.forward(hidden, ctx)
+        x, cache = self._mixer_input(hidden, ctx, cache)
         ctx.may_defer = after
         hidden = self.mixer.forward(x, ctx, cache, residual=hidden)
         ctx.may_defer = False

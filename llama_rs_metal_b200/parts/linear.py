@@ -23,17 +23,20 @@ class LinearWeight:
     def out_features(self) -> int:
         return self.weight.shape[0]
 
-    def pick(self, x: torch.Tensor, temperature=None, seed: int = 0, keys=None):
+    def pick(self, x: torch.Tensor, temperature=None, seed: int = 0, keys=None, softcap: Optional[float] = None):
         """The token chosen from each row's logits x . W^T (greedy, or temperature sampling with
         per-row keys), int32 [M], -1 for a row with a non-finite logit. The logits are not
-        written where a kernel chooses in the product's epilogue."""
-        if x.dtype == self.weight.dtype:
+        written where a kernel chooses in the product's epilogue. `softcap`: draws come from
+        cap * tanh(logits / cap), which rises with the logit, so the greedy choice needs no cap."""
+        if x.dtype == self.weight.dtype and (softcap is None or temperature is None):
             ids = ops.linear_pick(x, self.weight, temperature, seed, keys)
             if ids is not None:
                 return ids
         logits = self(x, out_dtype=torch.float32)
         if temperature is None:
             return ops.argmax_rows(logits)
+        if softcap is not None:
+            ops.softcap_(logits, softcap)
         return ops.sample_gumbel_rows(logits, temperature, seed, keys)
 
     def supports_fused_gate(self, x_dtype: torch.dtype) -> bool:
@@ -66,3 +69,26 @@ class LinearWeight:
         # bfloat16 matrix under float32 activations does not occur: the float32
         # runtime widens every weight when it loads.
         return ops.linear(x, ops.cast(w, x.dtype), epilogue, out, out_dtype)
+
+
+class GroupedLinear:
+    """Several matrices [out_i, in], one input each, as one stacked weight whose products are one launch
+    (ops.linear_grouped): every matrix but the last is filled up with rows of zeros to `group_cols`
+    rows, a whole number of tiles. Column c of matrix i is column i * group_cols + c of the result."""
+
+    def __init__(self, matrices):
+        multiple = ops.GROUP_MULTIPLE
+        self.group_cols = max(-(-m.shape[0] // multiple) * multiple for m in matrices)
+        rows = []
+        for m in matrices[:-1]:
+            pad = self.group_cols - m.shape[0]
+            rows += [m] + ([torch.zeros((pad, m.shape[1]), dtype=m.dtype, device=m.device)] if pad else [])
+        self.weight = torch.cat(rows + [matrices[-1]], dim=0).contiguous()
+
+    def column(self, i: int) -> int:
+        return i * self.group_cols
+
+    def __call__(self, inputs: torch.Tensor) -> torch.Tensor:
+        """inputs [matrices, T, in] -> float32 [T, columns]."""
+        # precision follows storage, as for LinearWeight
+        return ops.linear_grouped(ops.cast(inputs, self.weight.dtype), self.weight, self.group_cols)

@@ -1,4 +1,4 @@
-"""Norms: RMSNorm, layer norm with weight and bias, and the plain rounding of the stream."""
+"""Norms: RMSNorm, layer norm with weight and (optional) bias, and the plain rounding of the stream."""
 from __future__ import annotations
 
 from typing import Dict, Optional
@@ -75,24 +75,39 @@ class StreamCast(Norm):
 @register_norm("layer_norm")
 class LayerNorm(Norm):
     """y = (x - mean) / sqrt(variance + eps) * w + b over a row, with the variance the mean of the
-    squared deviations; statistics, weight and bias in float32. The bias is the tensor `bias`."""
+    squared deviations; statistics, weight and bias in float32. The bias is the tensor `bias`; with
+    `bias` False there is none."""
 
     graph_safe = True
+    folds_pending = True
 
-    def __init__(self, size: int, eps: float):
-        self.size, self.eps = size, float(eps)
+    def __init__(self, size: int, eps: float, bias: bool = True):
+        self.size, self.eps, self.has_bias = size, float(eps), bool(bias)
         self.weight: Optional[torch.Tensor] = None
         self.bias: Optional[torch.Tensor] = None
 
     def tensors(self) -> Dict[str, TensorSpec]:
-        return {"weight": TensorSpec((self.size,)), "bias": TensorSpec((self.size,))}
+        out = {"weight": TensorSpec((self.size,))}
+        if self.has_bias:
+            out["bias"] = TensorSpec((self.size,))
+        return out
 
     def bind(self, weights, runtime) -> None:
         self.weight = weights["weight"].to(torch.float32).contiguous()
-        self.bias = weights["bias"].to(torch.float32).contiguous()
+        if self.has_bias:
+            self.bias = weights["bias"].to(torch.float32).contiguous()
 
     def forward(self, hidden, ctx, rows=None):
-        return ops.layer_norm(hidden, self.weight, self.bias, self.eps, ctx.runtime.dtype, rows=rows)
+        # partial sums a product left for the residual stream are added in the same pass
+        return ops.layer_norm(hidden, self.weight, self.bias, self.eps, ctx.runtime.dtype, rows=rows,
+                              partials=ctx.take_pending())
+
+    def forward_conv(self, hidden, ctx, taps, tails):
+        if ctx.phase != "decode" or tails is None:
+            return super().forward_conv(hidden, ctx, taps, tails)
+        # one token per sequence: the norm and the convolution behind it are one pass over the rows
+        return ops.layer_norm_conv(hidden, self.weight, self.bias, self.eps, ctx.runtime.dtype, taps, tails, ctx.slots,
+                                   partials=ctx.take_pending())
 
     def add_into(self, hidden, y, ctx, mult=1.0, then=None):
         # the pass that adds the normed output also writes the updated row in the activation type

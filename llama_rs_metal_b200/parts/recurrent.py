@@ -12,6 +12,13 @@ update it token by token and read it out with the query (csrc/recurrent_scan.cu)
   a per key channel, both computed from the input, u the unit key, both terms reading the old S
   (csrc/general_delta.cu prepares its inputs).
 
+* `head_decay_delta_rule`: the delta rule with one decay per head computed from the input, S <- g S;
+  S <- S + k (b (v - S^T k))^T; q, k, v pass a short causal convolution first
+  (csrc/head_decay_delta.cu prepares its inputs).
+* `time_mix`: S <- diag(w) S + k v^T with decays w per key channel computed from the input, read before the
+  write with a bonus for the current token; every projection reads its own mix of a token's row with
+  the row before (csrc/time_mix.cu).
+
 A third keeps one number per channel (csrc/gated_recurrence.cu):
 
 * `gated_linear_recurrence`: S <- a S + sqrt(1 - a^2) (i u) with a decay a and an input gate i
@@ -40,7 +47,7 @@ from ..kernels import ops
 from ..registry import POSITION_ENCODINGS, build_part, register_mixer
 from ..weights.loader import TensorSpec
 from .base import CompositeRequest, Mixer, PartSpec, StateRequest
-from .linear import LinearWeight
+from .linear import GroupedLinear, LinearWeight
 
 
 def _needs_own_state(ctx) -> None:
@@ -256,6 +263,146 @@ class GeneralizedDeltaRule(Mixer):
         mixed = ops.head_norm_gate(o, self.eps, x.dtype, weight=self.norm_weight, gate=projected, gate_column=at_g,
                                    gate_act=ops.GATE_SIGMOID)
         return self.out(mixed, epilogue=ops.ADD, out=residual, ctx=ctx)
+
+
+@register_mixer("head_decay_delta_rule")
+class HeadDecayDeltaRule(Mixer):
+    """q = W_q x, k = W_k x (kv_heads x head_dim), v = W_v x (heads x value_dim); each passes a causal
+    convolution of `conv_taps` taps per channel (no bias, zeros before the start) and SiLU; q and k become
+    unit vectors per head (x / sqrt(sum x^2 + unit_eps)), q times head_dim^-1/2. b = sigmoid(W_b x) and
+    g = exp(-exp(A_log_h) softplus(W_a x + dt_bias_h)), one number per head each. Per head, with q/k head
+    h // (heads / kv_heads):
+        S <- g S;  u = b (v - S^T k);  S <- S + k u^T;  o = S^T q.
+    o is divided by its root mean square over value_dim (`eps`), multiplied by a weight shared by the heads
+    and by silu(W_g x), then projected. The projections keep their float32 sums.
+    State: S in float32 and the last conv_taps - 1 convolution inputs of every channel."""
+
+    graph_safe = True
+
+    def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int, value_dim: int,
+                 conv_taps: int, eps: float, unit_eps: float = 1e-6, output_scale: float = 1.0):
+        if min(num_heads, num_kv_heads, head_dim, value_dim, conv_taps) <= 0 or num_heads % num_kv_heads:
+            raise InvalidError("head-decay delta rule: heads must be a multiple of key heads, and sizes positive")
+        self.hidden_size, self.num_heads, self.num_kv_heads = hidden_size, num_heads, num_kv_heads
+        self.head_dim, self.value_dim, self.conv_taps = head_dim, value_dim, conv_taps
+        self.eps, self.unit_eps, self.output_scale = float(eps), float(unit_eps), float(output_scale)
+        self.channels = 2 * num_kv_heads * head_dim + num_heads * value_dim
+        self.mixed_width = num_heads * value_dim
+        self.fused: Optional[LinearWeight] = None
+        self.out: Optional[LinearWeight] = None
+
+    def tensors(self) -> Dict[str, TensorSpec]:
+        H, G, d, dv, h, n = (self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim, self.hidden_size,
+                             self.conv_taps)
+        return {"q_proj.weight": TensorSpec((G * d, h)), "k_proj.weight": TensorSpec((G * d, h)),
+                "v_proj.weight": TensorSpec((H * dv, h)), "q_conv.weight": TensorSpec((G * d, n)),
+                "k_conv.weight": TensorSpec((G * d, n)), "v_conv.weight": TensorSpec((H * dv, n)),
+                "b_proj.weight": TensorSpec((H, h)), "a_proj.weight": TensorSpec((H, h)), "A_log": TensorSpec((H,)),
+                "dt_bias": TensorSpec((H,)), "g_proj.weight": TensorSpec((H * dv, h)),
+                "norm.weight": TensorSpec((dv,)), "o_proj.weight": TensorSpec((h, H * dv))}
+
+    def bind(self, weights, runtime) -> None:
+        f32 = torch.float32
+        # q | k | v | g | b | a in one product
+        self.fused = LinearWeight(torch.cat([weights[n + "_proj.weight"] for n in "qkvgba"], dim=0))
+        self.out = LinearWeight(weights["o_proj.weight"])
+        # [taps, channels]: the kernel reads one tap of many channels at a time
+        self.taps = torch.cat([weights[n + "_conv.weight"] for n in "qkv"], dim=0).to(f32).t().contiguous()
+        self.rate = torch.exp(weights["A_log"].to(f32)).contiguous()      # exp(A_log), float32
+        self.dt_bias = weights["dt_bias"].to(f32).contiguous()
+        self.norm_weight = weights["norm.weight"].to(f32).contiguous()
+
+    def cache_request(self):
+        state = StateRequest((self.num_heads, self.head_dim, self.value_dim), torch.float32)
+        if self.conv_taps == 1:
+            return state
+        return CompositeRequest((state, StateRequest((self.conv_taps - 1, self.channels), torch.float32)))
+
+    def mix(self, x, ctx, cache, out=None, column=0):
+        _needs_own_state(ctx)
+        H, G, d, dv = self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim
+        state, tails = cache if self.conv_taps > 1 else (cache, None)
+        projected = self.fused(x, out_dtype=torch.float32)               # [T, q | k | v | g | b | a], float32
+        at_g = self.channels
+        at_b = at_g + H * dv
+        q, k, v, decay, step = ops.head_decay_delta_prepare(
+            projected, 0, at_b, at_b + H, self.dt_bias, self.rate, self.taps, tails.state if tails is not None else None,
+            ctx.cu_seqlens, ctx.seq_of_token, ctx.slots, H, G, d, dv, self.unit_eps, d ** -0.5,
+            one_each=ctx.phase == "decode")
+        o = ops.head_decay_delta_scan(q, k, v, decay, step, state.state, ctx.cu_seqlens, ctx.slots)
+        return ops.head_norm_gate(o, self.eps, x.dtype, weight=self.norm_weight, gate=projected, gate_column=at_g,
+                                  gate_act=ops.GATE_SILU, out_scale=self.output_scale, out=out, out_column=column)
+
+    def forward(self, x, ctx, cache, residual):
+        return self.out(self.mix(x, ctx, cache), epilogue=ops.ADD, out=residual, ctx=ctx)
+
+
+@register_mixer("time_mix")
+class TimeMix(Mixer):
+    """A matrix state per head with a decay per key channel computed from the input. With x' the previous
+    token's x (zeros for a sequence's first token), each of r, k, v, g and w reads its own mix
+    x + (x' - x) * mu_s: r, k, v = W x_s (heads x head_dim), gate = silu(W_g x_g), and the decay
+    w = exp(-exp(W_w2 tanh(W_w1 x_w) + w_bias)) per head and key channel. Per head
+        o_t = (S_(t-1) + diag(u) k_t v_t^T)^T r_t,    S_t = diag(w_t) S_(t-1) + k_t v_t^T.
+    Each head's o is divided by its root mean square (`eps`), multiplied by a weight over all heads' columns
+    and by the gate, then projected. The inner rank of the decay's product is the checkpoint's (`decay_rank`
+    None) unless given. The five products are one launch over the five mixes; they keep their float32
+    sums (the tanh is rounded to the activation type where it enters the second product).
+    State: S in float32 and the last x."""
+
+    graph_safe = True
+    STREAMS = "rkvgw"
+
+    def __init__(self, hidden_size: int, num_heads: int, head_dim: int, eps: float, decay_rank: Optional[int] = None,
+                 output_scale: float = 1.0):
+        if min(num_heads, head_dim) <= 0:
+            raise InvalidError("time mix: sizes must be positive")
+        self.hidden_size, self.num_heads, self.head_dim = hidden_size, num_heads, head_dim
+        self.eps, self.decay_rank, self.output_scale = float(eps), decay_rank, float(output_scale)
+        self.mixed_width = num_heads * head_dim
+        self.fused: Optional[GroupedLinear] = None
+        self.out: Optional[LinearWeight] = None
+
+    def tensors(self) -> Dict[str, TensorSpec]:
+        n, h = self.num_heads * self.head_dim, self.hidden_size
+        out = {f"{s}_mix": TensorSpec((h,)) for s in self.STREAMS}
+        out.update({f"{s}_proj.weight": TensorSpec((n, h)) for s in "rkvg"})
+        out.update({"w_down.weight": TensorSpec((self.decay_rank, h)), "w_up.weight": TensorSpec((n, self.decay_rank)),
+                    "w_bias": TensorSpec((n,)), "bonus": TensorSpec((self.num_heads, self.head_dim)),
+                    "norm.weight": TensorSpec((n,)), "o_proj.weight": TensorSpec((h, n))})
+        return out
+
+    def bind(self, weights, runtime) -> None:
+        f32 = torch.float32
+        down, up = weights["w_down.weight"], weights["w_up.weight"]
+        if up.shape[1] != down.shape[0]:
+            raise InvalidError("time mix: the two halves of the decay's product disagree on its rank")
+        self.fused = GroupedLinear([weights[f"{s}_proj.weight"] for s in "rkvg"] + [down])
+        self.up = up.contiguous()
+        self.out = LinearWeight(weights["o_proj.weight"])
+        self.shifts = torch.stack([weights[f"{s}_mix"] for s in self.STREAMS]).to(f32).contiguous()
+        self.w_bias = weights["w_bias"].to(f32).contiguous()
+        self.bonus = weights["bonus"].to(f32).contiguous()
+        self.norm_weight = weights["norm.weight"].to(f32).contiguous()
+
+    def cache_request(self):
+        return CompositeRequest((StateRequest((self.num_heads, self.head_dim, self.head_dim), torch.float32),
+                                 StateRequest((1, self.hidden_size), torch.float32)))
+
+    def mix(self, x, ctx, cache, out=None, column=0):
+        _needs_own_state(ctx)
+        state, last = cache
+        at = self.fused.column
+        mixes = ops.token_mixes(x, self.shifts, last.state, ctx.cu_seqlens, ctx.seq_of_token, ctx.slots)
+        projected = self.fused(mixes)                                    # [T, r | k | v | g | low], float32
+        w = ops.decay_product(projected, at(4), self.up, self.w_bias)    # [T, heads * head_dim], float32
+        o = ops.bonus_state_scan(projected, at(0), at(1), at(2), w, self.bonus, state.state, ctx.cu_seqlens, ctx.slots,
+                                 self.head_dim)
+        return ops.head_norm_gate(o, self.eps, x.dtype, weight=self.norm_weight, gate=projected, gate_column=at(3),
+                                  gate_act=ops.GATE_SILU, out_scale=self.output_scale, out=out, out_column=column)
+
+    def forward(self, x, ctx, cache, residual):
+        return self.out(self.mix(x, ctx, cache), epilogue=ops.ADD, out=residual, ctx=ctx)
 
 
 @register_mixer("gated_linear_recurrence")
