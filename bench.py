@@ -293,13 +293,30 @@ def tarupel_shape(width, heads, kv_heads, ff, experts, top, window, layers, voca
                 residual_mult=0.5, layers=[dict(kinds[i % 3]) for i in range(layers)], loop=dict(start=0, stop=2, times=2))
 
 
+def tolurax_shape(width, heads, kv_heads, ff, window, layers, vocab=32768):
+    """A Tolurax configuration with layers of a real model's widths: one delta-rule layer (head size 128, 4
+    taps), then parallel layers (sigmoid-weight attention through a window, head size 128; a time mix with
+    heads of 64 and a decay rank of 64), a dense feed-forward behind each, an input convolution of 4 taps.
+    The first two layers loop twice."""
+    d = 128
+    mlp = dict(kind="dense", ff=ff)
+    delta = dict(type="delta", mlp=mlp, mixer=dict(heads=heads, kv_heads=kv_heads, dim=d, vdim=d, conv=4))
+    left = dict(heads=heads, kv_heads=kv_heads, dim=d, vdim=d, scale=d ** -0.5, mask=dict(size=window),
+                rot=dict(dims=d, base=500000.0, scaling=dict(factor=8.0, low=1.0, high=4.0, original=8192)))
+    parallel = dict(type="parallel", mlp=mlp, mixer=dict(
+        left=left, right=dict(heads=width // 64, dim=64, decay_rank=64), left_scale=0.5, right_scale=0.5))
+    return dict(architecture="Tolurax", vocab=vocab, width=width, norm=dict(eps=1e-5), canon=dict(taps=4), logit_softcap=30.0,
+                layers=[delta] + [parallel] * (layers - 1), loop=dict(start=0, stop=2, times=2))
+
+
 def design_bench(args) -> int:
-    """Prefill and decode throughput of the Kikalix, the Pibuvik, the Norevik or the Tarupel design at a few
+    """Prefill and decode throughput of the Kikalix, Pibuvik, Norevik, Tarupel or Tolurax design at a few
     layer sizes, beside an existing decoder at equal size: Kikalix and Pibuvik beside Llama (the same
     width, head geometry, vocabulary and number of layer runs; its feed-forward as wide as the
-    experts a token uses, or as the dense one), Norevik and Tarupel beside Kikalix, the closest of the
-    designs (state mixers on the same scan, the same experts, a looped run: equal width, heads, experts,
-    chosen experts, expert width, vocabulary and layer runs). Random weights, one GPU, bfloat16."""
+    experts a token uses, or as the dense one), Norevik, Tarupel and Tolurax beside Kikalix, the closest of
+    the designs (state mixers on the same scan, a looped run, windowed attention: equal width, heads, experts,
+    chosen experts, expert width, vocabulary and layer runs; Tolurax's dense feed-forward is as wide as the
+    experts a token uses). Random weights, one GPU, bfloat16."""
     if args.profile:
         os.environ["LRM_PROFILE"] = "1"
     import numpy as np
@@ -319,6 +336,16 @@ def design_bench(args) -> int:
         session = model.session(context=prompt + steps + 64, max_batch=batch)
         ids = rng.integers(0, vocab, size=prompt).tolist()
         times = []
+        if args.profile:  # every kernel once: what a first launch costs (loading the kernel) is not its time
+            from llama_rs_metal_b200.kernels import profile
+            slots = [session.open_slot() for _ in range(batch)]
+            for slot in slots:
+                session.runner.step([StepEntry(slot, ids, (prompt - 1,))])
+            session.runner.step_pick([StepEntry(slot, [1], (0,)) for slot in slots], DevicePick(None, 0, [0] * batch))
+            for slot in slots:
+                session.close_slot(slot)
+            torch.cuda.synchronize()
+            profile.reset()
         for rep in range(2 + 5):                      # prefill of one prompt: median of five after two
             slot = session.open_slot()
             begin, end = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
@@ -378,6 +405,13 @@ def design_bench(args) -> int:
             twin, twin_name = kikalix_shape(width, heads, kv_heads, ff, experts, top, window, layers), "kikalix_equal_size"
             shape = dict(width=width, heads=heads, kv_heads=kv_heads, head_dim=128, expert_ff=ff, shared_ff=ff,
                          experts=experts, top=top, state_heads=width // 64, window=window, layer_runs=runs)
+        elif args.design == "tolurax":
+            width, heads, kv_heads, ff, experts, top, window, layers = DESIGN_SIZES[size]
+            runs, norm_mean = layers + 2, 1.0
+            config = tolurax_shape(width, heads, kv_heads, top * ff, window, layers)
+            twin, twin_name = kikalix_shape(width, heads, kv_heads, ff, experts, top, window, layers), "kikalix_equal_size"
+            shape = dict(width=width, heads=heads, kv_heads=kv_heads, head_dim=128, ff=top * ff, twin_expert_ff=ff,
+                         twin_experts=experts, twin_top=top, time_mix_heads=width // 64, window=window, layer_runs=runs)
         elif args.design == "pibuvik":
             width, heads, kv_heads, ff, kv_rank, window, layers = PIBUVIK_SIZES[size]
             config = pibuvik_shape(width, heads, kv_heads, ff, kv_rank, window, layers)
@@ -394,7 +428,7 @@ def design_bench(args) -> int:
         row = {args.design: measure(model, config["vocab"], f"{design_name} {size}")}
         del model
         torch.cuda.empty_cache()
-        if args.design in ("norevik", "tarupel"):
+        if args.design in ("norevik", "tarupel", "tolurax"):
             model = engine.random(twin, seed=0, std=0.02, norm_mean=0.0)
         else:
             twin = llama(width, twin_ff, runs, heads, kv_heads, 128, 8.0, False)
@@ -406,7 +440,7 @@ def design_bench(args) -> int:
         row["shape"] = shape
         out[size] = row
     print(json.dumps({"metric": f"prefill tok/s (one {prompt}-token prompt) and decode tok/s (batch {batch} at "
-                                f"{prompt} tokens), {design_name} beside {'Kikalix' if args.design in ('norevik', 'tarupel') else 'Llama'} at equal size",
+                                f"{prompt} tokens), {design_name} beside {'Kikalix' if args.design in ('norevik', 'tarupel', 'tolurax') else 'Llama'} at equal size",
                       "dtype": "bf16", "data": "synthetic token ids, random-init weights", "n_gpus": 1,
                       "decode_steps": steps, "peaks": peak_source, "cuda_graph": not args.profile, "sizes": out}))
     return 0
@@ -439,7 +473,7 @@ def main() -> int:
     parser.add_argument("--profile", action="store_true",
                         help="time every kernel launch (LRM_PROFILE=1) and print the table to stderr; the "
                              "line's numbers are then those of unfused, uncaptured launches")
-    parser.add_argument("--design", choices=["kikalix", "pibuvik", "norevik", "tarupel"], default=None,
+    parser.add_argument("--design", choices=["kikalix", "pibuvik", "norevik", "tarupel", "tolurax"], default=None,
                         help="instead of the default workload: prefill and decode throughput of this design at "
                              "a few layer sizes beside an existing decoder at equal size (see design_bench)")
     parser.add_argument("--design-size", choices=sorted(DESIGN_SIZES), default=None,

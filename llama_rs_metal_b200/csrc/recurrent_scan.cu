@@ -1,302 +1,14 @@
-// Mixers with a fixed-size state per sequence and head: a matrix S [d, dv] in float32 that every
-// token updates and reads,
-//
-//   plain decay (retention):   S <- a S + k v^T                      o = S^T q
-//   decay per token:           S <- a_t S + k v^T                    o = S^T q
-//   gated delta rule:          S <- diag(g) S;  u = b (v - S^T k);   S <- S + k u^T;   o = S^T q
-//   delta rule, head decay:    S <- a_t S;  u = b (v - S^T k);   S <- S + k u^T;   o = S^T q
-//   generalized delta rule:    S <- diag(g) S + e (c^T S) + k v^T   (both terms read the old S)   o = S^T q
-//   bonus for the newest:      o = (S + diag(m) k v^T)^T q;   S <- diag(g) S + k v^T   (read before the write)
-//
-// with a one decay per head (or, per token, one per head and token: state-space and matrix-memory
-// mixers, whose step size or input gate the caller has multiplied into v), g one decay per head
-// and key channel and token, b one step size per head and token; in the generalized rule c is the
-// direction that is read (a unit key) and e what is written back along it (minus a removal rate
-// per key channel times that direction), both per head, key channel and token; m is one factor per
-// head and key channel that the current token's own contribution has in the read-out. Everything here is float32: the inputs are prepared in float32 by the kernels
-// below (rotation, short convolutions, unit norms, decays), the state lives in float32 in the
-// cache's state storage, one matrix per slot and head, and is carried from step to step.
-//
-// The scan: one CTA per (sequence, head, tile of value columns). Columns of S do not depend on
-// one another, so a CTA keeps its columns in registers for the whole step: thread (column j,
-// part p of P) holds a run of consecutive rows of column j. Per token every thread forms, over its
-// rows, the three partial sums  r = sum g_i S_ij k_i,  s = sum g_i S_ij q_i,  c = sum k_i q_i,
-// which are added over the P parts by shuffles, and then
-//   u_j = b (v_j - r)   (or v_j without the delta rule),   o_j = s + u_j c,   S_ij <- g_i S_ij + k_i u_j,
-// which is the update above with the read-out taken after the write. Tokens are staged through
-// shared memory a chunk at a time by asynchronous copies, the next chunk under way while this
-// one is worked on, so the inner loop has no block-wide barrier and waits for no load. A step of one
-// token (decoding) and a step of a whole prompt run the same arithmetic in the same order, so
-// the state after a prompt does not depend on how it was cut.
-//
-// A sequence of padding (slot < 0) starts from zero and stores nothing.
-#include "common.cuh"
+// The state scans with a plain decay (see recurrent_scan.cuh), the read-out's norm and gate, and the
+// inputs of retention and of the gated delta rule.
+#include "recurrent_scan.cuh"
+
+int g_scan_rows = 16;
+
+extern "C" int lrm_scan_gated_delta(const float* q, const float* k, const float* v, const float* g, const float* beta,
+                                    float* state, float* out, const int* cu_seqlens, const int* slots, int seqs, int H,
+                                    int KH, int d, int dv, cudaStream_t stream);  // recurrent_scan_delta.cu
 
 namespace {
-
-constexpr int kScanThreads = 128;
-constexpr int kChunk = 16;  // tokens per stage, halved while two stages do not fit the shared memory
-
-__device__ __forceinline__ void scan_cp_async(float* dst, const float* src, bool valid, bool wide) {
-  const uint32_t d = static_cast<uint32_t>(__cvta_generic_to_shared(dst));
-  if (wide)
-    asm volatile("cp.async.ca.shared.global [%0], [%1], 16, %2;\n" ::"r"(d), "l"(src), "r"(valid ? 16 : 0));
-  else
-    asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;\n" ::"r"(d), "l"(src), "r"(valid ? 4 : 0));
-}
-
-// Thread (column j, part p) holds rows p * ROWS .. p * ROWS + ROWS - 1 of column j. A token's q, k
-// and g rows lie in shared memory as [P][ROWS + 4] (the 4 floats between the parts keep the parts'
-// 16-byte reads on different banks); tokens come in chunks of kChunk, two chunks in flight.
-// MODE 0: one decay per head (head_decay); 1: the gated delta rule (g, beta); 2: one decay per head
-// and token (in `beta`'s place, [T, H]); 3: the generalized delta rule (g, and the two more rows
-// `look` = c and `put` = e per token, [T, H, d]): with t_j = sum_i c_i S_ij over the old state,
-// S_ij <- g_i S_ij + e_i t_j + k_i v_j and o_j = sum_i g_i S_ij q_i + t_j (e . q) + v_j (k . q);
-// 4: the read-out before the write with a bonus (g, and `look` = m [H, d], the same for every token):
-// o_j = sum_i S_ij q_i + v_j sum_i m_i k_i q_i, then S_ij <- g_i S_ij + k_i v_j: nothing a token adds to
-// the state waits for a sum over it; 5: the delta rule with one decay per head and token (`beta`
-// [T, H] step sizes, `put` [T, H] decays).
-// q and k rows of a token are q_stride floats after those of the token before, v rows v_stride.
-template <int ROWS, int MODE>
-__global__ __launch_bounds__(kScanThreads) void linear_scan_kernel(
-    const float* __restrict__ q, const float* __restrict__ k, const float* __restrict__ v,
-    const float* __restrict__ g, const float* __restrict__ head_decay, const float* __restrict__ beta,
-    const float* __restrict__ look, const float* __restrict__ put,
-    float* __restrict__ state, float* __restrict__ out, const int* __restrict__ cu_seqlens,
-    const int* __restrict__ slots, int H, int KH, int d, int dv, int P, int chunk, long long q_stride,
-    long long v_stride, int wide_rows) {
-  extern __shared__ __align__(16) float smem[];
-  constexpr bool DELTA = MODE == 1 || MODE == 5;
-  constexpr bool GEN = MODE == 3;
-  constexpr bool BONUS = MODE == 4;
-  constexpr bool ROW_DECAY = MODE == 1 || MODE == 3 || MODE == 4;  // a row g of decays per token
-  constexpr int NR = GEN ? 5 : ROW_DECAY ? 3 : 2;      // rows of d floats a token brings
-  constexpr int RS = ROWS + 4;
-  const int TS = P * RS, COLS = kScanThreads / P;
-  const int VS = (COLS + 3) & ~3;                       // v of a token, padded to whole 16 bytes
-  const int TOKEN = NR * TS + VS + 4;                   // q | k | (g) | (look | put) | v | beta, decay
-  const int STAGE = chunk * TOKEN;
-
-  const int tid = threadIdx.x, pidx = tid % P, jl = tid / P;
-  const int h = blockIdx.y, b = blockIdx.z, kh = h / (H / KH);
-  const int j = blockIdx.x * COLS + jl;
-  pdl_wait();
-  const int start = cu_seqlens[b], n = cu_seqlens[b + 1] - start;
-  const int slot = slots[b];
-  float S[ROWS];
-  float* mine = slot >= 0 ? state + (static_cast<size_t>(slot) * H + h) * d * dv : nullptr;
-#pragma unroll
-  for (int i = 0; i < ROWS; ++i) {
-    const int row = pidx * ROWS + i;
-    S[i] = (mine != nullptr && row < d && j < dv) ? mine[static_cast<size_t>(row) * dv + j] : 0.f;
-  }
-  const float a = MODE == 0 ? head_decay[h] : 1.f;
-  float bonus[BONUS ? ROWS : 1];
-  if constexpr (BONUS) {
-#pragma unroll
-    for (int i = 0; i < ROWS; ++i) {
-      const int row = pidx * ROWS + i;
-      bonus[i] = row < d ? look[h * d + row] : 0.f;
-    }
-  }
-  // 16-byte copies where every row of the inputs starts on a 16-byte boundary
-  const bool wide = wide_rows && COLS % 4 == 0;
-  const int step = wide ? 4 : 1;
-
-  auto issue = [&](int c0, int stage) {
-    float* base = smem + stage * STAGE;
-    const int cn = min(chunk, n - c0);
-    const int per_token = ROWS * P / step;  // granules of a q (k, g) row, padding rows included
-    for (int idx = tid; idx < cn * per_token; idx += kScanThreads) {
-      const int c = idx / per_token, r = (idx % per_token) * step;
-      const size_t tok = static_cast<size_t>(start + c0 + c);
-      const bool in = r < d;
-      float* dst = base + c * TOKEN + (r / ROWS) * RS + r % ROWS;
-      scan_cp_async(dst, q + tok * q_stride + kh * d + (in ? r : 0), in, wide);
-      scan_cp_async(dst + TS, k + tok * q_stride + kh * d + (in ? r : 0), in, wide);
-      if (ROW_DECAY) scan_cp_async(dst + 2 * TS, g + (tok * H + h) * d + (in ? r : 0), in, wide);
-      if (GEN) {
-        scan_cp_async(dst + 3 * TS, look + (tok * H + h) * d + (in ? r : 0), in, wide);
-        scan_cp_async(dst + 4 * TS, put + (tok * H + h) * d + (in ? r : 0), in, wide);
-      }
-    }
-    const int v_per_token = COLS / step;
-    for (int idx = tid; idx < cn * v_per_token; idx += kScanThreads) {
-      const int c = idx / v_per_token, cl = (idx % v_per_token) * step, col = blockIdx.x * COLS + cl;
-      const size_t tok = static_cast<size_t>(start + c0 + c);
-      const bool in = col < dv;
-      scan_cp_async(base + c * TOKEN + NR * TS + cl, v + tok * v_stride + h * dv + (in ? col : 0), in, wide);
-    }
-    if (MODE == 1 || MODE == 2 || MODE == 5)
-      for (int c = tid; c < cn; c += kScanThreads) {
-        scan_cp_async(base + c * TOKEN + NR * TS + VS, beta + static_cast<size_t>(start + c0 + c) * H + h,
-                      true, false);
-        if (MODE == 5)
-          scan_cp_async(base + c * TOKEN + NR * TS + VS + 1, put + static_cast<size_t>(start + c0 + c) * H + h,
-                        true, false);
-      }
-    asm volatile("cp.async.commit_group;\n" ::);
-  };
-
-  if (n > 0) issue(0, 0);
-  for (int c0 = 0, it = 0; c0 < n; c0 += chunk, ++it) {
-    const int cn = min(chunk, n - c0);
-    if (c0 + chunk < n) {
-      issue(c0 + chunk, (it + 1) & 1);
-      asm volatile("cp.async.wait_group 1;\n" ::);
-    } else {
-      asm volatile("cp.async.wait_group 0;\n" ::);
-    }
-    __syncthreads();
-    const float* base = smem + (it & 1) * STAGE;
-#pragma unroll (BONUS ? 4 : 2)
-    for (int c = 0; c < cn; ++c) {
-      const float* qc = base + c * TOKEN + pidx * RS;
-      const float* kc = qc + TS;
-      const float* gc = kc + TS;
-      const float at = MODE == 2 ? base[c * TOKEN + 2 * TS + VS] : MODE == 5 ? base[c * TOKEN + 2 * TS + VS + 1] : a;
-      float kr[ROWS];
-      float er[GEN ? ROWS : 1];
-      float r0 = 0.f, r1 = 0.f, s0 = 0.f, s1 = 0.f, kq0 = 0.f, kq1 = 0.f, eq0 = 0.f, eq1 = 0.f;
-#pragma unroll
-      for (int i = 0; i < ROWS; i += 4) {
-        const float4 k4 = *reinterpret_cast<const float4*>(kc + i);
-        const float4 q4 = *reinterpret_cast<const float4*>(qc + i);
-        float4 g4 = make_float4(at, at, at, at);
-        if (ROW_DECAY) g4 = *reinterpret_cast<const float4*>(gc + i);
-        kr[i] = k4.x, kr[i + 1] = k4.y, kr[i + 2] = k4.z, kr[i + 3] = k4.w;
-        if constexpr (GEN) {  // what the old state holds along `look`, before the decay
-          const float4 c4 = *reinterpret_cast<const float4*>(gc + TS + i);
-          const float4 e4 = *reinterpret_cast<const float4*>(gc + 2 * TS + i);
-          r0 = fmaf(S[i], c4.x, r0), r1 = fmaf(S[i + 1], c4.y, r1);
-          r0 = fmaf(S[i + 2], c4.z, r0), r1 = fmaf(S[i + 3], c4.w, r1);
-          er[i] = e4.x, er[i + 1] = e4.y, er[i + 2] = e4.z, er[i + 3] = e4.w;
-          eq0 = fmaf(e4.x, q4.x, eq0), eq1 = fmaf(e4.y, q4.y, eq1);
-          eq0 = fmaf(e4.z, q4.z, eq0), eq1 = fmaf(e4.w, q4.w, eq1);
-        }
-        if constexpr (BONUS) {  // the old state is read, then decayed
-          s0 = fmaf(S[i], q4.x, s0), s1 = fmaf(S[i + 1], q4.y, s1);
-          s0 = fmaf(S[i + 2], q4.z, s0), s1 = fmaf(S[i + 3], q4.w, s1);
-          kq0 = fmaf(k4.x * bonus[i], q4.x, kq0), kq1 = fmaf(k4.y * bonus[i + 1], q4.y, kq1);
-          kq0 = fmaf(k4.z * bonus[i + 2], q4.z, kq0), kq1 = fmaf(k4.w * bonus[i + 3], q4.w, kq1);
-          S[i] *= g4.x, S[i + 1] *= g4.y, S[i + 2] *= g4.z, S[i + 3] *= g4.w;
-          continue;
-        }
-        S[i] *= g4.x, S[i + 1] *= g4.y, S[i + 2] *= g4.z, S[i + 3] *= g4.w;
-        if (DELTA) {
-          r0 = fmaf(S[i], k4.x, r0), r1 = fmaf(S[i + 1], k4.y, r1);
-          r0 = fmaf(S[i + 2], k4.z, r0), r1 = fmaf(S[i + 3], k4.w, r1);
-        }
-        s0 = fmaf(S[i], q4.x, s0), s1 = fmaf(S[i + 1], q4.y, s1);
-        s0 = fmaf(S[i + 2], q4.z, s0), s1 = fmaf(S[i + 3], q4.w, s1);
-        kq0 = fmaf(k4.x, q4.x, kq0), kq1 = fmaf(k4.y, q4.y, kq1);
-        kq0 = fmaf(k4.z, q4.z, kq0), kq1 = fmaf(k4.w, q4.w, kq1);
-      }
-      float r = r0 + r1, s = s0 + s1, kq = kq0 + kq1, eq = eq0 + eq1;
-      for (int o = 1; o < P; o <<= 1) {
-        if (DELTA || GEN) r += __shfl_xor_sync(0xffffffffu, r, o);
-        if (GEN) eq += __shfl_xor_sync(0xffffffffu, eq, o);
-        s += __shfl_xor_sync(0xffffffffu, s, o);
-        kq += __shfl_xor_sync(0xffffffffu, kq, o);
-      }
-      const float vj = base[c * TOKEN + NR * TS + jl];
-      const float u = DELTA ? base[c * TOKEN + NR * TS + VS] * (vj - r) : vj;
-#pragma unroll
-      for (int i = 0; i < ROWS; ++i) S[i] = fmaf(kr[i], u, S[i]);
-      if constexpr (GEN) {
-#pragma unroll
-        for (int i = 0; i < ROWS; ++i) S[i] = fmaf(er[i], r, S[i]);
-        s = fmaf(r, eq, s);
-      }
-      if (pidx == 0 && j < dv)
-        out[(static_cast<size_t>(start + c0 + c) * H + h) * dv + j] = fmaf(u, kq, s);
-    }
-    __syncthreads();
-  }
-  if (mine != nullptr) {
-#pragma unroll
-    for (int i = 0; i < ROWS; ++i) {
-      const int row = pidx * ROWS + i;
-      if (row < d && j < dv) mine[static_cast<size_t>(row) * dv + j] = S[i];
-    }
-  }
-}
-
-// How far apart a token's q and k rows, and its v row, are from those of the token before (0: packed).
-struct RowStrides {
-  long long q = 0, v = 0;
-};
-
-template <int ROWS, int MODE>
-int launch_scan(const float* q, const float* k, const float* v, const float* g, const float* head_decay,
-                const float* beta, const float* look, const float* put, float* state, float* out, const int* cu_seqlens, const int* slots,
-                int seqs, int H, int KH, int d, int dv, int P, const RowStrides& rows, cudaStream_t stream) {
-  constexpr int NR = MODE == 3 ? 5 : MODE == 1 || MODE == 4 ? 3 : 2;
-  const int COLS = kScanThreads / P, TS = P * (ROWS + 4), VS = (COLS + 3) & ~3;
-  int chunk = kChunk;
-  while (chunk > 1 && sizeof(float) * 2 * chunk * (static_cast<size_t>(NR) * TS + VS + 4) > 200 * 1024) chunk >>= 1;
-  const size_t bytes = sizeof(float) * 2 * chunk * (static_cast<size_t>(NR) * TS + VS + 4);
-  if (bytes > 200 * 1024) return LRM_UNSUPPORTED;
-  static bool raised = false;  // per instantiation
-  if (bytes > 48 * 1024 && !raised) {
-    cudaError_t e = cudaFuncSetAttribute(linear_scan_kernel<ROWS, MODE>,
-                                         cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
-    if (e != cudaSuccess) return static_cast<int>(e);
-    raised = true;
-  }
-  const long long q_stride = rows.q > 0 ? rows.q : static_cast<long long>(KH) * d;
-  const long long v_stride = rows.v > 0 ? rows.v : static_cast<long long>(H) * dv;
-  auto aligned = [](const float* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
-  const int wide = d % 4 == 0 && dv % 4 == 0 && q_stride % 4 == 0 && v_stride % 4 == 0 && aligned(q) && aligned(k) &&
-                   aligned(v) && aligned(g) && (MODE != 3 || (aligned(look) && aligned(put)));
-  const dim3 grid((dv + COLS - 1) / COLS, H, seqs);
-  LRM_LAUNCH((linear_scan_kernel<ROWS, MODE>), grid, kScanThreads, bytes, stream, q, k, v, g, head_decay, beta,
-             look, put, state, out, cu_seqlens, slots, H, KH, d, dv, P, chunk, q_stride, v_stride, wide);
-  return 0;
-}
-
-// How a head's key rows are cut over threads: P parts (a power of two up to 32) of ROWS rows.
-// Few parts when the head is small (less to add up by shuffles), more when it is large (the
-// registers a thread can keep bound ROWS to 64).
-int g_scan_rows = 16;  // most rows a thread holds (tuning: lrm_linear_state_scan_rows)
-
-void scan_shape(int d, int* rows, int* parts, int most_rows) {
-  int P = 1;
-  while (P < 32 && (d + P - 1) / P > most_rows) P <<= 1;
-  int need = (d + P - 1) / P, R = 4;
-  while (R < need) R <<= 1;
-  *rows = R;
-  *parts = P;
-}
-
-template <int MODE>
-int dispatch_scan(const float* q, const float* k, const float* v, const float* g, const float* head_decay,
-                  const float* beta, const float* look, const float* put, float* state, float* out, const int* cu_seqlens, const int* slots,
-                  int seqs, int H, int KH, int d, int dv, cudaStream_t stream, const RowStrides& rows = RowStrides{}) {
-  int R, P;
-  scan_shape(d, &R, &P, g_scan_rows);
-  if (MODE == 3 && g_scan_rows > 8) {
-    // Few sequences (one prompt) leave most SMs without a CTA, and every CTA walks its tokens one
-    // after another: with half the rows per thread a head's columns go to twice as many CTAs and a
-    // token's chain of sums is shorter (one prompt of 2,048 tokens, 32 heads of 64 x 64: 643 against
-    // 792 us; a quarter of the rows: 861). Steps that fill the device keep the standard shape.
-    const long long ctas = static_cast<long long>((dv + kScanThreads / P - 1) / (kScanThreads / P)) * H * seqs;
-    if (ctas < 148) scan_shape(d, &R, &P, g_scan_rows / 2);
-  }
-#define LRM_SCAN_CASE(N)                                                                             \
-  case N:                                                                                            \
-    return launch_scan<N, MODE>(q, k, v, g, head_decay, beta, look, put, state, out, cu_seqlens, slots, seqs, H, \
-                                 KH, d, dv, P, rows, stream)
-  switch (R) {
-    LRM_SCAN_CASE(4);
-    LRM_SCAN_CASE(8);
-    LRM_SCAN_CASE(16);
-    LRM_SCAN_CASE(32);
-    LRM_SCAN_CASE(64);
-  }
-#undef LRM_SCAN_CASE
-  return LRM_UNSUPPORTED;
-}
 
 // --------------------------------------------------------------------------- read-out: norm and gate per head
 // out[t, h, :] = o / sqrt(mean(o^2) + eps) * w * act(gate[t, h, :]) * out_scale; w and gate optional.
@@ -333,6 +45,46 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, int o_stride,
       y *= gate_act == 1 ? z * sig : sig;
     }
     out[static_cast<size_t>(t) * out_stride + h * dv + j] = from_f32<A>(y * out_scale);
+  }
+}
+
+// The same with a warp per (token, head), for heads of up to 32 * PER values, which stay in registers.
+template <typename A, typename G, int PER>
+__global__ void head_norm_gate_warp_kernel(const float* o, int o_stride, const float* __restrict__ weight,
+                                           int w_stride, const float* floor, float den_eps, const G* gate,
+                                           long long gate_stride, int gate_act, A* __restrict__ out,
+                                           long long out_stride, long long heads, int H, int dv, float eps,
+                                           float out_scale) {
+  pdl_trigger();
+  pdl_wait();
+  const long long idx = static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (idx >= heads) return;
+  const int lane = threadIdx.x & 31, h = static_cast<int>(idx % H);
+  const size_t t = static_cast<size_t>(idx / H);
+  const float* row = o + idx * o_stride;
+  float under = 1.0f;
+  if (floor != nullptr) under = 1.0f / (fmaxf(fabsf(row[dv]), floor[idx]) + den_eps);
+  float v[PER], z[PER];
+  float ss = 0.f;
+#pragma unroll
+  for (int u = 0; u < PER; ++u) {
+    const int j = lane + 32 * u;
+    v[u] = j < dv ? row[j] * under : 0.f;
+    z[u] = (gate != nullptr && j < dv) ? to_f32(gate[t * gate_stride + h * dv + j]) : 0.f;
+    ss = fmaf(v[u], v[u], ss);
+  }
+  const float inv = 1.0f / sqrtf(warp_sum(ss) / static_cast<float>(dv) + eps);
+#pragma unroll
+  for (int u = 0; u < PER; ++u) {
+    const int j = lane + 32 * u;
+    if (j >= dv) continue;
+    float y = v[u] * inv;
+    if (weight != nullptr) y *= weight[h * w_stride + j];
+    if (gate != nullptr) {
+      const float sig = 1.0f / (1.0f + expf(-z[u]));
+      y *= gate_act == 1 ? z[u] * sig : sig;
+    }
+    out[t * out_stride + h * dv + j] = from_f32<A>(y * out_scale);
   }
 }
 
@@ -504,55 +256,13 @@ LRM_API int lrm_linear_state_scan(const float* q, const float* k, const float* v
   if (d > 2048) return LRM_UNSUPPORTED;
   if (g != nullptr) {
     if (beta == nullptr) return LRM_BAD_ARGUMENT;
-    return dispatch_scan<1>(q, k, v, g, nullptr, beta, nullptr, nullptr, state, out, cu_seqlens, slots, seqs, H, KH, d, dv, stream);
+    return lrm_scan_gated_delta(q, k, v, g, beta, state, out, cu_seqlens, slots, seqs, H, KH, d, dv, stream);
   }
   if (head_decay == nullptr) {  // one decay per head and token, where beta would be
     if (beta == nullptr) return LRM_BAD_ARGUMENT;
     return dispatch_scan<2>(q, k, v, nullptr, nullptr, beta, nullptr, nullptr, state, out, cu_seqlens, slots, seqs, H, KH, d, dv, stream);
   }
   return dispatch_scan<0>(q, k, v, nullptr, head_decay, nullptr, nullptr, nullptr, state, out, cu_seqlens, slots, seqs, H, KH, d,
-                          dv, stream);
-}
-
-// The generalized delta rule: q, k, v, g as above (one key head per head), look and put float32
-// [T, H, d]: S <- diag(g) S + put (look^T S) + k v^T with both terms reading the old S; o = S^T q.
-LRM_API int lrm_general_delta_scan(const float* q, const float* k, const float* v, const float* g, const float* look,
-                                   const float* put, float* state, float* out, const int* cu_seqlens,
-                                   const int* slots, int seqs, int H, int d, int dv, cudaStream_t stream) {
-  if (seqs <= 0) return 0;
-  if (H <= 0 || d <= 0 || dv <= 0 || seqs > 65535 || H > 65535) return LRM_BAD_ARGUMENT;
-  if (g == nullptr || look == nullptr || put == nullptr) return LRM_BAD_ARGUMENT;
-  if (d > 2048) return LRM_UNSUPPORTED;
-  return dispatch_scan<3>(q, k, v, g, nullptr, nullptr, look, put, state, out, cu_seqlens, slots, seqs, H, H, d, dv,
-                          stream);
-}
-
-// The read-out before the write, with a bonus for the current token: q, k at [t * q_stride + h * d], v at
-// [t * v_stride + h * dv] (strides in floats; columns of a wider activation), g float32 [T, H, d], bonus
-// float32 [H, d]: o = (S + diag(bonus) k v^T)^T q, then S <- diag(g) S + k v^T. out float32 [T, H, dv].
-LRM_API int lrm_bonus_state_scan(const float* q, const float* k, long long q_stride, const float* v,
-                                 long long v_stride, const float* g, const float* bonus, float* state, float* out,
-                                 const int* cu_seqlens, const int* slots, int seqs, int H, int d, int dv,
-                                 cudaStream_t stream) {
-  if (seqs <= 0) return 0;
-  if (H <= 0 || d <= 0 || dv <= 0 || seqs > 65535 || H > 65535) return LRM_BAD_ARGUMENT;
-  if (g == nullptr || bonus == nullptr || q_stride < static_cast<long long>(H) * d || v_stride < static_cast<long long>(H) * dv)
-    return LRM_BAD_ARGUMENT;
-  if (d > 2048) return LRM_UNSUPPORTED;
-  return dispatch_scan<4>(q, k, v, g, nullptr, nullptr, bonus, nullptr, state, out, cu_seqlens, slots, seqs, H, H, d,
-                          dv, stream, RowStrides{q_stride, v_stride});
-}
-
-// The delta rule with one decay per head and token: q, k float32 [T, KH, d], v [T, H, dv], decay and beta
-// float32 [T, H]: S <- decay S;  S <- S + k (beta (v - S^T k))^T;  o = S^T q.
-LRM_API int lrm_head_decay_delta_scan(const float* q, const float* k, const float* v, const float* decay,
-                                      const float* beta, float* state, float* out, const int* cu_seqlens,
-                                      const int* slots, int seqs, int H, int KH, int d, int dv, cudaStream_t stream) {
-  if (seqs <= 0) return 0;
-  if (H <= 0 || KH <= 0 || H % KH || d <= 0 || dv <= 0 || seqs > 65535 || H > 65535) return LRM_BAD_ARGUMENT;
-  if (decay == nullptr || beta == nullptr) return LRM_BAD_ARGUMENT;
-  if (d > 2048) return LRM_UNSUPPORTED;
-  return dispatch_scan<5>(q, k, v, nullptr, nullptr, beta, nullptr, decay, state, out, cu_seqlens, slots, seqs, H, KH, d,
                           dv, stream);
 }
 
@@ -569,20 +279,31 @@ LRM_API int lrm_head_norm_gate(const float* o, int o_stride, const float* weight
   if (o_stride < dv || (floor != nullptr && o_stride <= dv) || (w_stride != 0 && w_stride != dv)) return LRM_BAD_ARGUMENT;
   const int threads = dv >= 256 ? 256 : ((dv + 31) / 32) * 32;
   const dim3 grid(tokens, H);
+  const long long heads = static_cast<long long>(tokens) * H;
+#define LRM_HEAD_WARP(AT, GT, PER)                                                                          \
+  LRM_LAUNCH((head_norm_gate_warp_kernel<AT, GT, PER>), static_cast<unsigned>((heads + 3) / 4), 128, 0, stream, o, \
+             o_stride, weight, w_stride, floor, den_eps, static_cast<const GT*>(gate), gate_stride, gate_act, \
+             static_cast<AT*>(out), out_stride, heads, H, dv, eps, out_scale)
 #define LRM_HEAD_NORM(AT, GT)                                                                              \
+  if (dv <= 64) LRM_HEAD_WARP(AT, GT, 2);                                                                  \
+  else if (dv <= 128) LRM_HEAD_WARP(AT, GT, 4);                                                            \
+  else if (dv <= 256) LRM_HEAD_WARP(AT, GT, 8);                                                            \
+  else                                                                                                     \
   LRM_LAUNCH((head_norm_gate_kernel<AT, GT>), grid, threads, 0, stream, o, o_stride, weight, w_stride, floor,    \
              den_eps, static_cast<const GT*>(gate), gate_stride, gate_act, static_cast<AT*>(out), out_stride, H, dv, eps, \
              out_scale)
-  if (dtype == LRM_F32 && gate_dtype == LRM_F32)
+  if (dtype == LRM_F32 && gate_dtype == LRM_F32) {
     LRM_HEAD_NORM(float, float);
-  else if (dtype == LRM_F32 && gate_dtype == LRM_BF16)
+  } else if (dtype == LRM_F32 && gate_dtype == LRM_BF16) {
     LRM_HEAD_NORM(float, __nv_bfloat16);
-  else if (dtype == LRM_BF16 && gate_dtype == LRM_F32)
+  } else if (dtype == LRM_BF16 && gate_dtype == LRM_F32) {
     LRM_HEAD_NORM(__nv_bfloat16, float);
-  else if (dtype == LRM_BF16 && gate_dtype == LRM_BF16)
+  } else if (dtype == LRM_BF16 && gate_dtype == LRM_BF16) {
     LRM_HEAD_NORM(__nv_bfloat16, __nv_bfloat16);
-  else
+  } else {
     return LRM_BAD_ARGUMENT;
+  }
+#undef LRM_HEAD_WARP
 #undef LRM_HEAD_NORM
   return 0;
 }

@@ -12,7 +12,8 @@
 //      query heads and one for all key heads;
 //   5. a rotation by position of the first `rotary` dimensions of every query and key head,
 //      dimension i paired with i + rotary/2 (pairing 0) or 2i with 2i + 1 (pairing 1), angle =
-//      position * inv_freq[i] formed in double precision;
+//      position * inv_freq[i] formed in double precision, here or, for layers that share their
+//      frequencies, once per step in a table of cosines and sines (lrm_rope_table64);
 //   6. the division of every query and key head by its root mean square (no weight),
 // and writes q, k, v in the activation type: q packed, k and v packed (when asked for) and into
 // the paged cache at dest_rows[t] (see qkv_store.cu for the layout). Everything between the
@@ -33,7 +34,8 @@ __global__ void shaped_qkv_kernel(const S* proj, long long stride, const float* 
                                   const int* __restrict__ positions, const float* __restrict__ q_norm,
                                   const float* __restrict__ k_norm, float row_eps,
                                   const float* __restrict__ q_head_w, const float* __restrict__ k_head_w,
-                                  float head_w_eps, const double* __restrict__ inv_freq, int rotary, int pairing, int head_norm,
+                                  float head_w_eps, const double* __restrict__ inv_freq, const float2* table,
+                                  int rotary, int pairing, int head_norm,
                                   float head_eps, A* __restrict__ q_out, A* __restrict__ k_out,
                                   A* __restrict__ v_out, A* __restrict__ k_pages, A* __restrict__ v_pages,
                                   const int* __restrict__ dest_rows, int q_heads, int kv_heads, int d, int dv,
@@ -47,13 +49,20 @@ __global__ void shaped_qkv_kernel(const S* proj, long long stride, const float* 
   pdl_trigger();
   const int t = blockIdx.x;
   const int pos = positions[t];
-  for (int i = threadIdx.x; i < half; i += blockDim.x) {
-    double sn, c;
-    sincos(static_cast<double>(pos) * inv_freq[i], &sn, &c);
-    cs[i] = static_cast<float>(c);
-    cs[half + i] = static_cast<float>(sn);
-  }
+  if (table == nullptr)
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+      double sn, c;
+      sincos(static_cast<double>(pos) * inv_freq[i], &sn, &c);
+      cs[i] = static_cast<float>(c);
+      cs[half + i] = static_cast<float>(sn);
+    }
   pdl_wait();
+  if (table != nullptr)
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+      const float2 entry = table[static_cast<size_t>(t) * half + i];
+      cs[i] = entry.x;
+      cs[half + i] = entry.y;
+    }
   const S* src = proj + static_cast<size_t>(t) * stride;
   if (taps == nullptr || n <= 1) {
     for (int c = threadIdx.x; c < width; c += blockDim.x) {
@@ -173,25 +182,29 @@ template <typename S, typename A, int VEC>
 __global__ void shaped_heads_kernel(const S* proj, long long stride, const float* __restrict__ bias,
                                     const int* __restrict__ positions, const float* __restrict__ q_head_w,
                                     const float* __restrict__ k_head_w, float head_w_eps,
-                                    const double* __restrict__ inv_freq, int rotary, int pairing,
+                                    const double* __restrict__ inv_freq, const float2* table, int rotary, int pairing,
                                     A* __restrict__ q_out, A* __restrict__ k_out, A* __restrict__ v_out,
                                     A* __restrict__ k_pages, A* __restrict__ v_pages,
                                     const int* __restrict__ dest_rows, int q_heads, int kv_heads, int d, int dv,
                                     int page_size) {
-  extern __shared__ float cs[];  // [rotary / 2] cosines, then as many sines
+  extern __shared__ float cs[];  // without a table: [rotary / 2] cosines, then as many sines
   const int half = rotary / 2;
   pdl_trigger();
-  const int t = blockIdx.x, pos = positions[t];
-  for (int i = threadIdx.x; i < half; i += blockDim.x) {
-    double sn, c;
-    sincos(static_cast<double>(pos) * inv_freq[i], &sn, &c);
-    cs[i] = static_cast<float>(c);
-    cs[half + i] = static_cast<float>(sn);
+  const int t = blockIdx.x;
+  const float2* angles = table != nullptr ? table + static_cast<size_t>(t) * half : nullptr;
+  if (table == nullptr) {
+    const int pos = positions[t];
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+      double sn, c;
+      sincos(static_cast<double>(pos) * inv_freq[i], &sn, &c);
+      cs[i] = static_cast<float>(c);
+      cs[half + i] = static_cast<float>(sn);
+    }
+    __syncthreads();
   }
   const int dest = k_pages != nullptr ? dest_rows[t] : -1;
   const size_t page = dest >= 0 ? static_cast<size_t>(dest / page_size) : 0;
   const int in_page = dest >= 0 ? dest % page_size : 0;
-  __syncthreads();
   pdl_wait();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
   const S* row = proj + static_cast<size_t>(t) * stride;
@@ -239,7 +252,8 @@ __global__ void shaped_heads_kernel(const S* proj, long long stride, const float
           const int other = pairing == 0 ? (leads ? c + half : c - half) : (leads ? c + 1 : c - 1);
           float p = to_f32(src[other]) + (add != nullptr ? add[other] : 0.f);
           if (w != nullptr) p = (p * inv) * w[other];
-          const float co = cs[pair], sn = cs[half + pair];
+          const float2 turn = angles != nullptr ? angles[pair] : make_float2(cs[pair], cs[half + pair]);
+          const float co = turn.x, sn = turn.y;
           v = leads ? fmaf(v, co, -__fmul_rn(p, sn)) : fmaf(v, co, __fmul_rn(p, sn));
         }
         y[e] = from_f32<A>(v);
@@ -268,15 +282,16 @@ LRM_API int lrm_shaped_qkv_store(const void* proj, int in_dtype, long long strid
                                  const float* tails, const int* cu_seqlens, const int* seq_of_token,
                                  const int* slots, const int* positions, const float* q_norm, const float* k_norm,
                                  float row_eps, const float* q_head_w, const float* k_head_w, float head_w_eps,
-                                 const double* inv_freq, int rotary, int pairing, int head_norm,
+                                 const double* inv_freq, const float* table, int rotary, int pairing, int head_norm,
                                  float head_eps, void* q_out, void* k_out, void* v_out, void* k_pages, void* v_pages,
                                  const int* dest_rows, int out_dtype, int tokens, int q_heads, int kv_heads, int d,
                                  int dv, int page_size, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (q_heads <= 0 || kv_heads < 0 || d <= 0 || dv < 0 || page_size <= 0 || positions == nullptr) return LRM_BAD_ARGUMENT;
-  if (rotary < 0 || rotary > d || rotary % 2 || (rotary > 0 && inv_freq == nullptr) || (pairing != 0 && pairing != 1))
+  if (rotary < 0 || rotary > d || rotary % 2 || (rotary > 0 && inv_freq == nullptr && table == nullptr) || (pairing != 0 && pairing != 1))
     return LRM_BAD_ARGUMENT;
-  if (inv_freq == nullptr) rotary = 0;
+  if (inv_freq == nullptr && table == nullptr) rotary = 0;
+  const float2* turns = reinterpret_cast<const float2*>(table);
   if ((q_norm != nullptr && kv_heads > 0 && k_norm == nullptr) || (q_norm == nullptr && k_norm != nullptr))
     return LRM_BAD_ARGUMENT;
   if (taps != nullptr && n > 1 && (tails == nullptr || cu_seqlens == nullptr || seq_of_token == nullptr || slots == nullptr))
@@ -294,7 +309,7 @@ LRM_API int lrm_shaped_qkv_store(const void* proj, int in_dtype, long long strid
     const bool pairs = d % 2 == 0 && dv % 2 == 0 && stride % 2 == 0 && reinterpret_cast<uintptr_t>(proj) % in_pair == 0;
 #define LRM_HEADS(ST, AT, V)                                                                                        \
   LRM_LAUNCH((shaped_heads_kernel<ST, AT, V>), grid, threads, sizeof(float) * rotary, stream, static_cast<const ST*>(proj), \
-             stride, bias, positions, q_head_w, k_head_w, head_w_eps, inv_freq, rotary, pairing, static_cast<AT*>(q_out), \
+             stride, bias, positions, q_head_w, k_head_w, head_w_eps, inv_freq, turns, rotary, pairing, static_cast<AT*>(q_out), \
              static_cast<AT*>(k_out), static_cast<AT*>(v_out), static_cast<AT*>(k_pages), static_cast<AT*>(v_pages), \
              dest_rows, q_heads, kv_heads, d, dv, page_size)
     if (in_dtype == LRM_F32 && out_dtype == LRM_F32) {
@@ -321,7 +336,7 @@ LRM_API int lrm_shaped_qkv_store(const void* proj, int in_dtype, long long strid
       raised = true;                                                                                            \
     }                                                                                                           \
     LRM_LAUNCH((shaped_qkv_kernel<ST, AT>), tokens, width >= 2048 ? 512 : 256, bytes, stream, static_cast<const ST*>(proj), stride, bias, taps, n, \
-               tails, cu_seqlens, seq_of_token, slots, positions, q_norm, k_norm, row_eps, q_head_w, k_head_w, head_w_eps, inv_freq, rotary, \
+               tails, cu_seqlens, seq_of_token, slots, positions, q_norm, k_norm, row_eps, q_head_w, k_head_w, head_w_eps, inv_freq, turns, rotary, \
                pairing, head_norm, head_eps, static_cast<AT*>(q_out), static_cast<AT*>(k_out),                  \
                static_cast<AT*>(v_out), static_cast<AT*>(k_pages), static_cast<AT*>(v_pages), dest_rows, q_heads, \
                kv_heads, d, dv, page_size);                                                                     \

@@ -100,7 +100,8 @@ __device__ __forceinline__ void mma_bf16_16816(float (&c)[4], const uint32_t (&a
 __global__ __launch_bounds__(128) void decay_product_bf16_kernel(const float* z, long long stride,
                                                                  const __nv_bfloat16* __restrict__ W,
                                                                  const float* __restrict__ bias,
-                                                                 float* __restrict__ g, int M, int N, int K) {
+                                                                 float* __restrict__ g, int M, int N, int K,
+                                                                 int fours) {
   constexpr int BK = 64, PITCH = BK + 8;
   __shared__ __align__(16) __nv_bfloat16 Zs[kM][PITCH], Ws[kN][PITCH];
   pdl_trigger();
@@ -108,14 +109,31 @@ __global__ __launch_bounds__(128) void decay_product_bf16_kernel(const float* z,
   const int wm = (warp >> 1) * 32, wn = (warp & 1) * 32, m0 = blockIdx.y * kM, n0 = blockIdx.x * kN;
   float acc[2][4][4] = {};
   for (int k0 = 0; k0 < K; k0 += BK) {
-    for (int idx = tid; idx < kN * BK; idx += 128) {  // a weight: needs no wait
-      const int r = idx / BK, c = idx % BK;
-      Ws[r][c] = (n0 + r < N && k0 + c < K) ? W[static_cast<size_t>(n0 + r) * K + k0 + c] : __float2bfloat16_rn(0.f);
-    }
-    if (k0 == 0) pdl_wait();
-    for (int idx = tid; idx < kM * BK; idx += 128) {
-      const int r = idx / BK, c = idx % BK;
-      Zs[r][c] = __float2bfloat16_rn((m0 + r < M && k0 + c < K) ? tanhf(z[static_cast<size_t>(m0 + r) * stride + k0 + c]) : 0.f);
+    if (fours) {
+      for (int idx = tid; idx < kN * BK / 4; idx += 128) {  // a weight: needs no wait
+        const int r = idx / (BK / 4), c = idx % (BK / 4) * 4;
+        uint2 w = make_uint2(0u, 0u);
+        if (n0 + r < N && k0 + c < K) w = *reinterpret_cast<const uint2*>(W + static_cast<size_t>(n0 + r) * K + k0 + c);
+        *reinterpret_cast<uint2*>(&Ws[r][c]) = w;
+      }
+      if (k0 == 0) pdl_wait();
+      for (int idx = tid; idx < kM * BK / 4; idx += 128) {
+        const int r = idx / (BK / 4), c = idx % (BK / 4) * 4;
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (m0 + r < M && k0 + c < K) v = *reinterpret_cast<const float4*>(z + static_cast<size_t>(m0 + r) * stride + k0 + c);
+        __nv_bfloat162 lo = __floats2bfloat162_rn(tanhf(v.x), tanhf(v.y)), hi = __floats2bfloat162_rn(tanhf(v.z), tanhf(v.w));
+        *reinterpret_cast<uint2*>(&Zs[r][c]) = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
+      }
+    } else {
+      for (int idx = tid; idx < kN * BK; idx += 128) {
+        const int r = idx / BK, c = idx % BK;
+        Ws[r][c] = (n0 + r < N && k0 + c < K) ? W[static_cast<size_t>(n0 + r) * K + k0 + c] : __float2bfloat16_rn(0.f);
+      }
+      if (k0 == 0) pdl_wait();
+      for (int idx = tid; idx < kM * BK; idx += 128) {
+        const int r = idx / BK, c = idx % BK;
+        Zs[r][c] = __float2bfloat16_rn((m0 + r < M && k0 + c < K) ? tanhf(z[static_cast<size_t>(m0 + r) * stride + k0 + c]) : 0.f);
+      }
     }
     __syncthreads();
 #pragma unroll
@@ -147,9 +165,17 @@ __global__ __launch_bounds__(128) void decay_product_bf16_kernel(const float* z,
 #pragma unroll
     for (int j = 0; j < 4; ++j)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int m = m0 + wm + i * 16 + gq + 8 * (e >> 1), n = n0 + wn + j * 8 + 2 * t + (e & 1);
-        if (m < M && n < N) g[static_cast<size_t>(m) * N + n] = decay_of(acc[i][j][e] + bias[n]);
+      for (int half = 0; half < 2; ++half) {
+        const int m = m0 + wm + i * 16 + gq + 8 * half, n = n0 + wn + j * 8 + 2 * t;
+        if (m >= M || n >= N) continue;
+        float* dst = g + static_cast<size_t>(m) * N + n;
+        const float first = decay_of(acc[i][j][2 * half] + bias[n]);
+        if (N % 2 == 0) {
+          *reinterpret_cast<float2*>(dst) = make_float2(first, decay_of(acc[i][j][2 * half + 1] + bias[n + 1]));
+        } else {
+          dst[0] = first;
+          if (n + 1 < N) dst[1] = decay_of(acc[i][j][2 * half + 1] + bias[n + 1]);
+        }
       }
 }
 
@@ -194,7 +220,9 @@ LRM_API int lrm_decay_product(const float* z, long long stride, const void* W, i
     LRM_LAUNCH(decay_product_f32_kernel, grid, 256, 0, stream, z, stride, static_cast<const float*>(W), bias, g, M, N, K);
   else if (w_dtype == LRM_BF16)
     LRM_LAUNCH(decay_product_bf16_kernel, grid, 128, 0, stream, z, stride, static_cast<const __nv_bfloat16*>(W), bias, g,
-               M, N, K);
+               M, N, K,
+               K % 4 == 0 && stride % 4 == 0 && reinterpret_cast<uintptr_t>(z) % 16 == 0 &&
+                   reinterpret_cast<uintptr_t>(W) % 8 == 0);
   else
     return LRM_BAD_ARGUMENT;
   return 0;

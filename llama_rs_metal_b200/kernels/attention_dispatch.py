@@ -460,12 +460,19 @@ def attend(projected, *, q_heads: int, kv_heads: int, head_dim: int, rotary, ctx
                       keep_packed=prefill_phase and writes_cache)
         if shaping is not None:
             s = shaping
+            table = None
+            if s.inv_freq is not None:  # one table of angles per step and set of frequencies
+                key = ("rope_table64", s.inv_freq.data_ptr())
+                table = ctx.scratch.get(key)
+                if table is None:
+                    table = ctx.scratch[key] = ops.rope_table64(ctx.positions, s.inv_freq)
             q, k, v = ops.shaped_qkv_store(
                 projected, q_heads, kv_heads if writes_cache else 0, head_dim, dv, ctx.positions, ctx.runtime.dtype,
                 bias=bias, taps=s.taps, tails=s.tails.state if s.tails is not None else None,
                 cu_seqlens=ctx.cu_seqlens, seq_of_token=ctx.seq_of_token, slots=ctx.slots, row_norm=s.row_norm,
-                row_eps=s.row_eps, head_weights=s.head_weights, head_weight_eps=s.head_weight_eps, inv_freq=s.inv_freq, rotary=s.rotary, adjacent_pairs=s.adjacent_pairs,
-                head_norm_eps=s.head_norm_eps, **stored)
+                row_eps=s.row_eps, head_weights=s.head_weights, head_weight_eps=s.head_weight_eps,
+                inv_freq=s.inv_freq, rotary=s.rotary, adjacent_pairs=s.adjacent_pairs, head_norm_eps=s.head_norm_eps,
+                table=table, **stored)
         else:
             q, k, v = ops.qkv_bias_store(projected, bias, q_heads, kv_heads if writes_cache else 0, head_dim, dv,
                                          **stored)

@@ -148,6 +148,9 @@ def rms_norm_add_(stream: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, e
     return out
 
 
+LAYER_NORM_FOLDS = 8192  # rows of up to this length are held in registers with room to add slices to them
+
+
 def _check_norm(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], partials: Optional[torch.Tensor],
                 what: str):
     """Shared checks of the layer norms; -> (planes to add, elements between them)."""
@@ -172,6 +175,9 @@ def layer_norm(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tenso
     the rows (and written back, unless rows are gathered). -> [T or len(rows), h] in `out_dtype`."""
     n_partials, stride = _check_norm(x, weight, bias, partials, "layer_norm")
     hidden = x.shape[1]
+    if n_partials and hidden > LAYER_NORM_FOLDS:
+        add_planes_(x, partials)
+        partials, n_partials, stride = None, 0, 0
     n_rows = x.shape[0]
     if rows is not None:
         _check(rows, "rows", torch.int32, 1)
@@ -600,6 +606,17 @@ def rope_table(positions: torch.Tensor, inv_freq: torch.Tensor) -> torch.Tensor:
     return table
 
 
+def rope_table64(positions: torch.Tensor, inv_freq: torch.Tensor) -> torch.Tensor:
+    """float32 [T, R/2, 2]: (cos, sin) of position * inv_freq with the angle in double precision (inv_freq
+    float64), the angles shaped_qkv_store forms."""
+    _check(positions, "positions", torch.int32, 1)
+    _check(inv_freq, "inv_freq", torch.float64, 1)
+    T, half = positions.numel(), inv_freq.numel()
+    table = torch.empty((T, half, 2), dtype=torch.float32, device=positions.device)
+    _done(_lib().lrm_rope_table64(_ptr(positions), _ptr(inv_freq), _ptr(table), T, half, _stream()), "rope_table64")
+    return table
+
+
 def linear_rope_store(x: torch.Tensor, weight: torch.Tensor, q_heads: int, kv_heads: int, head_dim: int,
                       table: Optional[torch.Tensor], kv=None, dest_rows: Optional[torch.Tensor] = None):
     """rope_store(linear(x, weight)) for a prompt in one launch where the tensor-core product takes
@@ -669,7 +686,7 @@ def shaped_qkv_store(qkv: torch.Tensor, q_heads: int, kv_heads: int, head_dim: i
                      slots: Optional[torch.Tensor] = None, row_norm=None, row_eps: float = 0.0,
                      head_weights=None, head_weight_eps: float = 0.0, inv_freq: Optional[torch.Tensor] = None, rotary: int = 0, adjacent_pairs: bool = False,
                      head_norm_eps: Optional[float] = None, kv=None, dest_rows: Optional[torch.Tensor] = None,
-                     keep_packed: bool = True):
+                     keep_packed: bool = True, table: Optional[torch.Tensor] = None):
     """Split a fused [T, Hq*d + Hk*d + Hk*dv (+ more)] projection (float32, or `out_dtype`; columns behind
     the row are left alone) whose queries and keys are shaped on the way, each step only if asked for and in this order: `bias` (float32
     [row]); a causal convolution per channel (`taps` float32 [n, row], the last row the current
@@ -678,7 +695,8 @@ def shaped_qkv_store(qkv: torch.Tensor, q_heads: int, kv_heads: int, head_dim: i
     query columns and one over all key columns (`row_norm` = (q weight, k weight), `row_eps`); an RMS
     norm over every query and every key head (`head_weights` = (q weight, k weight), float32 [d] each,
     `head_weight_eps`); the rotation of each head's first `rotary` dimensions by `inv_freq` (float64 [rotary/2]; split halves,
-    or neighbours with `adjacent_pairs`); each head divided by its root mean square
+    or neighbours with `adjacent_pairs`; `table`: rope_table64 of the step, which saves the kernel its
+    angles); each head divided by its root mean square
     (`head_norm_eps`). Returns (q [T,Hq,d], k, v) like qkv_bias_store, and writes the cache view."""
     _check(qkv, "qkv", dims=2)
     T = qkv.shape[0]
@@ -725,6 +743,10 @@ def shaped_qkv_store(qkv: torch.Tensor, q_heads: int, kv_heads: int, head_dim: i
         _check(inv_freq, "inv_freq", torch.float64, 1)
         if inv_freq.numel() != rotary // 2 or rotary % 2 or rotary > head_dim:
             raise InvalidError("shaped_qkv_store: one frequency per rotated pair")
+        if table is not None:
+            _check(table, "table", torch.float32, 3)
+            if tuple(table.shape) != (T, rotary // 2, 2):
+                raise InvalidError("shaped_qkv_store: the table has one angle per token and rotated pair")
     dev = qkv.device
     q = torch.empty((T, q_heads, head_dim), dtype=out_dtype, device=dev)
     k = torch.empty((T, kv_heads, head_dim), dtype=out_dtype, device=dev) if keep_packed and kv_heads else None
@@ -747,7 +769,7 @@ def shaped_qkv_store(qkv: torch.Tensor, q_heads: int, kv_heads: int, head_dim: i
         _ptr(tails if n > 1 else None),
         _ptr(cu_seqlens if n > 1 else None), _ptr(seq_of_token if n > 1 else None), _ptr(slots if n > 1 else None),
         _ptr(positions), _ptr(q_norm), _ptr(k_norm), ctypes.c_float(row_eps), _ptr(q_head), _ptr(k_head),
-        ctypes.c_float(head_weight_eps), _ptr(inv_freq if rotary else None), rotary, int(bool(adjacent_pairs)), int(head_norm_eps is not None),
+        ctypes.c_float(head_weight_eps), _ptr(inv_freq if rotary else None), _ptr(table if rotary else None), rotary, int(bool(adjacent_pairs)), int(head_norm_eps is not None),
         ctypes.c_float(head_norm_eps if head_norm_eps is not None else 0.0), _ptr(q), _ptr(k), _ptr(v),
         _ptr(k_pages), _ptr(v_pages), _ptr(dest_rows if k_pages is not None else None), _code(out_dtype), T, q_heads,
         kv_heads, head_dim, value_dim, page_size, _stream()), "shaped_qkv_store")

@@ -60,6 +60,7 @@ WORK: Dict[str, Callable[..., Tuple[float, float]]] = {
     # the fused q|k|v projection of a prompt: the product, its bfloat16 result stored packed and k, v again in the cache
     "lrm_gemm_bf16_umma_qkv": lambda a: _gemm(_v(a[2]), _v(a[3]), _v(a[4]), 2),
     "lrm_gemm_bf16_umma_pair_qkv": lambda a: _gemm(_v(a[2]), _v(a[3]), _v(a[4]), 2),
+    "lrm_rope_table64": lambda a: (_v(a[3]) * _v(a[4]) * 8.0 + _v(a[3]) * 4.0, 0),
     "lrm_rope_table": lambda a: (_v(a[3]) * _v(a[4]) * 8.0 + _v(a[3]) * 4.0, 0),
     "lrm_gemm_bf16_stream_pick": lambda a: _gemm(_v(a[2]), _v(a[3]), _v(a[4]), 0),
     "lrm_rope_store": lambda a: (2.0 * _v(a[11]) * (_v(a[12]) + 2 * _v(a[13])) * _v(a[14]) * _ELEM[_v(a[1])], 0),
@@ -153,14 +154,45 @@ WORK: Dict[str, Callable[..., Tuple[float, float]]] = {
         _v(a[18]) * _v(a[19]) * ((3 * _v(a[20]) + _v(a[21])) * _ELEM[_v(a[1])] + 4.0 * (6 * _v(a[20]) + _v(a[21]))), 0),
     # the shaped split: the projection row read (taps times, from cache), q, k, v written, k and v again into the cache
     "lrm_shaped_qkv_store": lambda a: (
-        _v(a[25]) * ((_v(a[26]) * _v(a[28]) + _v(a[27]) * (_v(a[28]) + _v(a[29]))) * (_ELEM[_v(a[1])] + _ELEM[_v(a[24])])
-                     + _v(a[27]) * (_v(a[28]) + _v(a[29])) * _ELEM[_v(a[24])]),
-        2.0 * _v(a[25]) * (_v(a[26]) * _v(a[28]) + _v(a[27]) * (_v(a[28]) + _v(a[29]))) * max(1, _v(a[4]))),
+        _v(a[30]) * ((_v(a[31]) * _v(a[33]) + _v(a[32]) * (_v(a[33]) + _v(a[34]))) * (_ELEM[_v(a[1])] + _ELEM[_v(a[29])])
+                     + _v(a[32]) * (_v(a[33]) + _v(a[34])) * _ELEM[_v(a[29])]),
+        2.0 * _v(a[30]) * (_v(a[31]) * _v(a[33]) + _v(a[32]) * (_v(a[33]) + _v(a[34]))) * max(1, _v(a[5]))),
     "lrm_token_shift": lambda a: (_v(a[8]) * _v(a[9]) * 2.0 * _ELEM[_v(a[1])], 0),
     "lrm_scaled_add": lambda a: (12.0 * _v(a[3]) * _v(a[4]), 0),
     "lrm_row_gate": lambda a: (_v(a[4]) * (_v(a[5]) * _ELEM[_v(a[2])] + (8.0 + 4.0 * _v(a[8])) * _v(a[6])), 0),
     "lrm_scaled_add_norm": lambda a: (_v(a[8]) * _v(a[9]) * (12.0 + _ELEM[_v(a[7])]), 5.0 * _v(a[8]) * _v(a[9])),
     "lrm_gelu_tanh_mul": lambda a: (_v(a[4]) * _v(a[5]) * (2.0 * _ELEM[_v(a[1])] + _ELEM[_v(a[3])]), 0),
+    # several products in one launch: every input's rows once, the stacked matrix, float32 sums
+    "lrm_gemm_bf16_stream_grouped": lambda a: _gemm(_v(a[3]), _v(a[4]), _v(a[5]), 4),
+    "lrm_gemm_bf16_umma_grouped": lambda a: _gemm(_v(a[3]), _v(a[5]), _v(a[6]), 4),
+    "lrm_gemm_bf16_umma_pair_grouped": lambda a: _gemm(_v(a[3]), _v(a[5]), _v(a[6]), 4),
+    "lrm_gemm_bf16_mma_grouped": lambda a: _gemm(_v(a[3]), _v(a[4]), _v(a[5]), 4),
+    "lrm_gemm_f32_grouped": lambda a: _gemm(_v(a[3]), _v(a[4]), _v(a[5]), 4, 4),
+    "lrm_layer_norm_conv": lambda a: (_v(a[12]) * _v(a[13]) * (4.0 + _ELEM[_v(a[4])] + 8.0 * _v(a[9]) + 4.0 * _v(a[6])), 0),
+    "lrm_input_conv": lambda a: (_v(a[9]) * _v(a[10]) * 2.0 * _ELEM[_v(a[1])], 2.0 * _v(a[9]) * _v(a[10]) * _v(a[3])),
+    "lrm_stream_swap": lambda a: (_v(a[6]) * (12.0 + 4.0 * _v(a[3]) + _ELEM[_v(a[5])]), 0),
+    "lrm_softcap_inplace": lambda a: (8.0 * _v(a[2]), 0),
+    "lrm_token_mixes": lambda a: (_v(a[10]) * _v(a[11]) * (1.0 + _v(a[3])) * _ELEM[_v(a[1])], 0),
+    "lrm_decay_product": lambda a: (4.0 * _v(a[6]) * (_v(a[7]) + _v(a[8])) + _ELEM[_v(a[3])] * _v(a[7]) * _v(a[8]),
+                                    2.0 * _v(a[6]) * _v(a[7]) * _v(a[8])),
+    "lrm_head_decay_delta_prepare": lambda a: (
+        _v(a[19]) * ((2 * _v(a[21]) * _v(a[22]) + _v(a[20]) * _v(a[23])) * (_ELEM[_v(a[1])] + 4.0)
+                     + _v(a[20]) * (2.0 * _ELEM[_v(a[1])] + 8.0)), 0),
+    # the state scans: states read and written once, the step's inputs and outputs once; per token and
+    # state element a decay, two sums and the update (delta: three)
+    "lrm_bonus_state_scan": lambda a: (
+        8.0 * _v(a[11]) * _v(a[12]) * _v(a[13]) * _v(a[14]) + 4.0 * hints["tokens"] * _v(a[12]) * (3 * _v(a[13]) + 2 * _v(a[14])),
+        hints["tokens"] * _v(a[12]) * _v(a[13]) * _v(a[14]) * 5.0),
+    "lrm_head_decay_delta_scan": lambda a: (
+        8.0 * _v(a[9]) * _v(a[10]) * _v(a[12]) * _v(a[13])
+        + 4.0 * hints["tokens"] * (2 * _v(a[11]) * _v(a[12]) + 2 * _v(a[10]) * (_v(a[13]) + 1)),
+        hints["tokens"] * _v(a[10]) * _v(a[12]) * _v(a[13]) * 7.0),
+    # attention with sigmoid weights, counted like the softmax kernels above
+    "lrm_attention_sigmoid_tiled": lambda a: (2.0 * hints["kv_tokens"] * _v(a[13]) * _v(a[14]) * 2 if a[6] else 0,
+                                              4.0 * hints["pairs"] * _v(a[12]) * _v(a[14])),
+    "lrm_attention_sigmoid_decode": lambda a: (2.0 * hints["kv_tokens"] * _v(a[11]) * _v(a[12]) * 2, 0),
+    "lrm_attention_sigmoid_rowwise": lambda a: (
+        (2.0 * hints["kv_tokens"] * _v(a[15]) * _v(a[16]) * _ELEM[_v(a[4])], 0) if a[9] else (0, 4.0 * hints["pairs"] * _v(a[14]) * _v(a[16]))),
     "lrm_tanh_columns": lambda a: (_v(a[5]) * _v(a[6]) * (_ELEM[_v(a[1])] + _ELEM[_v(a[4])]), 0),
 }
 # entry points that only answer questions and launch nothing

@@ -26,7 +26,7 @@ from __future__ import annotations
 import math
 
 from ..config.tarupel import TarupelConfig
-from ..parts.base import LayerSpec, ModelPlan, PartSpec, ScheduleEntry
+from ..parts.base import LayerSpec, ModelPlan, PartSpec, ScheduleEntry, looped_runs
 from ..registry import register_architecture
 
 MAX_POSITIONS = 1 << 20          # the design names no limit
@@ -99,18 +99,6 @@ def _feed_forward(config: TarupelConfig, f, p: str) -> PartSpec:
         names=names)
 
 
-def layer_runs(config: TarupelConfig):
-    """[(layer, pass number or None)] in the order the layers run: the pass number stands at the
-    first layer of each pass of the looped run."""
-    n = len(config.layers)
-    if not config.loops:
-        return [(i, None) for i in range(n)]
-    runs = [(i, None) for i in range(config.loop_start)]
-    for t in range(config.loop_times):
-        runs += [(i, t if i == config.loop_start else None) for i in range(config.loop_start, config.loop_stop)]
-    return runs + [(i, None) for i in range(config.loop_stop, n)]
-
-
 def tarupel_plan(config: TarupelConfig) -> ModelPlan:
     def norm(name: str) -> PartSpec:
         return PartSpec("rms_norm", dict(size=config.width, eps=config.eps, scalar=True), names={"weight": name})
@@ -127,7 +115,8 @@ def tarupel_plan(config: TarupelConfig) -> ModelPlan:
                                 options=dict(hidden_size=config.width, residual_mult=config.residual_mult,
                                              layer_scale=True, token_shift=True), names=names))
     schedule = tuple(ScheduleEntry(layer=i, cache=n, add_offset=t, add_embedding=t is not None and t > 0)
-                     for n, (i, t) in enumerate(layer_runs(config)))
+                     for n, (i, t) in enumerate(looped_runs(len(layers), config.loop_start, config.loop_stop,
+                                                            config.loop_times)))
     return ModelPlan(
         hidden_size=config.width, vocab_size=config.vocab, max_positions=MAX_POSITIONS,
         embedding_name="embed", layers=tuple(layers), schedule=schedule,

@@ -19,9 +19,8 @@ norm's weight + `.norm`; the parallel mixer's two sides are under `.left` and `.
 from __future__ import annotations
 
 from ..config.tolurax import ToluraxConfig
-from ..parts.base import LayerSpec, ModelPlan, PartSpec, ScheduleEntry
+from ..parts.base import LayerSpec, ModelPlan, PartSpec, ScheduleEntry, looped_runs
 from ..registry import register_architecture
-from .tarupel import layer_runs
 
 MAX_POSITIONS = 1 << 20   # the design names no limit
 UNIT_EPS = 1e-6           # under the root of the delta rule's unit vectors
@@ -96,7 +95,8 @@ def tolurax_plan(config: ToluraxConfig) -> ModelPlan:
                                 options=dict(hidden_size=config.width, input_taps=config.canon_taps),
                                 names={"input_conv": p + "canon1"}))
     schedule = tuple(ScheduleEntry(layer=i, cache=n, join_embedding=starts is not None)
-                     for n, (i, starts) in enumerate(layer_runs(config)))
+                     for n, (i, starts) in enumerate(looped_runs(len(layers), config.loop_start, config.loop_stop,
+                                                                 config.loop_times)))
     return ModelPlan(
         hidden_size=config.width, vocab_size=config.vocab, max_positions=MAX_POSITIONS,
         embedding_name="embed", layers=tuple(layers), schedule=schedule,

@@ -122,6 +122,17 @@ class ModelPlan:
     logit_softcap: Optional[float] = None    # logits become cap * tanh(logits / cap) (None: as they are)
 
 
+def looped_runs(layers: int, start: int, stop: int, times: int) -> List[Tuple[int, Optional[int]]]:
+    """[(layer, pass number or None)] in the order layers run when layers start .. stop - 1 run `times` times
+    in a row: the pass number stands at the first layer of each pass (no loop when stop <= start)."""
+    if stop <= start:
+        return [(i, None) for i in range(layers)]
+    runs: List[Tuple[int, Optional[int]]] = [(i, None) for i in range(start)]
+    for t in range(times):
+        runs += [(i, t if i == start else None) for i in range(start, stop)]
+    return runs + [(i, None) for i in range(stop, layers)]
+
+
 # --------------------------------------------------------------------------- cache requests
 @dataclass(frozen=True)
 class KeyValueRequest:

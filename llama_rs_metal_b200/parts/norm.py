@@ -103,7 +103,7 @@ class LayerNorm(Norm):
                               partials=ctx.take_pending())
 
     def forward_conv(self, hidden, ctx, taps, tails):
-        if ctx.phase != "decode" or tails is None:
+        if ctx.phase != "decode" or tails is None or self.size > ops.LAYER_NORM_FOLDS:
             return super().forward_conv(hidden, ctx, taps, tails)
         # one token per sequence: the norm and the convolution behind it are one pass over the rows
         return ops.layer_norm_conv(hidden, self.weight, self.bias, self.eps, ctx.runtime.dtype, taps, tails, ctx.slots,

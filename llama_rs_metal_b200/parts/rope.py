@@ -11,7 +11,7 @@ from ..registry import register_position_encoding
 from .base import PositionEncoding
 
 
-_shared_frequencies = {}  # (device, frequencies) -> float32 tensor on that device
+_shared_frequencies = {}  # (device, frequencies) -> float32 and float64 tensors on that device
 
 @register_position_encoding("rope")
 class RotaryEmbedding(PositionEncoding):
@@ -77,11 +77,10 @@ class RotaryEmbedding(PositionEncoding):
         frequencies = tuple(self.inverse_frequencies())
         key = (str(runtime.device), frequencies)
         if key not in _shared_frequencies:
-            _shared_frequencies[key] = torch.tensor(frequencies, dtype=torch.float64) \
-                .to(torch.float32).to(runtime.device)
-        self.inv_freq = _shared_frequencies[key]
-        # the same in double precision, for kernels that form the angle in double precision
-        self.inv_freq64 = torch.tensor(frequencies, dtype=torch.float64).to(runtime.device)
+            exact = torch.tensor(frequencies, dtype=torch.float64)
+            # beside them in double precision, for kernels that form the angle in double precision
+            _shared_frequencies[key] = (exact.to(torch.float32).to(runtime.device), exact.to(runtime.device))
+        self.inv_freq, self.inv_freq64 = _shared_frequencies[key]
 
     def head_permutation(self) -> Optional[List[int]]:
         if not self.adjacent_pairs:
