@@ -46,30 +46,34 @@ __global__ void head_decay_delta_prepare_kernel(const S* proj, long long stride,
                : unit ? kf + (static_cast<size_t>(t) * G + seg - G) * d
                       : vf + (static_cast<size_t>(t) * H + seg - 2 * G) * dv;
   float* tail = (slot >= 0 && n > 1) ? tails + static_cast<size_t>(slot) * (n - 1) * C : nullptr;
-  float y[PER];
+  float y[PER], now[PER];
+#pragma unroll
+  for (int u = 0; u < PER; ++u) y[u] = 0.f;
+  for (int back = n - 1; back >= 0; --back) {  // oldest input first; a tap's loads are all under way together
+    const int at = local - back;
+    const S* input = at >= 0 ? row + conv_off + first - static_cast<long long>(back) * stride : nullptr;
+    const float* kept = (at < 0 && tail != nullptr) ? tail + static_cast<size_t>(n - 1 + at) * C + first : nullptr;
+    const float* tap = taps + static_cast<size_t>(n - 1 - back) * C + first;
+#pragma unroll
+    for (int u = 0; u < PER; ++u) {
+      const int i = lane + 32 * u;
+      if (i < size) {
+        now[u] = input != nullptr ? to_f32(input[i]) : kept != nullptr ? kept[i] : 0.f;
+        y[u] = fmaf(tap[i], now[u], y[u]);
+      }
+    }
+  }
   float ss = 0.f;
 #pragma unroll
   for (int u = 0; u < PER; ++u) {
     const int i = lane + 32 * u, c = first + i;
-    float acc = 0.f;
-    if (i < size) {
-      for (int back = n - 1; back >= 1; --back) {  // oldest input first
-        const int at = local - back;
-        const float x = at >= 0 ? to_f32(row[conv_off + c - static_cast<long long>(back) * stride])
-                        : tail != nullptr ? tail[static_cast<size_t>(n - 1 + at) * C + c] : 0.f;
-        acc = fmaf(taps[static_cast<size_t>(n - 1 - back) * C + c], x, acc);
-      }
-      const float now = to_f32(row[conv_off + c]);
-      acc = fmaf(taps[static_cast<size_t>(n - 1) * C + c], now, acc);
-      if (one_each && tail != nullptr) {
-        for (int s = 0; s + 1 < n - 1; ++s)
-          tail[static_cast<size_t>(s) * C + c] = tail[static_cast<size_t>(s + 1) * C + c];
-        tail[static_cast<size_t>(n - 2) * C + c] = now;
-      }
-      acc = acc / (1.0f + expf(-acc));
+    if (i < size && one_each && tail != nullptr) {
+      for (int s = 0; s + 1 < n - 1; ++s)
+        tail[static_cast<size_t>(s) * C + c] = tail[static_cast<size_t>(s + 1) * C + c];
+      tail[static_cast<size_t>(n - 2) * C + c] = now[u];  // the last input read is the token's own
     }
-    y[u] = acc;
-    ss = fmaf(acc, acc, ss);
+    y[u] = y[u] / (1.0f + expf(-y[u]));
+    ss = fmaf(y[u], y[u], ss);
   }
   float factor = 1.f;
   if (unit) factor = (seg < G ? q_scale : 1.0f) / sqrtf(warp_sum(ss) + unit_eps);

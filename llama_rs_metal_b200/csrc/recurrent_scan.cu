@@ -6,7 +6,7 @@ int g_scan_rows = 16;
 
 extern "C" int lrm_scan_gated_delta(const float* q, const float* k, const float* v, const float* g, const float* beta,
                                     float* state, float* out, const int* cu_seqlens, const int* slots, int seqs, int H,
-                                    int KH, int d, int dv, cudaStream_t stream);  // recurrent_scan_delta.cu
+                                    int KH, int d, int dv, int tokens, cudaStream_t stream);  // recurrent_scan_delta.cu
 
 namespace {
 
@@ -250,20 +250,20 @@ LRM_API int lrm_linear_state_scan_rows(int rows) {
 LRM_API int lrm_linear_state_scan(const float* q, const float* k, const float* v, const float* g,
                                   const float* head_decay, const float* beta, float* state, float* out,
                                   const int* cu_seqlens, const int* slots, int seqs, int H, int KH, int d,
-                                  int dv, cudaStream_t stream) {
+                                  int dv, int tokens, cudaStream_t stream) {
   if (seqs <= 0) return 0;
   if (H <= 0 || KH <= 0 || H % KH || d <= 0 || dv <= 0 || seqs > 65535 || H > 65535) return LRM_BAD_ARGUMENT;
   if (d > 2048) return LRM_UNSUPPORTED;
   if (g != nullptr) {
     if (beta == nullptr) return LRM_BAD_ARGUMENT;
-    return lrm_scan_gated_delta(q, k, v, g, beta, state, out, cu_seqlens, slots, seqs, H, KH, d, dv, stream);
+    return lrm_scan_gated_delta(q, k, v, g, beta, state, out, cu_seqlens, slots, seqs, H, KH, d, dv, tokens, stream);
   }
   if (head_decay == nullptr) {  // one decay per head and token, where beta would be
     if (beta == nullptr) return LRM_BAD_ARGUMENT;
-    return dispatch_scan<2>(q, k, v, nullptr, nullptr, beta, nullptr, nullptr, state, out, cu_seqlens, slots, seqs, H, KH, d, dv, stream);
+    return dispatch_scan<2>(q, k, v, nullptr, nullptr, beta, nullptr, nullptr, state, out, cu_seqlens, slots, seqs, H, KH, d, dv, stream, Rows{tokens});
   }
   return dispatch_scan<0>(q, k, v, nullptr, head_decay, nullptr, nullptr, nullptr, state, out, cu_seqlens, slots, seqs, H, KH, d,
-                          dv, stream);
+                          dv, stream, Rows{tokens});
 }
 
 // `gate` (type gate_dtype, may be null) is read at gate[t * gate_stride + h * dv + j]; o at

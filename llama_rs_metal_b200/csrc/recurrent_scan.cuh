@@ -310,15 +310,19 @@ __global__ __launch_bounds__(kScanThreads) void linear_scan_kernel(
   }
 }
 
-// How far apart a token's q and k rows, and its v row, are from those of the token before (0: packed).
-struct RowStrides {
+// How far apart a token's q and k rows, and its v row, are from those of the token before (0: packed), and
+// how many tokens the step has.
+struct Rows {
+  int tokens;
   long long q = 0, v = 0;
 };
+
+constexpr int kLongWalk = 16;  // tokens per sequence from which a scan is a long walk
 
 template <int ROWS, int MODE, int PT>
 int launch_scan(const float* q, const float* k, const float* v, const float* g, const float* head_decay,
                 const float* beta, const float* look, const float* put, float* state, float* out, const int* cu_seqlens, const int* slots,
-                int seqs, int H, int KH, int d, int dv, int P, const RowStrides& rows, cudaStream_t stream) {
+                int seqs, int H, int KH, int d, int dv, int P, const Rows& rows, cudaStream_t stream) {
   constexpr int NR = MODE == 3 ? 5 : MODE == 1 || MODE == 4 ? 3 : 2;
   const int COLS = kScanThreads / P, TS = P * (ROWS + 4), VS = (COLS + 3) & ~3;
   int chunk = kChunk;
@@ -338,8 +342,16 @@ int launch_scan(const float* q, const float* k, const float* v, const float* g, 
   const int wide = d % 4 == 0 && dv % 4 == 0 && q_stride % 4 == 0 && v_stride % 4 == 0 && aligned(q) && aligned(k) &&
                    aligned(v) && aligned(g) && (MODE != 3 || (aligned(look) && aligned(put)));
   const dim3 grid((dv + COLS - 1) / COLS, H, seqs);
-  LRM_LAUNCH((linear_scan_kernel<ROWS, MODE, PT>), grid, kScanThreads, bytes, stream, q, k, v, g, head_decay, beta,
-             look, put, state, out, cu_seqlens, slots, H, KH, d, dv, P, chunk, q_stride, v_stride, wide);
+  // A long walk is bound by its tokens' latency and wants an SM to itself. Let in while the kernel before
+  // still runs, its CTAs pile up on the SMs that kernel leaves first (one prompt of 2,048 tokens: 800
+  // us in the middle of a step against 260 alone), so it starts when that kernel is done.
+  const int pdl = g_lrm_pdl;
+  if (rows.tokens >= static_cast<long long>(seqs) * kLongWalk) g_lrm_pdl = 0;
+  const cudaError_t launched = lrm_launch(linear_scan_kernel<ROWS, MODE, PT>, grid, kScanThreads, bytes, stream, q, k, v, g,
+                                          head_decay, beta, look, put, state, out, cu_seqlens, slots, H, KH, d, dv, P,
+                                          chunk, q_stride, v_stride, wide);
+  g_lrm_pdl = pdl;
+  if (launched != cudaSuccess) return static_cast<int>(launched);
   return 0;
 }
 
@@ -358,7 +370,7 @@ inline void scan_shape(int d, int* rows, int* parts, int most_rows) {
 template <int MODE>
 int dispatch_scan(const float* q, const float* k, const float* v, const float* g, const float* head_decay,
                   const float* beta, const float* look, const float* put, float* state, float* out, const int* cu_seqlens, const int* slots,
-                  int seqs, int H, int KH, int d, int dv, cudaStream_t stream, const RowStrides& rows = RowStrides{}) {
+                  int seqs, int H, int KH, int d, int dv, cudaStream_t stream, const Rows& rows) {
   int R, P;
   scan_shape(d, &R, &P, g_scan_rows);
   if (g_scan_rows > 8) {

@@ -884,7 +884,7 @@ def linear_state_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: 
             raise InvalidError("linear_state_scan: one decay per head")
     out = _f32((T, H, dv), q.device)
     _done(_lib().lrm_linear_state_scan(_ptr(q), _ptr(k), _ptr(v), _ptr(g), _ptr(head_decay), _ptr(beta), _ptr(state),
-                                       _ptr(out), _ptr(cu_seqlens), _ptr(slots), slots.numel(), H, KH, d, dv,
+                                       _ptr(out), _ptr(cu_seqlens), _ptr(slots), slots.numel(), H, KH, d, dv, T,
                                        _stream()), "linear_state_scan")
     return out
 
@@ -935,7 +935,7 @@ def general_delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: tor
         raise InvalidError("general_delta_scan: shapes do not agree")
     out = _f32((T, H, dv), q.device)
     _done(_lib().lrm_general_delta_scan(_ptr(q), _ptr(k), _ptr(v), _ptr(g), _ptr(look), _ptr(put), _ptr(state),
-                                        _ptr(out), _ptr(cu_seqlens), _ptr(slots), slots.numel(), H, d, dv, _stream()),
+                                        _ptr(out), _ptr(cu_seqlens), _ptr(slots), slots.numel(), H, d, dv, T, _stream()),
           "general_delta_scan")
     return out
 
@@ -964,7 +964,7 @@ def bonus_state_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, g: 
     out = _f32((T, H, value_dim), proj.device)
     _done(_lib().lrm_bonus_state_scan(_column_ptr(proj, q_off), _column_ptr(proj, k_off), ctypes.c_longlong(W),
                                       _column_ptr(proj, v_off), ctypes.c_longlong(W), _ptr(g), _ptr(bonus), _ptr(state),
-                                      _ptr(out), _ptr(cu_seqlens), _ptr(slots), slots.numel(), H, d, value_dim,
+                                      _ptr(out), _ptr(cu_seqlens), _ptr(slots), slots.numel(), H, d, value_dim, T,
                                       _stream()), "bonus_state_scan")
     return out
 
@@ -983,7 +983,7 @@ def head_decay_delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, dec
         raise InvalidError("head_decay_delta_scan: shapes do not agree")
     out = _f32((T, H, dv), q.device)
     _done(_lib().lrm_head_decay_delta_scan(_ptr(q), _ptr(k), _ptr(v), _ptr(decay), _ptr(step), _ptr(state), _ptr(out),
-                                           _ptr(cu_seqlens), _ptr(slots), slots.numel(), H, KH, d, dv, _stream()),
+                                           _ptr(cu_seqlens), _ptr(slots), slots.numel(), H, KH, d, dv, T, _stream()),
           "head_decay_delta_scan")
     return out
 
