@@ -412,6 +412,112 @@ def make_tarupel_dir(path, name, dtype=torch.bfloat16, edit=None, steady_routing
     return write_model_folder(path, config.to_dict(), tensors, spec["seed"])
 
 
+def _rotation(dims, base, scaling=None):
+    out = dict(dims=dims, base=base)
+    if scaling is not None:
+        out["scaling"] = dict(zip(("factor", "low", "high", "original"), scaling))
+    return out
+
+
+def _sigmoid_side(heads, kv_heads, dim, vdim, scale, window, rot=None):
+    out = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, scale=scale)
+    if window is not None:
+        out["mask"] = dict(size=window)
+    if rot is not None:
+        out["rot"] = rot
+    return out
+
+
+def _parallel(left, heads, dim, rank, left_scale, right_scale):
+    return dict(left=left, left_scale=left_scale, right=dict(heads=heads, dim=dim, decay_rank=rank), right_scale=right_scale)
+
+
+def _head_delta(heads, kv_heads, dim, vdim, conv):
+    return dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, conv=conv)
+
+
+# Three tiny Tolurax configurations. Between them: sizes that are multiples of nothing and sizes that take
+# the tensor-core products and the tiled attention kernels (X2: head sizes 64, 96 and 128); key heads fewer
+# than, and as many as, query heads; values wider and narrower than keys; windows of one token, shorter than
+# a page, of one page, and longer; rotation of a part of the head, of all of it, and none, with frequencies
+# kept, stretched and blended; one tap and several in both convolutions; delta layers with and parallel
+# layers without a feed-forward; a loop in the middle, from the first layer, and none; no soft cap.
+TOLURAX = {
+    "X1": dict(
+        config=dict(architecture="Tolurax", vocab=211, width=72, norm=dict(eps=1e-6), canon=dict(taps=4), logit_softcap=6.0,
+                    loop=dict(start=1, stop=3, times=2), layers=[
+            dict(type="delta", mixer=_head_delta(4, 2, 20, 12, 2), mlp=dict(kind="dense", ff=56)),
+            dict(type="parallel", mixer=_parallel(_sigmoid_side(4, 2, 12, 20, 0.4, 7, _rotation(6, 50.0, (8.0, 1.0, 4.0, 64.0))),
+                                                  3, 10, 5, 0.7, 1.2), mlp=None),
+            dict(type="delta", mixer=_head_delta(3, 3, 10, 24, 5), mlp=None),
+            dict(type="parallel", mixer=_parallel(_sigmoid_side(3, 1, 10, 6, 0.3, 70, _rotation(10, 100.0)), 2, 36, 3, 1.1, 0.6),
+                 mlp=dict(kind="dense", ff=40)),
+        ]), seed=61, std=0.12),
+    "X2": dict(
+        config=dict(architecture="Tolurax", vocab=512, width=192, norm=dict(eps=2e-5), canon=dict(taps=2), logit_softcap=9.0,
+                    loop=dict(start=0, stop=2, times=3), layers=[
+            dict(type="parallel", mixer=_parallel(_sigmoid_side(4, 2, 64, 64, 0.11, 64, _rotation(32, 10000.0, (4.0, 1.0, 2.0, 100.0))),
+                                                  2, 64, 8, 0.6, 0.9), mlp=dict(kind="dense", ff=448)),
+            dict(type="delta", mixer=_head_delta(4, 1, 64, 32, 4), mlp=dict(kind="dense", ff=256)),
+            dict(type="parallel", mixer=_parallel(_sigmoid_side(2, 1, 96, 96, 0.1, 100, _rotation(96, 500000.0, (8.0, 2.0, 8.0, 512.0))),
+                                                  3, 32, 16, 1.0, 0.5), mlp=None),
+            dict(type="parallel", mixer=_parallel(_sigmoid_side(20, 1, 128, 128, 0.08, 40, _rotation(64, 1000.0)), 1, 128, 4, 0.4, 0.7),
+                 mlp=dict(kind="dense", ff=128)),
+        ]), seed=62, std=0.06),
+    "X3": dict(
+        config=dict(architecture="Tolurax", vocab=300, width=64, norm=dict(eps=1e-5), canon=dict(taps=1), layers=[
+            dict(type="parallel", mixer=_parallel(_sigmoid_side(2, 2, 16, 24, 0.3, 1), 1, 16, 2, 1.0, 1.0), mlp=dict(kind="dense", ff=40)),
+            dict(type="delta", mixer=_head_delta(1, 1, 8, 8, 1), mlp=None),
+            dict(type="parallel", mixer=_parallel(_sigmoid_side(1, 1, 8, 8, 0.5, None, _rotation(2, 30.0)), 2, 8, 1, 0.5, 0.25), mlp=None),
+        ]), seed=63, std=0.15),
+}
+
+
+def make_tolurax_dir(path, name, dtype=torch.bfloat16, edit=None):
+    """A model folder of a tiny Tolurax configuration (a name of TOLURAX, or a spec of the caller's own) with
+    seeded random weights; `edit` (a function of the name -> tensor dict) may change them before they are
+    written. Norm weights are N(1, 0.2), score offsets N(-1, 1), the token mixes uniform in [0, 1], the time
+    mix's decay bias N(-2, 2) and the delta rule's A_log N(-2, 1): some channels and heads forget within a
+    few tokens, others carry their state over hundreds; the matrix ahead of a loop's passes is half the
+    identity on the stream plus the embedding, with noise, so that passes neither die out nor blow up."""
+    from llama_rs_metal_b200.engine.model import DecoderModel
+    from llama_rs_metal_b200.registry import find_architecture
+    from llama_rs_metal_b200.runtime import Runtime
+    from llama_rs_metal_b200.weights.random_init import _generator, random_tensors, write_model_folder
+    spec = TOLURAX[name] if isinstance(name, str) else name
+    arch = find_architecture(spec["config"])
+    config = arch.config_class.from_dict(spec["config"])
+    model = DecoderModel(arch.plan(config), Runtime(torch.device("cpu"), torch.float32))
+    tensors = random_tensors(model.tensor_specs(), spec["seed"], std=spec["std"], vector_mean=0.0, vector_std=0.5,
+                             dtype=dtype)
+    for name_, t in tensors.items():
+        last = name_.rsplit(".", 1)[-1]
+        if last in ("norm", "norm1", "norm2"):
+            t.mul_(0.4).add_(1.0)
+        elif last == "pb":
+            t.mul_(2.0).sub_(1.0)
+        elif ".mu." in name_:
+            t.copy_(torch.rand(t.shape, generator=_generator(spec["seed"], name_), dtype=torch.float32))
+        elif last == "w0":
+            t.mul_(4.0).sub_(2.0)
+        elif last == "A_log":
+            t.mul_(2.0).sub_(2.0)
+        elif last in ("conv", "canon1"):
+            t.mul_(0.3 / spec["std"])
+        elif last == "u":
+            t.mul_(0.5 / spec["std"])
+        elif name_ == "embed":
+            t.mul_(1.0 / spec["std"])
+        elif name_ == "loop.in":
+            n = t.shape[0]
+            t.mul_(0.3)
+            t[:, :n] += 0.5 * torch.eye(n, dtype=t.dtype)
+            t[:, n:] += torch.eye(n, dtype=t.dtype)
+    if edit is not None:
+        edit(tensors)
+    return write_model_folder(path, config.to_dict(), tensors, spec["seed"])
+
+
 def random_tokens(seed, length, vocab):
     rng = np.random.default_rng(seed)
     return [int(t) for t in rng.integers(0, vocab, size=length)]
