@@ -135,7 +135,7 @@ def test_cache_requests_keep_what_each_layer_needs():
 
 
 def test_stretched_frequencies_agree_with_the_position_encoding():
-    for rot in (helpers._rotation(32, 10000.0, (4.0, 1.0, 2.0, 100.0)), helpers._rotation(96, 20000.0, (8.0, 1.0, 4.0, 512.0)),
+    for rot in (helpers._rotation(32, 10000.0, (4.0, 1.0, 2.0, 100.0)), helpers._rotation(80, 30000.0, (6.0, 1.5, 5.0, 512.0)),
                 helpers._rotation(6, 50.0)):
         s = rot.get("scaling")
         params = dict(scaling="llama3", factor=s["factor"], low_freq_factor=s["low"], high_freq_factor=s["high"],
