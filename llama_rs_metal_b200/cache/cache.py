@@ -5,7 +5,8 @@
   - a key/value group keeps, per layer, pages [page][kv_head][page_size][head_dim]
     for keys and the same for values; every sequence has a row in the group's page
     table mapping position // page_size to a page. A group with a window keeps only
-    the pages that still hold positions inside the window and returns the others;
+    the pages that still hold positions inside the window (and those of the first tokens,
+    where its layers keep some) and returns the others;
   - a state group keeps, per layer, one fixed-size tensor per slot, zeroed when the
     slot is taken. Llama has none; the storage exists for mixers that do.
 * A mixer that keeps several things (a CompositeRequest: keys and values beside a state, two
@@ -74,8 +75,13 @@ class KeyValueGroup:
         self.v = self.k if request.values_in_keys else \
             {e: torch.zeros(value_shape, dtype=dtype, device=device) for e in entries}
 
+    @property
+    def always_kept(self) -> int:
+        """Logical pages 0 .. this - 1 hold the first tokens a windowed group keeps beside its window."""
+        return -(-self.request.keep_first // self.page_size) if self.request.window is not None else 0
+
     def first_kept_page(self, length: int) -> int:
-        """Lowest logical page a sequence of `length` tokens still needs."""
+        """Lowest logical page a sequence of `length` tokens still needs (beside the first ones it always keeps)."""
         if self.request.window is None:
             return 0
         return max(0, length - self.request.window) // self.page_size
@@ -97,22 +103,23 @@ class KeyValueGroup:
         row = self.table_host[slot]
         last = (new_length - 1) // self.page_size
         first = self.first_needed_page(new_length, reads_from)
+        head = min(self.always_kept, first)
         if last >= len(row):
-            return last + 1 - first  # more than the table can name: more than any pool holds
-        return int(np.count_nonzero(row[first:last + 1] < 0))
+            return last + 1 - first + head  # more than the table can name: more than any pool holds
+        return int(np.count_nonzero(row[first:last + 1] < 0)) + int(np.count_nonzero(row[:head] < 0))
 
     def pages_released(self, slot: int, new_length: int, reads_from: Optional[int] = None) -> int:
         first = self.first_needed_page(new_length, reads_from)
-        return int(np.count_nonzero(self.table_host[slot][:first] >= 0))
+        return int(np.count_nonzero(self.table_host[slot][self.always_kept:first] >= 0))
 
     def release_stale(self, slot: int, new_length: int, reads_from: Optional[int] = None) -> None:
         """Return the pages that lie wholly before what a step to `new_length` still needs."""
         row = self.table_host[slot]
         first = self.first_needed_page(new_length, reads_from)
-        stale = [int(p) for p in row[:first] if p >= 0]
+        stale = [int(p) for p in row[self.always_kept:first] if p >= 0]
         if stale:
             self.pool.give_back(stale)
-            row[:first] = -1
+            row[self.always_kept:first] = -1
             self.dirty = True
 
     def take_missing(self, slot: int, new_length: int, reads_from: Optional[int] = None) -> None:
@@ -121,7 +128,7 @@ class KeyValueGroup:
         row = self.table_host[slot]
         first = self.first_needed_page(new_length, reads_from)
         last = (new_length - 1) // self.page_size
-        missing = [i for i in range(first, last + 1) if row[i] < 0]
+        missing = [i for i in (*range(min(self.always_kept, first)), *range(first, last + 1)) if row[i] < 0]
         if missing:
             for i, page in zip(missing, self.pool.take(len(missing))):
                 row[i] = page
@@ -306,9 +313,11 @@ class Cache:
             if group.request.window is not None:
                 # Pages below the first one the new token still sees. Pages leave a window lowest
                 # first, so a sequence holds stale pages exactly when it holds the one right below.
+                # (The pages of kept first tokens never leave.)
+                head = group.always_kept
                 first = np.maximum(0, before + 1 - group.request.window) // ps
-                leaving = np.nonzero((first > 0) & (group.table_host[slots, np.maximum(first - 1, 0)] >= 0))[0]
-            freed = sum(int(np.count_nonzero(group.table_host[slots[i], :first[i]] >= 0)) for i in leaving)
+                leaving = np.nonzero((first > head) & (group.table_host[slots, np.maximum(first - 1, 0)] >= 0))[0]
+            freed = sum(int(np.count_nonzero(group.table_host[slots[i], head:first[i]] >= 0)) for i in leaving)
             stale.append(leaving)
             if len(lacking) > group.pool.available + freed:
                 raise CacheMemoryError(f"step needs {len(lacking)} pages of {ps} tokens, "

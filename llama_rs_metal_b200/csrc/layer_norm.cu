@@ -5,7 +5,8 @@
 //
 // lrm_layer_norm: rows of the residual stream (all, or those `rows` names) -> activations. `partials`:
 // float32 [n, T, h] slices of a product that are first added, in slice order, into the row, which is
-// written back (a gathered row is not); rows of up to 8192 elements.
+// written back (a gathered row is not); rows of up to 8192 elements. `add`: float32 [h], added to every row of the
+// stream once the row that is normalized has been read (the bias of an output that joins the stream later).
 // lrm_layer_norm_conv: the same for a step of one token per sequence, and in the same pass the
 // causal convolution over time in front of a mixer: h + sum_j taps[j] * (the h of n - 1 - j tokens
 // ago), with the older rows from the sequence's tail [n - 1, h], which is moved on by one row.
@@ -123,7 +124,7 @@ __device__ __forceinline__ void normalize(float (&v)[PER], int hidden, float eps
 template <typename O, int PER, int VEC>
 __global__ __launch_bounds__(1024) void layer_norm_kernel(float* x, const float* __restrict__ w, const float* __restrict__ b, O* out,
                                   const int* rows, const float* partials, int n_partials, size_t partial_stride,
-                                  int hidden, float eps) {
+                                  const float* __restrict__ add, int hidden, float eps) {
   __shared__ float scratch[32];
   constexpr bool EARLY = PER <= 8;
   constexpr int KEPT = EARLY ? PER : VEC;
@@ -136,7 +137,16 @@ __global__ __launch_bounds__(1024) void layer_norm_kernel(float* x, const float*
   pdl_wait();
   const size_t src = static_cast<size_t>(rows != nullptr ? rows[blockIdx.x] : blockIdx.x) * hidden;
   float v[PER];
-  load_row<PER, VEC>(v, x, src, hidden, partials, n_partials, partial_stride, rows == nullptr);
+  load_row<PER, VEC>(v, x, src, hidden, partials, n_partials, partial_stride, rows == nullptr && add == nullptr);
+  if constexpr (EARLY) {
+    if (add != nullptr) {
+      float moved[PER];
+      read_row<PER, VEC>(moved, add, hidden);
+#pragma unroll
+      for (int e = 0; e < PER; ++e) moved[e] += v[e];
+      write_row<PER, VEC>(moved, x + src, hidden);
+    }
+  }
   normalize<PER, VEC>(v, hidden, eps, scratch);
 #pragma unroll
   for (int e = 0; e < PER; ++e) {
@@ -357,25 +367,26 @@ bool fours(int hidden, long long partial_stride, const void* x, const void* w, c
 }  // namespace
 
 // x float32 [*, hidden]; w float32 [hidden], b likewise or null; rows int32 [n_rows] or null (row r of
-// out is row r of x); partials float32, n_partials planes partial_stride apart, or null.
+// out is row r of x); partials float32, n_partials planes partial_stride apart, or null; add float32
+// [hidden] or null (not with rows).
 LRM_API int lrm_layer_norm(float* x, const float* w, const float* b, void* out, int out_dtype, const int* rows,
                            int n_rows, int hidden, float eps, const float* partials, int n_partials,
-                           long long partial_stride, cudaStream_t stream) {
+                           long long partial_stride, const float* add, cudaStream_t stream) {
   if (n_rows <= 0) return 0;
   if (hidden <= 0 || !(eps > 0.f) || x == nullptr || w == nullptr || out == nullptr ||
-      n_partials < 0 || (n_partials > 0 && partials == nullptr))
+      n_partials < 0 || (n_partials > 0 && partials == nullptr) || (add != nullptr && rows != nullptr))
     return LRM_BAD_ARGUMENT;
   const int threads = row_threads(hidden), per = (hidden + threads - 1) / threads;
-  if (per > 8 && n_partials > 0) return LRM_UNSUPPORTED;
-  const bool four = fours(hidden, partial_stride, x, w, b, out, partials);
+  if (per > 8 && (n_partials > 0 || add != nullptr)) return LRM_UNSUPPORTED;
+  const bool four = fours(hidden, partial_stride, x, w, b, out, partials) && reinterpret_cast<uintptr_t>(add) % 16 == 0;
 #define LRM_LAYER_NORM(OT, PER)                                                                                   \
   do {                                                                                                            \
     if (four)                                                                                                     \
       LRM_LAUNCH((layer_norm_kernel<OT, PER, 4>), n_rows, threads, 0, stream, x, w, b, static_cast<OT*>(out), rows, \
-                 partials, n_partials, static_cast<size_t>(partial_stride), hidden, eps);                         \
+                 partials, n_partials, static_cast<size_t>(partial_stride), add, hidden, eps);                    \
     else                                                                                                          \
       LRM_LAUNCH((layer_norm_kernel<OT, PER, 1>), n_rows, threads, 0, stream, x, w, b, static_cast<OT*>(out), rows, \
-                 partials, n_partials, static_cast<size_t>(partial_stride), hidden, eps);                         \
+                 partials, n_partials, static_cast<size_t>(partial_stride), add, hidden, eps);                    \
     return 0;                                                                                                     \
   } while (0)
   if (out_dtype == LRM_F32) {

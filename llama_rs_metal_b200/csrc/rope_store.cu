@@ -248,26 +248,27 @@ LRM_API int lrm_rope_table(const int* positions, const float* inv_freq, float* t
   return 0;
 }
 
-// The same with the angle formed in double precision from frequencies in double precision.
+// The same with the angle formed in double precision from frequencies in double precision, cosines and sines
+// multiplied by `magnitude`.
 __global__ void rope_table64_kernel(const int* __restrict__ positions, const double* __restrict__ inv_freq,
-                                    float2* __restrict__ table, int tokens, int half) {
+                                    float2* __restrict__ table, int tokens, int half, double magnitude) {
   pdl_trigger();
   const int item = blockIdx.x * blockDim.x + threadIdx.x;
   float2 entry = make_float2(0.f, 0.f);
   if (item < tokens * half) {
     double sn, cs;
     sincos(static_cast<double>(positions[item / half]) * inv_freq[item % half], &sn, &cs);
-    entry = make_float2(static_cast<float>(cs), static_cast<float>(sn));
+    entry = make_float2(static_cast<float>(cs * magnitude), static_cast<float>(sn * magnitude));
   }
   pdl_wait();  // the table's memory may have been another kernel's
   if (item < tokens * half) table[item] = entry;
 }
 
 LRM_API int lrm_rope_table64(const int* positions, const double* inv_freq, float* table, int tokens, int half,
-                             cudaStream_t stream) {
+                             double magnitude, cudaStream_t stream) {
   if (tokens <= 0 || half <= 0) return 0;
   if (positions == nullptr || inv_freq == nullptr || table == nullptr || tokens > 0x7fffffff / half) return LRM_BAD_ARGUMENT;
   LRM_LAUNCH(rope_table64_kernel, dim3((tokens * half + 127) / 128), 128, 0, stream, positions, inv_freq,
-             reinterpret_cast<float2*>(table), tokens, half);
+             reinterpret_cast<float2*>(table), tokens, half, magnitude);
   return 0;
 }

@@ -13,7 +13,8 @@
 //   5. a rotation by position of the first `rotary` dimensions of every query and key head,
 //      dimension i paired with i + rotary/2 (pairing 0) or 2i with 2i + 1 (pairing 1), angle =
 //      position * inv_freq[i] formed in double precision, here or, for layers that share their
-//      frequencies, once per step in a table of cosines and sines (lrm_rope_table64);
+//      frequencies, once per step in a table of cosines and sines (lrm_rope_table64); `magnitude`
+//      multiplies cosines and sines (a table holds it already);
 //   6. the division of every query and key head by its root mean square (no weight),
 // and writes q, k, v in the activation type: q packed, k and v packed (when asked for) and into
 // the paged cache at dest_rows[t] (see qkv_store.cu for the layout). Everything between the
@@ -34,7 +35,7 @@ __global__ void shaped_qkv_kernel(const S* proj, long long stride, const float* 
                                   const int* __restrict__ positions, const float* __restrict__ q_norm,
                                   const float* __restrict__ k_norm, float row_eps,
                                   const float* __restrict__ q_head_w, const float* __restrict__ k_head_w,
-                                  float head_w_eps, const double* __restrict__ inv_freq, const float2* table,
+                                  float head_w_eps, const double* __restrict__ inv_freq, double magnitude, const float2* table,
                                   int rotary, int pairing, int head_norm,
                                   float head_eps, A* __restrict__ q_out, A* __restrict__ k_out,
                                   A* __restrict__ v_out, A* __restrict__ k_pages, A* __restrict__ v_pages,
@@ -53,8 +54,8 @@ __global__ void shaped_qkv_kernel(const S* proj, long long stride, const float* 
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
       double sn, c;
       sincos(static_cast<double>(pos) * inv_freq[i], &sn, &c);
-      cs[i] = static_cast<float>(c);
-      cs[half + i] = static_cast<float>(sn);
+      cs[i] = static_cast<float>(c * magnitude);
+      cs[half + i] = static_cast<float>(sn * magnitude);
     }
   pdl_wait();
   if (table != nullptr)
@@ -182,7 +183,7 @@ template <typename S, typename A, int VEC>
 __global__ void shaped_heads_kernel(const S* proj, long long stride, const float* __restrict__ bias,
                                     const int* __restrict__ positions, const float* __restrict__ q_head_w,
                                     const float* __restrict__ k_head_w, float head_w_eps,
-                                    const double* __restrict__ inv_freq, const float2* table, int rotary, int pairing,
+                                    const double* __restrict__ inv_freq, double magnitude, const float2* table, int rotary, int pairing,
                                     A* __restrict__ q_out, A* __restrict__ k_out, A* __restrict__ v_out,
                                     A* __restrict__ k_pages, A* __restrict__ v_pages,
                                     const int* __restrict__ dest_rows, int q_heads, int kv_heads, int d, int dv,
@@ -197,8 +198,8 @@ __global__ void shaped_heads_kernel(const S* proj, long long stride, const float
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
       double sn, c;
       sincos(static_cast<double>(pos) * inv_freq[i], &sn, &c);
-      cs[i] = static_cast<float>(c);
-      cs[half + i] = static_cast<float>(sn);
+      cs[i] = static_cast<float>(c * magnitude);
+      cs[half + i] = static_cast<float>(sn * magnitude);
     }
     __syncthreads();
   }
@@ -282,7 +283,7 @@ LRM_API int lrm_shaped_qkv_store(const void* proj, int in_dtype, long long strid
                                  const float* tails, const int* cu_seqlens, const int* seq_of_token,
                                  const int* slots, const int* positions, const float* q_norm, const float* k_norm,
                                  float row_eps, const float* q_head_w, const float* k_head_w, float head_w_eps,
-                                 const double* inv_freq, const float* table, int rotary, int pairing, int head_norm,
+                                 const double* inv_freq, double magnitude, const float* table, int rotary, int pairing, int head_norm,
                                  float head_eps, void* q_out, void* k_out, void* v_out, void* k_pages, void* v_pages,
                                  const int* dest_rows, int out_dtype, int tokens, int q_heads, int kv_heads, int d,
                                  int dv, int page_size, cudaStream_t stream) {
@@ -309,7 +310,7 @@ LRM_API int lrm_shaped_qkv_store(const void* proj, int in_dtype, long long strid
     const bool pairs = d % 2 == 0 && dv % 2 == 0 && stride % 2 == 0 && reinterpret_cast<uintptr_t>(proj) % in_pair == 0;
 #define LRM_HEADS(ST, AT, V)                                                                                        \
   LRM_LAUNCH((shaped_heads_kernel<ST, AT, V>), grid, threads, sizeof(float) * rotary, stream, static_cast<const ST*>(proj), \
-             stride, bias, positions, q_head_w, k_head_w, head_w_eps, inv_freq, turns, rotary, pairing, static_cast<AT*>(q_out), \
+             stride, bias, positions, q_head_w, k_head_w, head_w_eps, inv_freq, magnitude, turns, rotary, pairing, static_cast<AT*>(q_out), \
              static_cast<AT*>(k_out), static_cast<AT*>(v_out), static_cast<AT*>(k_pages), static_cast<AT*>(v_pages), \
              dest_rows, q_heads, kv_heads, d, dv, page_size)
     if (in_dtype == LRM_F32 && out_dtype == LRM_F32) {
@@ -336,7 +337,7 @@ LRM_API int lrm_shaped_qkv_store(const void* proj, int in_dtype, long long strid
       raised = true;                                                                                            \
     }                                                                                                           \
     LRM_LAUNCH((shaped_qkv_kernel<ST, AT>), tokens, width >= 2048 ? 512 : 256, bytes, stream, static_cast<const ST*>(proj), stride, bias, taps, n, \
-               tails, cu_seqlens, seq_of_token, slots, positions, q_norm, k_norm, row_eps, q_head_w, k_head_w, head_w_eps, inv_freq, turns, rotary, \
+               tails, cu_seqlens, seq_of_token, slots, positions, q_norm, k_norm, row_eps, q_head_w, k_head_w, head_w_eps, inv_freq, magnitude, turns, rotary, \
                pairing, head_norm, head_eps, static_cast<AT*>(q_out), static_cast<AT*>(k_out),                  \
                static_cast<AT*>(v_out), static_cast<AT*>(k_pages), static_cast<AT*>(v_pages), dest_rows, q_heads, \
                kv_heads, d, dv, page_size);                                                                     \

@@ -13,6 +13,9 @@ extend kernel in bfloat16). bfloat16 attention over one key head whose rows also
 values (latent attention's cache) runs csrc/attention_shared_keys.cu in every phase.
 Attention without a softmax (a key's weight is the sigmoid of its score) has kernels of its own in
 csrc/attention_sigmoid.cu: tiled in bfloat16 for head sizes 32, 64, 96 and 128, row-wise otherwise.
+Softmax attention with a cap on its scores, kept first keys or an output gate (and then also with sinks and
+values of another width) runs csrc/attention_gated.cu: tiled in bfloat16 for head sizes that are multiples of
+8 up to 128, row-wise otherwise.
 
 `attend` is the one call a mixer makes: it takes the step's projection and picks
 rotation, cache write and attention kernels for the step's phase and geometry.
@@ -36,6 +39,7 @@ force_unfused_decode = False  # tests keep decode steps on the separate rotation
 force_cluster_size = None  # tests fix the CTAs per cluster of the fused decode kernel
 force_shared_key_splits = None  # tests fix the splits of the shared-key kernel's decode step
 force_sigmoid_ranks = None  # tests fix the CTAs per cluster of the sigmoid decode kernel
+force_gated_ranks = None  # tests fix the CTAs per cluster of the gated softmax kernel's decode step
 prefill_kernel = None  # tests pin the tcgen05 prompt kernel: "pingpong" or "single" (None: the rule in prefill())
 
 
@@ -75,8 +79,8 @@ class Shaping:
     row_norm: (q weight, k weight), an RMS norm over all query columns and one over all key columns
         (eps `row_eps`).
     inv_freq, rotary, adjacent_pairs: a rotation of each head's first `rotary` dimensions, angle =
-        position * inv_freq[i] (float64 [rotary / 2]); dimension i pairs with i + rotary / 2, or 2i
-        with 2i + 1.
+        position * inv_freq[i] (float64 [rotary / 2]), cosines and sines times `magnitude`; dimension i
+        pairs with i + rotary / 2, or 2i with 2i + 1.
     head_weights: (q weight, k weight), an RMS norm over every query and every key head ahead of the
         rotation, one weight of the head size each (eps `head_weight_eps`).
     head_norm_eps: each query and key head is divided by its root mean square afterwards.
@@ -89,6 +93,7 @@ class Shaping:
     head_weights: Optional[tuple] = None
     head_weight_eps: float = 0.0
     inv_freq: Optional[torch.Tensor] = None
+    magnitude: float = 1.0
     rotary: int = 0
     adjacent_pairs: bool = False
     head_norm_eps: Optional[float] = None
@@ -324,6 +329,41 @@ def sigmoid(q, k, v, kv, kv_heads: int, dv: int, out, out_stride: int, offset, g
                                             kv_heads, d, dv, page_size, *tail, _stream()), "attention_sigmoid_rowwise")
 
 
+def gated(q, k, v, kv, kv_heads: int, dv: int, out, out_stride: int, form, gate, gate_stride: int, scale: float,
+          window: int, out_scale: float, max_seq_len: int, max_kv_len: int, cu_seqlens, seq_of_token, positions, slots,
+          kv_lens) -> None:
+    """Softmax attention of an ops.SoftmaxForm (csrc/attention_gated.cu): packed keys k, v, or the cache view
+    kv (one query per sequence where cu_seqlens is None). `out` and `gate` are pointers at first columns."""
+    T, Hq, d = q.shape
+    lib = library.load()
+    paged = kv is not None
+    one_each = paged and cu_seqlens is None
+    keys, values = (kv.k, kv.v) if paged else (k, v)
+    page_size = kv.page_size if paged else 64
+    pages = (_ptr(kv.page_table), kv.page_table.shape[1], _ptr(slots), _ptr(kv_lens)) if paged else (None, 0, None, None)
+    tail = (ctypes.c_float(scale), ctypes.c_float(form.cap or 0.0), window, form.keep_first, _ptr(form.sinks), gate,
+            ctypes.c_longlong(gate_stride), int(form.gate_per_head), out, ctypes.c_longlong(out_stride),
+            ctypes.c_float(out_scale))
+    if (not force_rowwise and q.dtype == torch.bfloat16 and lib.lrm_attention_gated_supports(d, dv, page_size)
+            and out_stride % 2 == 0 and all(t.data_ptr() % 16 == 0 for t in (q, keys, values)) and out.value % 4 == 0):
+        ranks = 0
+        if one_each:
+            # the CTAs of a cluster share a sequence's pages; about two CTAs per SM, no CTA without a page
+            seen = min(max_kv_len, abs(window) + 63 + form.keep_first) if window else max_kv_len
+            clusters = T * kv_heads * -(-(Hq // kv_heads) // 16)
+            ranks = max(1, min(8, -(-seen // 64), -(-2 * SM_COUNT // clusters)))
+            if force_gated_ranks is not None:
+                ranks = force_gated_ranks
+        _done(lib.lrm_attention_gated(_ptr(q), _ptr(keys), _ptr(values), _ptr(None if one_each else cu_seqlens), *pages,
+                                      T if one_each else cu_seqlens.numel() - 1, max_seq_len, Hq, kv_heads, d, dv, *tail,
+                                      ranks, _stream()), "attention_gated_decode" if one_each else "attention_gated")
+        return
+    _done(lib.lrm_attention_gated_rowwise(_ptr(q), _ptr(keys), _ptr(values), _code(q.dtype), _ptr(cu_seqlens),
+                                          _ptr(None if one_each else seq_of_token),
+                                          _ptr(None if one_each or not paged else positions), *pages, T, Hq, kv_heads, d,
+                                          dv, page_size, *tail, _stream()), "attention_gated_rowwise")
+
+
 _cluster_room = {}
 
 
@@ -413,7 +453,7 @@ def decode_fused(qkv, positions, inv_freq, rotary: int, kv, dest_rows, out, slot
 def attend(projected, *, q_heads: int, kv_heads: int, head_dim: int, rotary, ctx, cache, writes_cache: bool,
            cache_entry: int, scale: float, window, projection=None, value_dim=None, bias=None, slopes=None,
            out_scale: float = 1.0, extras=None, values_are_keys: bool = False, shaping: Optional[Shaping] = None,
-           chunk: Optional[int] = None, sigmoid_weights=None):
+           chunk: Optional[int] = None, sigmoid_weights=None, form=None):
     """A layer's attention for one step: position rotation, cache write and attention, with the
     kernels chosen here for the step's phase, dtype and geometry. -> mixed heads [T, q_heads * d].
 
@@ -436,7 +476,7 @@ def attend(projected, *, q_heads: int, kv_heads: int, head_dim: int, rotary, ctx
         counted from position 0, and a query sees only the keys of its own chunk (`window` is then
         what the cache keeps, and the kernels are told the chunk as a negative window).
     sigmoid_weights: an ops.SigmoidWeights (with a `shaping`): no softmax, see there; the result may then
-        go to columns of a tensor it names.
+        go to columns of a tensor it names. form: an ops.SoftmaxForm (with a `shaping`), likewise.
     """
     from . import ops
     inv_freq, width = rotary if rotary is not None else (None, 0)
@@ -462,17 +502,17 @@ def attend(projected, *, q_heads: int, kv_heads: int, head_dim: int, rotary, ctx
             s = shaping
             table = None
             if s.inv_freq is not None:  # one table of angles per step and set of frequencies
-                key = ("rope_table64", s.inv_freq.data_ptr())
+                key = ("rope_table64", s.inv_freq.data_ptr(), s.magnitude)
                 table = ctx.scratch.get(key)
                 if table is None:
-                    table = ctx.scratch[key] = ops.rope_table64(ctx.positions, s.inv_freq)
+                    table = ctx.scratch[key] = ops.rope_table64(ctx.positions, s.inv_freq, s.magnitude)
             q, k, v = ops.shaped_qkv_store(
                 projected, q_heads, kv_heads if writes_cache else 0, head_dim, dv, ctx.positions, ctx.runtime.dtype,
                 bias=bias, taps=s.taps, tails=s.tails.state if s.tails is not None else None,
                 cu_seqlens=ctx.cu_seqlens, seq_of_token=ctx.seq_of_token, slots=ctx.slots, row_norm=s.row_norm,
                 row_eps=s.row_eps, head_weights=s.head_weights, head_weight_eps=s.head_weight_eps,
                 inv_freq=s.inv_freq, rotary=s.rotary, adjacent_pairs=s.adjacent_pairs, head_norm_eps=s.head_norm_eps,
-                table=table, **stored)
+                table=table, magnitude=s.magnitude, **stored)
         else:
             q, k, v = ops.qkv_bias_store(projected, bias, q_heads, kv_heads if writes_cache else 0, head_dim, dv,
                                          **stored)
@@ -480,11 +520,13 @@ def attend(projected, *, q_heads: int, kv_heads: int, head_dim: int, rotary, ctx
             if writes_cache:
                 ctx.fresh_kv[cache_entry] = (k, k if values_are_keys else v)
             k, v = ctx.fresh_kv[cache_entry]
-        if sigmoid_weights is not None:
+        if sigmoid_weights is not None or form is not None:
             where = dict(k=k, v=v) if prefill_phase else dict(kv=cache, slots=ctx.slots, kv_lens=ctx.kv_lens,
                                                               max_kv_len=ctx.max_kv_len)
             if phase != "decode":
                 where.update(cu_seqlens=ctx.cu_seqlens, seq_of_token=ctx.seq_of_token, positions=ctx.positions)
+            if form is not None:
+                return ops.attention_gated(q, form, scale, window, out_scale, ctx.max_seq_len, **where)
             return ops.attention_sigmoid(q, sigmoid_weights, scale, window, out_scale, ctx.max_seq_len, **where)
         if prefill_phase:
             return ops.attention_prefill(q, k, v, ctx.cu_seqlens, ctx.seq_of_token, ctx.max_seq_len, scale, window,

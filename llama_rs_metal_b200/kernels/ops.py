@@ -169,15 +169,24 @@ def _check_norm(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tens
 
 
 def layer_norm(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], eps: float, out_dtype: torch.dtype,
-               rows: Optional[torch.Tensor] = None, partials: Optional[torch.Tensor] = None) -> torch.Tensor:
+               rows: Optional[torch.Tensor] = None, partials: Optional[torch.Tensor] = None,
+               add: Optional[torch.Tensor] = None) -> torch.Tensor:
     """(x - mean) / sqrt(variance + eps) * weight [+ bias] over float32 rows [T, h] (all, or those `rows`
     names); weight and bias float32 [h]. `partials` float32 [n, T, h]: slices that are first added into
-    the rows (and written back, unless rows are gathered). -> [T or len(rows), h] in `out_dtype`."""
+    the rows (and written back, unless rows are gathered). `add` float32 [h] (not with `rows`): added to
+    every row of x behind that, the norm is of the rows without it. -> [T or len(rows), h] in `out_dtype`."""
     n_partials, stride = _check_norm(x, weight, bias, partials, "layer_norm")
     hidden = x.shape[1]
     if n_partials and hidden > LAYER_NORM_FOLDS:
         add_planes_(x, partials)
         partials, n_partials, stride = None, 0, 0
+    late = None  # rows too long for the kernel to move: a pass of its own
+    if add is not None:
+        _check(add, "add", torch.float32, 1)
+        if add.numel() != hidden or rows is not None:
+            raise InvalidError("layer_norm: a row to add has one entry per column, and no rows are chosen")
+        if hidden > LAYER_NORM_FOLDS:
+            late, add = add, None
     n_rows = x.shape[0]
     if rows is not None:
         _check(rows, "rows", torch.int32, 1)
@@ -185,7 +194,9 @@ def layer_norm(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tenso
     out = _activation(n_rows, hidden, out_dtype, x.device)
     _done(_lib().lrm_layer_norm(_ptr(x), _ptr(weight), _ptr(bias), _ptr(out), _code(out_dtype), _ptr(rows), n_rows,
                                 hidden, ctypes.c_float(eps), _ptr(partials), n_partials, ctypes.c_longlong(stride),
-                                _stream()), "layer_norm")
+                                _ptr(add), _stream()), "layer_norm")
+    if late is not None:
+        add_row_(x, late)
     return out
 
 
@@ -606,14 +617,15 @@ def rope_table(positions: torch.Tensor, inv_freq: torch.Tensor) -> torch.Tensor:
     return table
 
 
-def rope_table64(positions: torch.Tensor, inv_freq: torch.Tensor) -> torch.Tensor:
-    """float32 [T, R/2, 2]: (cos, sin) of position * inv_freq with the angle in double precision (inv_freq
-    float64), the angles shaped_qkv_store forms."""
+def rope_table64(positions: torch.Tensor, inv_freq: torch.Tensor, magnitude: float = 1.0) -> torch.Tensor:
+    """float32 [T, R/2, 2]: (cos, sin) of position * inv_freq, both times `magnitude`, with the angle in double
+    precision (inv_freq float64), the angles shaped_qkv_store forms."""
     _check(positions, "positions", torch.int32, 1)
     _check(inv_freq, "inv_freq", torch.float64, 1)
     T, half = positions.numel(), inv_freq.numel()
     table = torch.empty((T, half, 2), dtype=torch.float32, device=positions.device)
-    _done(_lib().lrm_rope_table64(_ptr(positions), _ptr(inv_freq), _ptr(table), T, half, _stream()), "rope_table64")
+    _done(_lib().lrm_rope_table64(_ptr(positions), _ptr(inv_freq), _ptr(table), T, half, ctypes.c_double(magnitude),
+                                  _stream()), "rope_table64")
     return table
 
 
@@ -686,7 +698,7 @@ def shaped_qkv_store(qkv: torch.Tensor, q_heads: int, kv_heads: int, head_dim: i
                      slots: Optional[torch.Tensor] = None, row_norm=None, row_eps: float = 0.0,
                      head_weights=None, head_weight_eps: float = 0.0, inv_freq: Optional[torch.Tensor] = None, rotary: int = 0, adjacent_pairs: bool = False,
                      head_norm_eps: Optional[float] = None, kv=None, dest_rows: Optional[torch.Tensor] = None,
-                     keep_packed: bool = True, table: Optional[torch.Tensor] = None):
+                     keep_packed: bool = True, table: Optional[torch.Tensor] = None, magnitude: float = 1.0):
     """Split a fused [T, Hq*d + Hk*d + Hk*dv (+ more)] projection (float32, or `out_dtype`; columns behind
     the row are left alone) whose queries and keys are shaped on the way, each step only if asked for and in this order: `bias` (float32
     [row]); a causal convolution per channel (`taps` float32 [n, row], the last row the current
@@ -695,8 +707,8 @@ def shaped_qkv_store(qkv: torch.Tensor, q_heads: int, kv_heads: int, head_dim: i
     query columns and one over all key columns (`row_norm` = (q weight, k weight), `row_eps`); an RMS
     norm over every query and every key head (`head_weights` = (q weight, k weight), float32 [d] each,
     `head_weight_eps`); the rotation of each head's first `rotary` dimensions by `inv_freq` (float64 [rotary/2]; split halves,
-    or neighbours with `adjacent_pairs`; `table`: rope_table64 of the step, which saves the kernel its
-    angles); each head divided by its root mean square
+    or neighbours with `adjacent_pairs`; cosines and sines times `magnitude`; `table`: rope_table64 of the step
+    with the same frequencies and magnitude, which saves the kernel its angles); each head divided by its root mean square
     (`head_norm_eps`). Returns (q [T,Hq,d], k, v) like qkv_bias_store, and writes the cache view."""
     _check(qkv, "qkv", dims=2)
     T = qkv.shape[0]
@@ -769,7 +781,8 @@ def shaped_qkv_store(qkv: torch.Tensor, q_heads: int, kv_heads: int, head_dim: i
         _ptr(tails if n > 1 else None),
         _ptr(cu_seqlens if n > 1 else None), _ptr(seq_of_token if n > 1 else None), _ptr(slots if n > 1 else None),
         _ptr(positions), _ptr(q_norm), _ptr(k_norm), ctypes.c_float(row_eps), _ptr(q_head), _ptr(k_head),
-        ctypes.c_float(head_weight_eps), _ptr(inv_freq if rotary else None), _ptr(table if rotary else None), rotary, int(bool(adjacent_pairs)), int(head_norm_eps is not None),
+        ctypes.c_float(head_weight_eps), _ptr(inv_freq if rotary else None), ctypes.c_double(magnitude),
+        _ptr(table if rotary else None), rotary, int(bool(adjacent_pairs)), int(head_norm_eps is not None),
         ctypes.c_float(head_norm_eps if head_norm_eps is not None else 0.0), _ptr(q), _ptr(k), _ptr(v),
         _ptr(k_pages), _ptr(v_pages), _ptr(dest_rows if k_pages is not None else None), _code(out_dtype), T, q_heads,
         kv_heads, head_dim, value_dim, page_size, _stream()), "shaped_qkv_store")
@@ -1682,6 +1695,44 @@ def attention_extend(q: torch.Tensor, kv, cu_seqlens: torch.Tensor, seq_of_token
     return out
 
 
+def _attention_geometry(what: str, q, k, v, kv, cu_seqlens, seq_of_token, slots, kv_lens):
+    """Checks of attention over packed keys k, v or the cache view kv; -> (T, Hq, d, key heads, dv)."""
+    _check(q, "q", dims=3)
+    T, Hq, d = q.shape
+    if kv is None:
+        _check(k, "k", q.dtype, 3)
+        _check(v, "v", q.dtype, 3)
+        heads, dv = k.shape[1], v.shape[2]
+        if k.shape[0] != T or k.shape[2] != d or k.shape[:2] != v.shape[:2] or Hq % heads:
+            raise InvalidError(f"{what}: q, k, v shapes do not agree")
+    else:
+        _check(kv.k, "k pages", q.dtype, 4)
+        _check(kv.v, "v pages", q.dtype, 4)
+        _check(kv.page_table, "page table", torch.int32, 2)
+        heads, dv = kv.kv_heads, _value_dim(kv)
+        if tuple(kv.k.shape[1:]) != (heads, kv.page_size, d) or Hq % heads:
+            raise InvalidError(f"{what}: cache pages do not match the query geometry")
+        for name, t in (("slots", slots), ("kv_lens", kv_lens)):
+            _check(t, name, torch.int32, 1)
+    if kv is None or cu_seqlens is not None:
+        _check(cu_seqlens, "cu_seqlens", torch.int32, 1)
+        _check(seq_of_token, "seq_of_token", torch.int32, 1)
+    elif slots.numel() != T:
+        raise InvalidError(f"{what}: one query per sequence")
+    return T, Hq, d, heads, dv
+
+
+def _gate_columns(what: str, gate, rows: int, width: int):
+    """(pointer at the first column, row stride) of a gate (tensor float32 [rows, W], column), or (null, 0)."""
+    if gate is None:
+        return ctypes.c_void_p(0), 0
+    tensor, column = gate
+    _check(tensor, "gate", torch.float32, 2)
+    if tensor.shape[0] != rows or column < 0 or column + width > tensor.shape[1]:
+        raise InvalidError(f"{what}: gate columns outside the activation")
+    return _column_ptr(tensor, column), tensor.shape[1]
+
+
 @dataclass(frozen=True)
 class SigmoidWeights:
     """Attention without a softmax: a visible key's weight is sigmoid(score + offset_h), not normalized
@@ -1703,44 +1754,59 @@ def attention_sigmoid(q: torch.Tensor, weights: SigmoidWeights, scale: float, wi
     With k, v (packed [T, Hk, d | dv], sequences from position 0: cu_seqlens, seq_of_token) a prompt; with
     the cache view `kv` one query per sequence (slots, kv_lens), or, where cu_seqlens, seq_of_token and
     positions are given too, a portion per sequence whose keys the cache already holds."""
-    _check(q, "q", dims=3)
-    T, Hq, d = q.shape
+    T, Hq, d, heads, dv = _attention_geometry("attention_sigmoid", q, k, v, kv, cu_seqlens, seq_of_token, slots, kv_lens)
     _check(weights.offset, "offset", torch.float32, 1)
     if weights.offset.numel() != Hq:
         raise InvalidError("attention_sigmoid: one offset per query head")
-    if kv is None:
-        _check(k, "k", q.dtype, 3)
-        _check(v, "v", q.dtype, 3)
-        heads, dv = k.shape[1], v.shape[2]
-        if k.shape[0] != T or k.shape[2] != d or k.shape[:2] != v.shape[:2] or Hq % heads:
-            raise InvalidError("attention_sigmoid: q, k, v shapes do not agree")
-    else:
-        _check(kv.k, "k pages", q.dtype, 4)
-        _check(kv.v, "v pages", q.dtype, 4)
-        _check(kv.page_table, "page table", torch.int32, 2)
-        heads, dv = kv.kv_heads, _value_dim(kv)
-        if tuple(kv.k.shape[1:]) != (heads, kv.page_size, d) or Hq % heads:
-            raise InvalidError("attention_sigmoid: cache pages do not match the query geometry")
-        for name, t in (("slots", slots), ("kv_lens", kv_lens)):
-            _check(t, name, torch.int32, 1)
-    if kv is None or cu_seqlens is not None:
-        _check(cu_seqlens, "cu_seqlens", torch.int32, 1)
-        _check(seq_of_token, "seq_of_token", torch.int32, 1)
-    elif slots.numel() != T:
-        raise InvalidError("attention_sigmoid: one query per sequence")
-    gate, gate_stride = ctypes.c_void_p(0), 0
-    if weights.gate is not None:
-        tensor, column = weights.gate
-        _check(tensor, "gate", torch.float32, 2)
-        if tensor.shape[0] != T or column < 0 or column + Hq * dv > tensor.shape[1]:
-            raise InvalidError("attention_sigmoid: gate columns outside the activation")
-        gate, gate_stride = _column_ptr(tensor, column), tensor.shape[1]
+    gate, gate_stride = _gate_columns("attention_sigmoid", weights.gate, T, Hq * dv)
     given, column = weights.out if weights.out is not None else (None, 0)
     out, out_ptr = _output_columns(given, column, T, Hq * dv, q.dtype, q.device)
     from . import attention_dispatch
     attention_dispatch.sigmoid(q, k, v, kv, heads, dv, out_ptr, out.shape[1], weights.offset, gate, gate_stride, scale,
                                window or 0, out_scale, max_seq_len, max_kv_len, cu_seqlens, seq_of_token, positions,
                                slots, kv_lens)
+    return out
+
+
+@dataclass(frozen=True)
+class SoftmaxForm:
+    """Softmax attention beyond the plain form (csrc/attention_gated.cu), each step only if asked for.
+
+    cap: scores become cap * tanh(score / cap). sinks: float32 [query heads], exp(sink_h) joins the
+    denominator. keep_first: beside its window (or chunk) every query sees the sequence's first so many
+    keys. gate (tensor float32 [T, W], column): the result is multiplied by the sigmoid of those columns, one
+    per head and value dimension, or with `gate_per_head` one per head. out (tensor [T, W'], column): where
+    the result goes (None: a tensor of its own)."""
+
+    cap: Optional[float] = None
+    sinks: Optional[torch.Tensor] = None
+    keep_first: int = 0
+    gate: Optional[Tuple[torch.Tensor, int]] = None
+    gate_per_head: bool = False
+    out: Optional[Tuple[torch.Tensor, int]] = None
+
+
+def attention_gated(q: torch.Tensor, form: SoftmaxForm, scale: float, window: Optional[int], out_scale: float,
+                    max_seq_len: int, k: Optional[torch.Tensor] = None, v: Optional[torch.Tensor] = None, kv=None,
+                    cu_seqlens: Optional[torch.Tensor] = None, seq_of_token: Optional[torch.Tensor] = None,
+                    positions: Optional[torch.Tensor] = None, slots: Optional[torch.Tensor] = None,
+                    kv_lens: Optional[torch.Tensor] = None, max_kv_len: int = 0) -> torch.Tensor:
+    """Causal softmax attention of the form `form` -> [T, Hq*dv] (or the columns form.out names). Where keys
+    come from is told as for attention_sigmoid; `window` > 0 a window, < 0 a chunk."""
+    what = "attention_gated"
+    T, Hq, d, heads, dv = _attention_geometry(what, q, k, v, kv, cu_seqlens, seq_of_token, slots, kv_lens)
+    if form.sinks is not None:
+        _check(form.sinks, "sinks", torch.float32, 1)
+        if form.sinks.numel() != Hq:
+            raise InvalidError(f"{what}: one sink per query head")
+    if (form.cap is not None and form.cap <= 0) or form.keep_first < 0:
+        raise InvalidError(f"{what}: a cap is positive, and so are kept keys")
+    gate, gate_stride = _gate_columns(what, form.gate, T, Hq if form.gate_per_head else Hq * dv)
+    given, column = form.out if form.out is not None else (None, 0)
+    out, out_ptr = _output_columns(given, column, T, Hq * dv, q.dtype, q.device)
+    from . import attention_dispatch
+    attention_dispatch.gated(q, k, v, kv, heads, dv, out_ptr, out.shape[1], form, gate, gate_stride, scale, window or 0,
+                             out_scale, max_seq_len, max_kv_len, cu_seqlens, seq_of_token, positions, slots, kv_lens)
     return out
 
 

@@ -50,9 +50,14 @@ class Attention(Mixer):
 
     `weights` "sigmoid": no softmax. A visible key's weight is sigmoid(score + `score_offset`[head]) (a stored
     tensor, one number per query head), not normalized over the keys (csrc/attention_sigmoid.cu; the layer takes
-    the shaped split). `gate` (with sigmoid weights): the heads are multiplied element by element by
-    sigmoid(W_g x) ahead of the output projection (tensor `g_proj.weight`); it rides in the fused projection
-    and the attention kernels apply it where they write.
+    the shaped split). `gate`: the heads are multiplied by sigmoid(W_g x) ahead of the output projection (tensor
+    `g_proj.weight`), element by element ("element", or True) or, with softmax weights, with one number per head
+    ("head"); it rides in the fused projection and the attention kernels apply it where they write.
+
+    Softmax weights beyond the plain form (any of these, and a softmax gate, make the layer take the shaped split
+    and csrc/attention_gated.cu, sinks included): `score_cap` c, scores become c tanh(score / c); `keep_first` n,
+    beside its window a query sees the sequence's first n keys, whose pages the cache then never gives back.
+    `output_bias`: the output projection has a bias (tensor `o_proj.bias`).
     """
 
     def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int,
@@ -61,8 +66,9 @@ class Attention(Mixer):
                  output_scale: float = 1.0, values_are_keys: bool = False, sinks: bool = False,
                  query_temperature: Optional[Sequence[float]] = None, conv_taps: int = 0,
                  row_norm_eps: Optional[float] = None, head_norm_eps: Optional[float] = None,
-                 chunk: Optional[int] = None, weights: str = "softmax", gate: bool = False,
-                 head_weight_eps: Optional[float] = None):
+                 chunk: Optional[int] = None, weights: str = "softmax", gate=False,
+                 head_weight_eps: Optional[float] = None, score_cap: Optional[float] = None, keep_first: int = 0,
+                 output_bias: bool = False):
         if weights not in ("softmax", "sigmoid"):
             raise UnsupportedError(f"attention weights {weights!r}")
         if num_heads <= 0 or num_kv_heads <= 0 or num_heads % num_kv_heads:
@@ -76,21 +82,34 @@ class Attention(Mixer):
             if every <= 0:
                 raise InvalidError("a query temperature grows every so many positions: a positive number")
             self.query_temperature = (coef, every)
-        self.extras = None
+        self.extras = self.sinks = None
         self.conv_taps = int(conv_taps)
         self.row_norm_eps = None if row_norm_eps is None else float(row_norm_eps)
         self.head_norm_eps = None if head_norm_eps is None else float(head_norm_eps)
         self.chunk = int(chunk) if chunk else None
         if self.conv_taps < 0 or (self.chunk is not None and (self.chunk <= 0 or window is not None)):
             raise InvalidError("attention: taps cannot be negative, and a chunked layer has no window besides")
-        self.sigmoid, self.gate = weights == "sigmoid", bool(gate)
+        self.sigmoid, self.gate = weights == "sigmoid", "element" if gate is True else (gate or None)
+        self.score_cap, self.keep_first = None if score_cap is None else float(score_cap), int(keep_first)
+        self.has_output_bias = bool(output_bias)
+        if self.gate not in (None, "element", "head") or (self.sigmoid and self.gate == "head"):
+            raise InvalidError(f"attention: output gate {gate!r}")
+        if (self.score_cap is not None and self.score_cap <= 0) or self.keep_first < 0:
+            raise InvalidError("attention: a cap on the scores is positive, and so is the number of kept keys")
+        if self.sigmoid and (self.score_cap is not None or self.keep_first):
+            raise InvalidError("attention: capped scores and kept keys are built for softmax weights only")
+        # softmax weights that the general kernels (csrc/attention_gated.cu) compute
+        self.formed = not self.sigmoid and (self.score_cap is not None or self.keep_first > 0 or self.gate is not None)
+        self.position = build_part(POSITION_ENCODINGS, position, "position encoding") \
+            if position is not None else None
+        if getattr(self.position, "magnitude", 1.0) != 1.0:
+            self.formed = not self.sigmoid  # only the shaped split applies a rotation's magnitude
         self.head_weight_eps = None if head_weight_eps is None else float(head_weight_eps)
         self.shaped = bool(self.conv_taps) or any(e is not None for e in (self.row_norm_eps, self.head_norm_eps,
-                                                                          self.head_weight_eps)) or self.sigmoid
-        if self.gate and not self.sigmoid:
-            raise InvalidError("an output gate is built together with sigmoid weights only")
+                                                                          self.head_weight_eps)) or self.sigmoid \
+            or self.formed
         self.head_weights = self.score_offset = None
-        if self.shaped and (values_are_keys or sinks or query_temperature is not None):
+        if self.shaped and (values_are_keys or (sinks and not self.formed) or query_temperature is not None):
             raise InvalidError("shaped queries and keys are not built together with sinks, a query temperature or keys as values")
         self.taps = self.row_norm = None
         self.hidden_size, self.num_heads, self.num_kv_heads = hidden_size, num_heads, num_kv_heads
@@ -99,8 +118,6 @@ class Attention(Mixer):
         self.has_bias, self.output_scale = bool(bias), float(output_scale)
         self.bias: Optional[torch.Tensor] = None
         self.scale = float(scale) if scale is not None else 1.0 / math.sqrt(head_dim)
-        self.position = build_part(POSITION_ENCODINGS, position, "position encoding") \
-            if position is not None else None
         self.qkv: Optional[LinearWeight] = None
         self.q_only: Optional[LinearWeight] = None
         self.out: Optional[LinearWeight] = None
@@ -132,7 +149,9 @@ class Attention(Mixer):
         if self.sigmoid:
             out["score_offset"] = TensorSpec((self.num_heads,))
         if self.gate:
-            out["g_proj.weight"] = TensorSpec((mixed, h))
+            out["g_proj.weight"] = TensorSpec((mixed if self.gate == "element" else self.num_heads, h))
+        if self.has_output_bias:
+            out["o_proj.bias"] = TensorSpec((h,))
         if self.position is not None:
             out.update({"position." + n: s for n, s in self.position.tensors().items()})
         return out
@@ -153,13 +172,17 @@ class Attention(Mixer):
         if self.gate:  # behind q | k | v
             rows.append(weights["g_proj.weight"])
         fused = torch.cat(rows, dim=0).contiguous()
-        if self.has_sinks or self.query_temperature is not None:
+        if self.formed:
+            self.sinks = weights["sinks"].to(torch.float32).contiguous() if self.has_sinks else None
+        elif self.has_sinks or self.query_temperature is not None:
             from ..kernels.attention_dispatch import Extras
             sinks = weights["sinks"].to(torch.float32).contiguous() if self.has_sinks else None
             self.extras = Extras(sinks, self.query_temperature)
         self.qkv = LinearWeight(fused)
         self.q_only = LinearWeight(fused[: self.num_heads * self.head_dim])
         self.out = LinearWeight(weights["o_proj.weight"])
+        if self.has_output_bias:
+            self.output_bias = (weights["o_proj.bias"].to(torch.float32) * self.output_scale).contiguous()
         if self.has_bias:
             if order is not None:
                 raise InvalidError("projection biases with a reordered head are not built")
@@ -178,7 +201,7 @@ class Attention(Mixer):
             self.head_weights = tuple(weights[n + "_head_norm.weight"].to(torch.float32).contiguous() for n in "qk")
         if self.sigmoid:
             self.score_offset = weights["score_offset"].to(torch.float32).contiguous()
-        if self.shaped and self.position is not None and self.position.rotary_table() is None:
+        if self.shaped and self.position is not None and getattr(self.position, "inv_freq64", None) is None:
             raise InvalidError("a shaped attention layer rotates by a rotary table or not at all")
 
     @property
@@ -189,44 +212,62 @@ class Attention(Mixer):
         # a chunk never shows a key more than `chunk` - 1 positions back: the cache keeps that window
         keys = KeyValueRequest(self.num_kv_heads, self.head_dim, self.chunk or self.window,
                                None if self.value_dim == self.head_dim else self.value_dim,
-                               values_in_keys=self.values_are_keys)
+                               values_in_keys=self.values_are_keys,
+                               keep_first=self.keep_first if self.chunk or self.window else 0)
         if self.conv_taps > 1:
             return CompositeRequest((keys, StateRequest((self.conv_taps - 1, self.projected_width), torch.float32)))
         return keys
 
     @property
     def mixed_width(self) -> Optional[int]:
-        return self.num_heads * self.value_dim if self.sigmoid else None
+        return self.num_heads * self.value_dim if self.sigmoid or self.formed else None
+
+    @property
+    def projection(self) -> Optional[LinearWeight]:
+        return self.qkv if self.shaped else None
 
     def mix(self, x, ctx, cache, out=None, column=0):
         """Projection in float32, then bias, convolution, norms and rotation in one kernel that also
         splits and stores, then attention under the window or the chunk."""
+        return self.mix_projected(self.qkv(x, out_dtype=torch.float32), ctx, cache, out, column)
+
+    def mix_projected(self, projected, ctx, cache, out=None, column=0):
         from ..kernels.attention_dispatch import Shaping
         entry = ctx.entry
         if not entry.writes_cache:
             raise UnsupportedError("a shaped attention layer reading another layer's cache is not built")
         keys, tails = cache if self.conv_taps > 1 else (cache, None)
-        inv_freq, rotary, adjacent = None, 0, False
+        inv_freq, rotary, adjacent, magnitude = None, 0, False, 1.0
         if self.position is not None:
+            magnitude = self.position.magnitude
             rotary, adjacent = self.position.rotary_dim, self.position.adjacent_pairs
             inv_freq = self.position.inv_freq64
         shaping = Shaping(taps=self.taps, tails=tails, row_norm=self.row_norm, row_eps=self.row_norm_eps or 0.0,
                           head_weights=self.head_weights, head_weight_eps=self.head_weight_eps or 0.0,
-                          inv_freq=inv_freq, rotary=rotary, adjacent_pairs=adjacent, head_norm_eps=self.head_norm_eps)
-        projected = self.qkv(x, out_dtype=torch.float32)
-        sigmoid = None
+                          inv_freq=inv_freq, magnitude=magnitude, rotary=rotary, adjacent_pairs=adjacent,
+                          head_norm_eps=self.head_norm_eps)
+        sigmoid = form = None
+        gate = (projected, self.projected_width) if self.gate else None
+        where = (out, column) if out is not None else None
         if self.sigmoid:
-            sigmoid = ops.SigmoidWeights(self.score_offset, (projected, self.projected_width) if self.gate else None,
-                                         (out, column) if out is not None else None)
+            sigmoid = ops.SigmoidWeights(self.score_offset, gate, where)
+        elif self.formed:
+            form = ops.SoftmaxForm(self.score_cap, self.sinks, self.keep_first, gate, self.gate == "head", where)
         elif out is not None:
             raise UnsupportedError("softmax attention writes a tensor of its own")
         return ops.attend(projected, q_heads=self.num_heads, kv_heads=self.num_kv_heads,
                           head_dim=self.head_dim, rotary=None, ctx=ctx, cache=keys, writes_cache=True,
                           cache_entry=entry.cache, scale=self.scale, window=self.chunk or self.window,
                           value_dim=self.value_dim, bias=self.bias, out_scale=self.output_scale, shaping=shaping,
-                          chunk=self.chunk, sigmoid_weights=sigmoid)
+                          chunk=self.chunk, sigmoid_weights=sigmoid, form=form)
 
     def forward(self, x, ctx, cache, residual):
+        hidden = self._forward(x, ctx, cache, residual)
+        if self.output_bias is not None:
+            ops.add_row_(hidden, self.output_bias)
+        return hidden
+
+    def _forward(self, x, ctx, cache, residual):
         if self.shaped:
             return self.out(self.mix(x, ctx, cache), epilogue=ops.ADD, out=residual, ctx=ctx)
         entry = ctx.entry

@@ -141,7 +141,8 @@ class KeyValueRequest:
     `window` None keeps every key; a number keeps the last `window` positions.
     `value_dim` None: values are as wide as keys. `values_in_keys`: a token's value row is the
     first `value_dim` columns of its key row (all of it when `value_dim` is None), so only keys
-    are stored and the attention kernels read values out of them. Layers with equal requests
+    are stored and the attention kernels read values out of them. `keep_first`: beside the window,
+    a sequence's first so many positions are kept as well. Layers with equal requests
     share one storage group.
     """
 
@@ -150,6 +151,7 @@ class KeyValueRequest:
     window: Optional[int] = None
     value_dim: Optional[int] = None
     values_in_keys: bool = False
+    keep_first: int = 0
 
 
 @dataclass(frozen=True)
@@ -197,6 +199,15 @@ class Norm(Part):
         """float32 residual [T,h] -> normalized activations [T,h] (or [len(rows),h])."""
         raise NotImplementedError
 
+    def forward_add(self, hidden: torch.Tensor, ctx, row: torch.Tensor) -> torch.Tensor:
+        """forward(hidden), and `row` (float32 [h]) is then added to every row of the stream: what a
+        sublayer adds whatever its input (a bias of its output) rides in a pass over the stream that is
+        made anyway."""
+        from ..kernels import ops
+        y = self.forward(hidden, ctx)
+        ops.add_row_(hidden, row)
+        return y
+
     def forward_conv(self, hidden: torch.Tensor, ctx, taps: torch.Tensor, tails: Optional[torch.Tensor]) -> torch.Tensor:
         """h + conv(h) for h = forward(hidden): a causal convolution over time per channel behind the norm
         (taps float32 [n, width], the last row the current token's), whose inputs before the step come
@@ -241,10 +252,21 @@ class Mixer(Part):
     # A mixer whose output is one product `out` (a LinearWeight) over a row of mixed heads of this many
     # columns, and that can make that row without the product (mix()); None for other mixers.
     mixed_width: Optional[int] = None
+    # float32 [h] that the mixer's output has beside `out` times the mixed row (forward() adds it), or None
+    output_bias: Optional[torch.Tensor] = None
 
     def mix(self, x: torch.Tensor, ctx, cache, out: Optional[torch.Tensor] = None, column: int = 0) -> torch.Tensor:
         """The mixed heads ahead of the output product, [T, mixed_width] in the activation type: a new
         tensor, or columns column .. of `out`, which is returned."""
+        raise NotImplementedError
+
+    # The one product a mixer makes from its input (a LinearWeight whose float32 result it can be given
+    # instead: mix_projected), once bound; None for mixers that read their input otherwise.
+    projection: Optional[Any] = None
+
+    def mix_projected(self, projected: torch.Tensor, ctx, cache, out: Optional[torch.Tensor] = None,
+                      column: int = 0) -> torch.Tensor:
+        """mix() from columns 0 .. of `projected`, float32 [T, at least projection.out_features]."""
         raise NotImplementedError
 
     def cache_request(self):

@@ -96,6 +96,49 @@ class PreNormMixerBlock(_PreNormBlock):
         return hidden
 
 
+class _ParallelBlock(Block):
+    """One norm whose output every sublayer reads: hidden += mixer(x) + feed_forward(x), x = norm(hidden).
+
+    A bias of the mixer's output rides in the norm's pass over the stream (Norm.forward_add)."""
+
+    graph_safe = True
+
+    @property
+    def folds_pending_on_entry(self) -> bool:
+        return self.norm.folds_pending
+
+
+@register_block("parallel")
+class ParallelBlock(_ParallelBlock):
+    """A mixer and a feed-forward side by side on the same input."""
+
+    roles = {"mixer": "mixer", "feed_forward": "feed_forward", "norm": "norm"}
+
+    def forward(self, hidden, ctx, cache):
+        after = ctx.next_folds_pending
+        x = self.norm.forward(hidden, ctx)
+        hidden = self.mixer.forward(x, ctx, cache, residual=hidden)
+        ctx.may_defer = after
+        hidden = self.feed_forward.forward(x, ctx, residual=hidden)
+        ctx.may_defer = False
+        return hidden
+
+
+@register_block("parallel_mixer")
+class ParallelMixerBlock(_ParallelBlock):
+    """The same for a layer without a feed-forward."""
+
+    roles = {"mixer": "mixer", "norm": "norm"}
+
+    def forward(self, hidden, ctx, cache):
+        after = ctx.next_folds_pending
+        x = self.norm.forward(hidden, ctx)
+        ctx.may_defer = after
+        hidden = self.mixer.forward(x, ctx, cache, residual=hidden)
+        ctx.may_defer = False
+        return hidden
+
+
 class _ScaledPreNormBlock(Block):
     """Pre-norm sublayers whose outputs enter the stream under a factor per channel:
     hidden += mult * scale * sublayer(norm(hidden)), with `scale` a stored vector per sublayer

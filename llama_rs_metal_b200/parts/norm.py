@@ -102,6 +102,10 @@ class LayerNorm(Norm):
         return ops.layer_norm(hidden, self.weight, self.bias, self.eps, ctx.runtime.dtype, rows=rows,
                               partials=ctx.take_pending())
 
+    def forward_add(self, hidden, ctx, row):
+        return ops.layer_norm(hidden, self.weight, self.bias, self.eps, ctx.runtime.dtype, partials=ctx.take_pending(),
+                              add=row)
+
     def forward_conv(self, hidden, ctx, taps, tails):
         if ctx.phase != "decode" or tails is None or self.size > ops.LAYER_NORM_FOLDS:
             return super().forward_conv(hidden, ctx, taps, tails)

@@ -28,7 +28,8 @@ class ParallelMixer(Mixer):
                                "mixer")
         self.right = build_part(MIXERS, PartSpec(right.kind, {**right.params, "output_scale": float(right_scale)}),
                                 "mixer")
-        self.joint = self.left.mixed_width is not None and self.right.mixed_width is not None
+        self.joint = all(m.mixed_width is not None and not getattr(m, "has_output_bias", False)
+                         for m in (self.left, self.right))
         self.out: Optional[LinearWeight] = None
 
     @property
