@@ -309,9 +309,33 @@ def tolurax_shape(width, heads, kv_heads, ff, window, layers, vocab=32768):
                 layers=[delta] + [parallel] * (layers - 1), loop=dict(start=0, stop=2, times=2))
 
 
+def munupel_shape(width, heads, kv_heads, ff, window, layers, vocab=32768):
+    """A Munupel configuration with layers of a real model's widths (head size 128, values as wide): chunked attention
+    with capped scores (chunks of `window`, half of each head rotated with stretched frequencies) and windowed
+    attention with sinks and 64 kept first keys in turn, a dense feed-forward beside each."""
+    d = 128
+    mlp = dict(kind="dense", ff=ff)
+    sizes = dict(heads=heads, kv_heads=kv_heads, dim=d, vdim=d, scale=d ** -0.5)
+    kinds = [
+        dict(type="attention", mlp=mlp, mixer=dict(sizes, softcap=30.0, mask=dict(size=window), rot=dict(
+            dims=64, base=500000.0, scaling=dict(factor=8.0, original=4096, fast=32.0, slow=1.0)))),
+        dict(type="attention_2", mlp=mlp, mixer=dict(sizes, rot=dict(dims=d, base=500000.0),
+                                                     mask=dict(size=window, keep_first=64))),
+    ]
+    return dict(architecture="Munupel", vocab=vocab, width=width, norm=dict(eps=1e-5),
+                layers=[dict(kinds[i % 2]) for i in range(layers)])
+
+
+MUNUPEL_SIZES = {   # width, heads, kv heads, feed-forward width, window and chunk, layers
+    "1k": (1024, 8, 2, 4096, 512, 4),
+    "2k": (2048, 16, 4, 8192, 1024, 4),
+    "4k": (4096, 32, 8, 14336, 2048, 4),
+}
+
+
 def design_bench(args) -> int:
-    """Prefill and decode throughput of the Kikalix, Pibuvik, Norevik, Tarupel or Tolurax design at a few
-    layer sizes, beside an existing decoder at equal size: Kikalix and Pibuvik beside Llama (the same
+    """Prefill and decode throughput of the Kikalix, Pibuvik, Norevik, Tarupel, Tolurax or Munupel design at a few
+    layer sizes, beside an existing decoder at equal size: Kikalix, Pibuvik and Munupel beside Llama (the same
     width, head geometry, vocabulary and number of layer runs; its feed-forward as wide as the
     experts a token uses, or as the dense one), Norevik, Tarupel and Tolurax beside Kikalix, the closest of
     the designs (state mixers on the same scan, a looped run, windowed attention: equal width, heads, experts,
@@ -412,6 +436,12 @@ def design_bench(args) -> int:
             twin, twin_name = kikalix_shape(width, heads, kv_heads, ff, experts, top, window, layers), "kikalix_equal_size"
             shape = dict(width=width, heads=heads, kv_heads=kv_heads, head_dim=128, ff=top * ff, twin_expert_ff=ff,
                          twin_experts=experts, twin_top=top, time_mix_heads=width // 64, window=window, layer_runs=runs)
+        elif args.design == "munupel":
+            width, heads, kv_heads, ff, window, layers = MUNUPEL_SIZES[size]
+            config = munupel_shape(width, heads, kv_heads, ff, window, layers)
+            runs, twin_ff, norm_mean = layers, ff, 1.0
+            shape = dict(width=width, heads=heads, kv_heads=kv_heads, head_dim=128, ff=ff, window=window, keep_first=64,
+                         layers=layers)
         elif args.design == "pibuvik":
             width, heads, kv_heads, ff, kv_rank, window, layers = PIBUVIK_SIZES[size]
             config = pibuvik_shape(width, heads, kv_heads, ff, kv_rank, window, layers)
@@ -473,7 +503,7 @@ def main() -> int:
     parser.add_argument("--profile", action="store_true",
                         help="time every kernel launch (LRM_PROFILE=1) and print the table to stderr; the "
                              "line's numbers are then those of unfused, uncaptured launches")
-    parser.add_argument("--design", choices=["kikalix", "pibuvik", "norevik", "tarupel", "tolurax"], default=None,
+    parser.add_argument("--design", choices=["kikalix", "pibuvik", "norevik", "tarupel", "tolurax", "munupel"], default=None,
                         help="instead of the default workload: prefill and decode throughput of this design at "
                              "a few layer sizes beside an existing decoder at equal size (see design_bench)")
     parser.add_argument("--design-size", choices=sorted(DESIGN_SIZES), default=None,

@@ -18,7 +18,9 @@
 //    of the window; tiles that every query sees whole take no test per score.
 //  * decode (same sizes): one query per sequence over the cache; the CTAs of a thread-block cluster take runs
 //    of the visible pages, and their sums, maxima and masses meet in distributed shared memory in rank order:
-//    one launch, no partial rows in memory.
+//    one launch, no partial rows in memory. It can begin at the float32 projection (Fresh): it then adds the
+//    biases, rotates the queries and the new key, and stores the new key and value in the cache itself, with
+//    the arithmetic of shaped_qkv.cu.
 // Rows of a tile that nobody sees are zero-filled on the way into shared memory, so stale cache contents never
 // reach a product.
 #include <cooperative_groups.h>
@@ -51,6 +53,17 @@ struct Source {
   int table_stride;
   const int* slots;
   const int* kv_lens;
+};
+
+// The step's projection rows [q_heads * d | kv_heads * d | kv_heads * dv | ...], for a decode step that splits them
+// in the attention kernel. Rotation: dimension i of the first `rotary` of a head with i + rotary / 2.
+struct Fresh {
+  const float* proj;        // row b at proj + b * stride; null: q, k and v were split before
+  long long stride;
+  const float* bias;        // [row] or null
+  const float2* table;      // [seqs, rotary / 2] (cos, sin), or null
+  int rotary;
+  const int* dest_rows;     // [seqs]: page * 64 + row of the new token in the cache
 };
 
 __device__ __forceinline__ float gate_at(const Form& f, size_t t, int h, int dv, int j) {
@@ -320,8 +333,8 @@ __global__ __launch_bounds__(kThreads) void gated_tiled_kernel(const __nv_bfloat
 // A cluster of gridDim.x CTAs per (sequence, kv head, group of up to 16 query heads) [blockIdx.y]; the
 // CTA of rank r takes a run of the visible pages, its four warps 16 keys of every page each.
 template <int D, int DV>
-__global__ __launch_bounds__(kThreads) void gated_decode_kernel(const __nv_bfloat16* q, Source src, Form f, int q_heads,
-                                                                int kv_heads, int row_groups, int d, int dv) {
+__global__ __launch_bounds__(kThreads) void gated_decode_kernel(const __nv_bfloat16* q, Source src, Form f, Fresh fresh,
+                                                                int q_heads, int kv_heads, int row_groups, int d, int dv) {
   constexpr int KSTRIDE = D + 8, VSTRIDE = DV + 8, KTILE = kTile * KSTRIDE, VTILE = kTile * VSTRIDE;
   constexpr int PART = DV + 2;  // a row's sums, maximum (log2 domain) and mass
   extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -351,14 +364,61 @@ __global__ __launch_bounds__(kThreads) void gated_decode_kernel(const __nv_bfloa
     load_rows<DV>(Vs + stage * VTILE, static_cast<const __nv_bfloat16*>(src.v) + row * dv, dv, dv, lo, hi);
     cp_async_commit();
   };
-  // only q and the newest key and value row (in the last page) come from the kernel before this one
-  const bool early = begin < end && begin != count - 1;
+  // only q and the newest key and value row (in the last page) come from the kernel before this one; where
+  // this kernel splits the projection it puts the newest row there itself
+  const bool split = fresh.proj != nullptr;
+  const bool early = begin < end && (split || begin != count - 1);
   if (early) issue(begin, 0);
   pdl_wait();
   if (!early && begin < end) issue(begin, 0);
 
   uint32_t qa[D / 16][4];
-  load_queries<D>(qa, q + (static_cast<size_t>(b) * q_heads + head0) * d, d, d, rows);
+  __nv_bfloat16* Qs = Vs + 2 * VTILE;      // [16][D + 8], behind it the new key [D] and the new value [DV]
+  __nv_bfloat16* new_key = Qs + 16 * KSTRIDE;
+  __nv_bfloat16* new_value = new_key + D;
+  const bool has_newest = split && end == count && begin < end;
+  if (split) {
+    const float* row = fresh.proj + static_cast<size_t>(b) * fresh.stride;
+    const int half = fresh.rotary / 2;
+    const float2* turns = fresh.table + static_cast<size_t>(b) * half;
+    auto shaped = [&](int first, int c) {  // column c of the head that begins at column `first`
+      auto at = [&](int i) { return row[first + i] + (fresh.bias != nullptr ? fresh.bias[first + i] : 0.f); };
+      const float x = at(c);
+      if (c >= 2 * half) return x;
+      const bool leads = c < half;
+      const float2 turn = turns[leads ? c : c - half];
+      const float p = at(leads ? c + half : c - half);
+      return leads ? fmaf(x, turn.x, -__fmul_rn(p, turn.y)) : fmaf(x, turn.x, __fmul_rn(p, turn.y));
+    };
+    for (int i = threadIdx.x; i < 16 * D; i += kThreads) {
+      const int r = i / D, c = i % D;
+      Qs[r * KSTRIDE + c] = __float2bfloat16_rn(r < rows && c < d ? shaped((head0 + r) * d, c) : 0.f);
+    }
+    if (has_newest) {
+      const int dest = rg == 0 ? fresh.dest_rows[b] : -1;  // one of the groups of query heads stores the row
+      const size_t cached = dest >= 0 ? (static_cast<size_t>(dest / kTile) * kv_heads + kh) * kTile + dest % kTile : 0;
+      for (int c = threadIdx.x; c < d + dv; c += kThreads) {
+        if (c < d) {
+          const __nv_bfloat16 x = __float2bfloat16_rn(shaped((q_heads + kh) * d, c));
+          new_key[c] = x;
+          if (dest >= 0) const_cast<__nv_bfloat16*>(static_cast<const __nv_bfloat16*>(src.k))[cached * d + c] = x;
+        } else {
+          const int first = (q_heads + kv_heads) * d + kh * dv + c - d;
+          const __nv_bfloat16 x = __float2bfloat16_rn(row[first] + (fresh.bias != nullptr ? fresh.bias[first] : 0.f));
+          new_value[c - d] = x;
+          if (dest >= 0) const_cast<__nv_bfloat16*>(static_cast<const __nv_bfloat16*>(src.v))[cached * dv + c - d] = x;
+        }
+      }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int ks = 0; ks < D / 16; ++ks)
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        qa[ks][e] = *reinterpret_cast<const uint32_t*>(Qs + (g + 8 * (e & 1)) * KSTRIDE + 16 * ks + 8 * (e >> 1) + 2 * t);
+  } else {
+    load_queries<D>(qa, q + (static_cast<size_t>(b) * q_heads + head0) * d, d, d, rows);
+  }
   float o[DV / 8][4];
 #pragma unroll
   for (int dn = 0; dn < DV / 8; ++dn)
@@ -370,6 +430,14 @@ __global__ __launch_bounds__(kThreads) void gated_decode_kernel(const __nv_bfloa
     cp_async_wait<0>();  // page i is here
     __syncthreads();     // ... for every thread, and everyone is done with page i - 1
     if (i + 1 < end) issue(i + 1, stage ^ 1);
+    if (has_newest && i == count - 1) {  // the page's copy of the newest row is older than the row
+      const int r = query % kTile;
+      for (int c = threadIdx.x; c < d + dv; c += kThreads) {
+        if (c < d) Ks[stage * KTILE + r * KSTRIDE + c] = new_key[c];
+        else Vs[stage * VTILE + r * VSTRIDE + c - d] = new_value[c - d];
+      }
+      __syncthreads();
+    }
     float s[2][4];
 #pragma unroll
     for (int nt = 0; nt < 2; ++nt)
@@ -444,10 +512,12 @@ __global__ __launch_bounds__(kThreads) void gated_decode_kernel(const __nv_bfloa
 }
 
 template <int D, int DV> constexpr int tiles_bytes() { return 2 * kTile * (D + 8 + DV + 8) * 2; }
+template <int D, int DV> constexpr int fresh_bytes() { return (16 * (D + 8) + D + DV) * 2; }
 template <int DV> constexpr int parts_bytes() { return (kThreads / 32 + 1) * 16 * (DV + 2) * 4; }
 
 struct Geometry {
   int seqs, max_seq_len, q_heads, kv_heads, d, dv, ranks;
+  Fresh fresh;
 };
 
 template <int D, int DV>
@@ -465,7 +535,8 @@ int launch_tiled(const void* q, const Source& src, const Form& f, const int* cu_
 template <int D, int DV>
 int launch_decode(const void* q, const Source& src, const Form& f, const int*, const Geometry& g, cudaStream_t stream) {
   auto kernel = gated_decode_kernel<D, DV>;
-  const int bytes = tiles_bytes<D, DV>() > parts_bytes<DV>() ? tiles_bytes<D, DV>() : parts_bytes<DV>();
+  const int held = tiles_bytes<D, DV>() + (g.fresh.proj != nullptr ? fresh_bytes<D, DV>() : 0);
+  const int bytes = held > parts_bytes<DV>() ? held : parts_bytes<DV>();
   cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
   if (e != cudaSuccess) return static_cast<int>(e);
   const int row_groups = (g.q_heads / g.kv_heads + 15) / 16;
@@ -485,8 +556,8 @@ int launch_decode(const void* q, const Source& src, const Form& f, const int*, c
   attributes[1].val.programmaticStreamSerializationAllowed = 1;
   config.attrs = attributes;
   config.numAttrs = g_lrm_pdl ? 2 : 1;
-  e = cudaLaunchKernelEx(&config, kernel, static_cast<const __nv_bfloat16*>(q), src, f, g.q_heads, g.kv_heads, row_groups,
-                         g.d, g.dv);
+  e = cudaLaunchKernelEx(&config, kernel, static_cast<const __nv_bfloat16*>(q), src, f, g.fresh, g.q_heads, g.kv_heads,
+                         row_groups, g.d, g.dv);
   return e == cudaSuccess ? 0 : static_cast<int>(e);
 }
 
@@ -585,7 +656,34 @@ LRM_API int lrm_attention_gated(const void* q, const void* k, const void* v, con
       (reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v)) % 16 != 0)
     return LRM_UNSUPPORTED;
   const Source src{k, v, page_table, table_stride, slots, kv_lens};
-  const Geometry g{seqs, max_seq_len, q_heads, kv_heads, d, dv, ranks};
+  const Geometry g{seqs, max_seq_len, q_heads, kv_heads, d, dv, ranks, Fresh{}};
   if (ranks > 0) LRM_BY_SIZES(launch_decode);
   LRM_BY_SIZES(launch_tiled);
+}
+
+// The decode step from the float32 projection on: proj [seqs, stride] holds rows [q_heads * d | kv_heads * d |
+// kv_heads * dv] (`gate`, where there is one, usually their further columns). bias float32 [row] or null; table float32
+// [seqs, rotary / 2, 2] (null with rotary 0); the new key and value go to rows dest_rows [seqs] of the pages.
+LRM_API int lrm_attention_gated_decode_fused(const float* proj, long long stride, const float* bias, const float* table,
+                                             int rotary, void* k_pages, void* v_pages, const int* dest_rows,
+                                             const int* page_table, int table_stride, const int* slots, const int* kv_lens,
+                                             int seqs, int q_heads, int kv_heads, int d, int dv, float scale, float cap,
+                                             int window, int keep, const float* sinks, const float* gate,
+                                             long long gate_stride, int gate_per_head, void* out, long long out_stride,
+                                             float out_scale, int ranks, cudaStream_t stream) {
+  if (seqs <= 0) return 0;
+  const Form f = make_form(scale, cap, window, keep, sinks, gate, gate_stride, gate_per_head, out, out_stride, out_scale);
+  if (bad_form(f, q_heads, kv_heads, d, dv) || ranks < 1 || ranks > 8 || proj == nullptr || dest_rows == nullptr ||
+      page_table == nullptr || slots == nullptr || kv_lens == nullptr || rotary < 0 || rotary % 2 || rotary > d ||
+      (rotary > 0 && table == nullptr) || stride < q_heads * d + static_cast<long long>(kv_heads) * (d + dv))
+    return LRM_BAD_ARGUMENT;
+  if (!lrm_attention_gated_supports(d, dv, kTile) || out_stride % 2 != 0 || reinterpret_cast<uintptr_t>(out) % 4 != 0 ||
+      (reinterpret_cast<uintptr_t>(k_pages) | reinterpret_cast<uintptr_t>(v_pages)) % 16 != 0)
+    return LRM_UNSUPPORTED;
+  const Source src{k_pages, v_pages, page_table, table_stride, slots, kv_lens};
+  const Geometry g{seqs, 1, q_heads, kv_heads, d, dv, ranks,
+                   Fresh{proj, stride, bias, reinterpret_cast<const float2*>(table), rotary, dest_rows}};
+  const void* q = nullptr;
+  const int* cu_seqlens = nullptr;
+  LRM_BY_SIZES(launch_decode);
 }

@@ -55,7 +55,7 @@ __global__ __launch_bounds__(128) void gemm_bf16_mma_kernel(const __nv_bfloat16*
                                                             const __nv_bfloat16* __restrict__ W,
                                                             void* __restrict__ C, int M, int N,
                                                             int K, int mode, int vector_ok, int group_cols,
-                                                            int group_rows) {
+                                                            int group_rows, long long gate_pitch) {
   __shared__ __align__(16) __nv_bfloat16 Xs[BM][BK + PAD];
   __shared__ __align__(16) __nv_bfloat16 Ws[BN][BK + PAD];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -117,7 +117,7 @@ __global__ __launch_bounds__(128) void gemm_bf16_mma_kernel(const __nv_bfloat16*
             if (col + 8 >= N) continue;
             const float gate = acc[i][j][half * 2 + e], up = acc[i][j + 1][half * 2 + e];
             const int out_col = (col / 16) * 8 + (col % 8);
-            static_cast<__nv_bfloat16*>(C)[static_cast<size_t>(row) * (N / 2) + out_col] =
+            static_cast<__nv_bfloat16*>(C)[static_cast<size_t>(row) * gate_pitch + out_col] =
                 __float2bfloat16_rn(silu_f32(gate) * up);
           }
         }
@@ -139,11 +139,9 @@ __global__ __launch_bounds__(128) void gemm_bf16_mma_kernel(const __nv_bfloat16*
     }
   }
 }
-}  // namespace
 
-// group_cols > 0 (a multiple of 64): several inputs `group_rows` rows apart in X.
-LRM_API int lrm_gemm_bf16_mma_grouped(const void* X, const void* W, void* C, int M, int N, int K, int mode,
-                                      int group_cols, int group_rows, cudaStream_t stream) {
+int launch_mma(const void* X, const void* W, void* C, int M, int N, int K, int mode, int group_cols, int group_rows,
+               long long gate_pitch, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (group_cols < 0 || group_cols % BN || (group_cols > 0 && group_rows < M)) return LRM_BAD_ARGUMENT;
   if (K <= 0 || mode < 0 || mode > 3) return LRM_BAD_ARGUMENT;
@@ -154,9 +152,23 @@ LRM_API int lrm_gemm_bf16_mma_grouped(const void* X, const void* W, void* C, int
                        (reinterpret_cast<uintptr_t>(W) % 16 == 0) && (K % 8 == 0);
   gemm_bf16_mma_kernel<<<grid, 128, 0, stream>>>(static_cast<const __nv_bfloat16*>(X),
                                                  static_cast<const __nv_bfloat16*>(W), C, M, N, K,
-                                                 mode, aligned ? 1 : 0, group_cols, group_rows);
+                                                 mode, aligned ? 1 : 0, group_cols, group_rows, gate_pitch);
   LRM_LAUNCH_CHECK();
   return 0;
+}
+}  // namespace
+
+// group_cols > 0 (a multiple of 64): several inputs `group_rows` rows apart in X.
+LRM_API int lrm_gemm_bf16_mma_grouped(const void* X, const void* W, void* C, int M, int N, int K, int mode,
+                                      int group_cols, int group_rows, cudaStream_t stream) {
+  return launch_mma(X, W, C, M, N, K, mode, group_cols, group_rows, N / 2, stream);
+}
+
+// The SiLU gate (mode 3) into rows `pitch` elements apart.
+LRM_API int lrm_gemm_bf16_mma_gate(const void* X, const void* W, void* gated, long long pitch, int M, int N, int K,
+                                   cudaStream_t stream) {
+  if (pitch < N / 2) return LRM_BAD_ARGUMENT;
+  return launch_mma(X, W, gated, M, N, K, 3, 0, 0, pitch, stream);
 }
 
 LRM_API int lrm_gemm_bf16_mma(const void* X, const void* W, void* C, int M, int N, int K, int mode,

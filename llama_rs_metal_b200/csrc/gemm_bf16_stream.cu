@@ -23,6 +23,10 @@
 // begins `rows` rows after input i - 1 in X: one launch for the products of several inputs of equal
 // shape with the rows of one stacked W. A variant of its own: the plain kernel's registers are counted.
 //
+// Two products with one input (SPLIT): output columns below `split` are stored in float32 to `out` [M, split],
+// the columns from it on are gate and up rows (as epilogue 3) whose gated values go to `gated`, rows
+// `pitch` elements apart. A variant of its own for the same reason.
+//
 // Epilogues: 0 store bf16, 1 store f32, 2 add into f32 in place, 3 SiLU gate
 // (rows alternate in blocks of 8 gate / 8 up rows, so a 16-row tile holds 8
 // gated pairs; out is [M, N/2] bf16), 4 store f32 partials per K slice, 5 token choice: the
@@ -75,13 +79,19 @@ struct PickArgs {
   unsigned long long seed;
 };
 
-// Output columns per input and rows of X between inputs (GROUPED).
+enum : int { PLAIN = 0, GROUPED = 1, SPLIT = 2 };  // kinds of the kernel
+
+// GROUPED: output columns per input and rows of X between inputs. SPLIT: the first gate column, and where the
+// gated values go.
 struct Grouped {
   int cols, rows;
+  int split;
+  __nv_bfloat16* gated;
+  long long pitch;
 };
 
 // MINB: CTAs per SM the register budget must allow (a single wave for the usual sizes).
-template <int NT, int WARPS, int MINB, bool GROUPED>
+template <int NT, int WARPS, int MINB, int KIND>
 __global__ __launch_bounds__(WARPS * 32, MINB) void gemm_bf16_stream_kernel(
     const __nv_bfloat16* __restrict__ X, const __nv_bfloat16* __restrict__ W, void* __restrict__ out,
     int M, int N, int K_total, int mode, int k_per_split, PickArgs pick, Grouped grouped) {
@@ -92,8 +102,9 @@ __global__ __launch_bounds__(WARPS * 32, MINB) void gemm_bf16_stream_kernel(
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int g = lane >> 2, t = lane & 3;
   const int n0 = blockIdx.x * 16;
-  if (GROUPED) __builtin_assume(mode >= 0 && mode <= 1);
-  if (GROUPED) X += static_cast<size_t>(n0 / grouped.cols) * grouped.rows * K_total;
+  if (KIND == GROUPED) __builtin_assume(mode >= 0 && mode <= 1);
+  if (KIND == GROUPED) X += static_cast<size_t>(n0 / grouped.cols) * grouped.rows * K_total;
+  if (KIND == SPLIT) __builtin_assume(mode == 6);
   const int k_lo = blockIdx.y * k_per_split;              // this CTA's slice of K: [k_lo, K)
   const int K = min(K_total, k_lo + k_per_split);
   // epilogue 4: this slice's partial product goes to its own [M, N] plane of `out`
@@ -226,6 +237,17 @@ __global__ __launch_bounds__(WARPS * 32, MINB) void gemm_bf16_stream_kernel(
     for (int e = 0; e < 2; ++e) {
       const int m = m0 + e;
       if (m >= M) continue;
+      if (KIND == SPLIT) {  // a tile of 16 columns lies on one side
+        if (n0 < grouped.split) {
+          float* dst = static_cast<float*>(out) + static_cast<size_t>(m) * grouped.split + n0 + gg;
+          dst[0] = vals[e][0];
+          dst[8] = vals[e][1];
+        } else {
+          grouped.gated[static_cast<size_t>(m) * grouped.pitch + ((n0 - grouped.split) >> 1) + gg] =
+              __float2bfloat16_rn(silu_f32(vals[e][0]) * vals[e][1]);
+        }
+        continue;
+      }
       if (mode == 3) {
         const int col = (n0 >> 1) + gg;  // gate row n0+gg pairs with up row n0+gg+8
         if (n0 + gg + 8 < N)
@@ -248,11 +270,11 @@ __global__ __launch_bounds__(WARPS * 32, MINB) void gemm_bf16_stream_kernel(
   }
 }
 
-template <int NT, int WARPS, int MINB, bool GROUPED = false>
+template <int NT, int WARPS, int MINB, int KIND = PLAIN>
 int launch_variant(const void* X, const void* W, void* out, int M, int N, int K, int mode, int splits,
-                   const PickArgs& pick, cudaStream_t stream, const Grouped& grouped = Grouped{0, 0}) {
+                   const PickArgs& pick, cudaStream_t stream, const Grouped& grouped = Grouped{}) {
   constexpr int smem = WARPS * NT * 32 * 4 * static_cast<int>(sizeof(float));
-  auto kernel = gemm_bf16_stream_kernel<NT, WARPS, MINB, GROUPED>;
+  auto kernel = gemm_bf16_stream_kernel<NT, WARPS, MINB, KIND>;
   if (smem > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return static_cast<int>(e);
@@ -300,8 +322,20 @@ int launch_grouped(const void* X, const void* W, void* out, int M, int N, int K,
   constexpr int kWarpsPerSm = NT <= 2 ? 32 : 16;
   // a stack of several matrices has tiles enough: few warps per CTA unless it is small
   if ((N + 15) / 16 >= 148 * 4 || K <= 512)
-    return launch_variant<NT, 4, kWarpsPerSm / 4, true>(X, W, out, M, N, K, mode, 1, PickArgs{}, stream, grouped);
-  return launch_variant<NT, 8, kWarpsPerSm / 8, true>(X, W, out, M, N, K, mode, 1, PickArgs{}, stream, grouped);
+    return launch_variant<NT, 4, kWarpsPerSm / 4, GROUPED>(X, W, out, M, N, K, mode, 1, PickArgs{}, stream, grouped);
+  return launch_variant<NT, 8, kWarpsPerSm / 8, GROUPED>(X, W, out, M, N, K, mode, 1, PickArgs{}, stream, grouped);
+}
+
+template <int NT>
+int launch_split(const void* X, const void* W, void* out, int M, int N, int K, const Grouped& parts, cudaStream_t stream) {
+  constexpr int kWarpsPerSm = NT <= 2 ? 32 : 16;
+  // enough warps in all to fill the SMs, no warp without a chunk of K (launch_rows' rule)
+  const int tiles = (N + 15) / 16, chunks = (K + 127) / 128;
+  int warps = 4;
+  while (warps < (NT <= 4 ? 16 : 8) && tiles * warps < 148 * 16 && warps * 2 <= chunks) warps *= 2;
+  if (warps == 16) return launch_variant<NT, 16, kWarpsPerSm / 16, SPLIT>(X, W, out, M, N, K, 6, 1, PickArgs{}, stream, parts);
+  if (warps == 8) return launch_variant<NT, 8, kWarpsPerSm / 8, SPLIT>(X, W, out, M, N, K, 6, 1, PickArgs{}, stream, parts);
+  return launch_variant<NT, 4, kWarpsPerSm / 4, SPLIT>(X, W, out, M, N, K, 6, 1, PickArgs{}, stream, parts);
 }
 
 }  // namespace
@@ -356,11 +390,27 @@ LRM_API int lrm_gemm_bf16_stream_grouped(const void* X, const void* W, void* out
   if (!lrm_gemm_bf16_stream_supports(M, N, K)) return LRM_UNSUPPORTED;
   if ((mode != 0 && mode != 1) || group_cols <= 0 || group_cols % 16 || group_rows < M) return LRM_BAD_ARGUMENT;
   if (reinterpret_cast<uintptr_t>(X) % 16 || reinterpret_cast<uintptr_t>(W) % 16) return LRM_UNSUPPORTED;
-  const Grouped grouped{group_cols, group_rows};
+  const Grouped grouped{group_cols, group_rows, 0, nullptr, 0};
   if (M <= 8) return launch_grouped<1>(X, W, out, M, N, K, mode, grouped, stream);
   if (M <= 16) return launch_grouped<2>(X, W, out, M, N, K, mode, grouped, stream);
   if (M <= 32) return launch_grouped<4>(X, W, out, M, N, K, mode, grouped, stream);
   return launch_grouped<8>(X, W, out, M, N, K, mode, grouped, stream);
+}
+
+// Two products with one input: out float32 [M, split] and gated (bfloat16, rows `pitch` elements apart) from
+// the gate and up rows behind the first `split` (a multiple of 16) rows of W.
+LRM_API int lrm_gemm_bf16_stream_split(const void* X, const void* W, void* out, int split, void* gated, long long pitch,
+                                       int M, int N, int K, cudaStream_t stream) {
+  if (M <= 0 || N <= 0) return 0;
+  if (!lrm_gemm_bf16_stream_supports(M, N, K)) return LRM_UNSUPPORTED;
+  if (split <= 0 || split % 16 || split >= N || (N - split) % 16 || pitch < (N - split) / 2 || out == nullptr || gated == nullptr)
+    return LRM_BAD_ARGUMENT;
+  if (reinterpret_cast<uintptr_t>(X) % 16 || reinterpret_cast<uintptr_t>(W) % 16) return LRM_UNSUPPORTED;
+  const Grouped parts{0, 0, split, static_cast<__nv_bfloat16*>(gated), pitch};
+  if (M <= 8) return launch_split<1>(X, W, out, M, N, K, parts, stream);
+  if (M <= 16) return launch_split<2>(X, W, out, M, N, K, parts, stream);
+  if (M <= 32) return launch_split<4>(X, W, out, M, N, K, parts, stream);
+  return launch_split<8>(X, W, out, M, N, K, parts, stream);
 }
 
 // The head product with the token choice in its epilogue: ids[m] = the chosen vocabulary row for

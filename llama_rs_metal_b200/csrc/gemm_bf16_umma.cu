@@ -54,7 +54,7 @@ template <int BN, int STAGES, int MT>
 __global__ __launch_bounds__(kUmmaThreads, 1) void gemm_bf16_umma_kernel(
     const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
     void* __restrict__ out, int M, int N, int K, int mode, int kb_per_split, int splits,
-    int* __restrict__ status, const QkvArgs qkv, int group_cols, int group_rows) {
+    int* __restrict__ status, const QkvArgs qkv, const SplitArgs parts, int group_cols, int group_rows) {
   constexpr uint32_t A_BYTES = MT * BM * BK * 2, B_BYTES = BN * BK * 2, STAGE_BYTES = A_BYTES + B_BYTES;
   constexpr uint32_t SET = MT * BN;                      // columns of one set of accumulators
   constexpr uint32_t NBUF = 2 * SET <= 512 ? 2 : 1;      // sets that fit in tensor memory
@@ -203,7 +203,7 @@ __global__ __launch_bounds__(kUmmaThreads, 1) void gemm_bf16_umma_kernel(
           const int m = m0 + (c / (BN / 32)) * BM + quarter * 32 + lane;
           uint32_t r[32];
           tmem_load32(tmem_base + acc * SET + (static_cast<uint32_t>(quarter * 32) << 16) + c * 32, r);
-          store_piece(r, plane, m, n0 + (c % (BN / 32)) * 32, M, N, mode);
+          store_piece(r, plane, m, n0 + (c % (BN / 32)) * 32, M, N, mode, parts);
         }
       }
       tc_fence_before();
@@ -220,7 +220,7 @@ __global__ __launch_bounds__(kUmmaThreads, 1) void gemm_bf16_umma_kernel(
 template <int BN, int STAGES, int MT = 1>
 int launch_umma(const void* X, const void* W, void* out, int M, int x_rows, int N, int K, int mode, int splits,
                 int* status, cudaStream_t stream, const QkvArgs& qkv = QkvArgs{}, int group_cols = 0,
-                int group_rows = 0) {
+                int group_rows = 0, const SplitArgs& parts = SplitArgs{}) {
   CUtensorMap map_x, map_w;
   if (!make_map_bf16(&map_x, X, x_rows, K, BM) || !make_map_bf16(&map_w, W, N, K, BN)) return LRM_UNSUPPORTED;
   constexpr int smem = STAGES * (MT * BM * BK * 2 + BN * BK * 2) + 1024 + 256;
@@ -240,7 +240,7 @@ int launch_umma(const void* X, const void* W, void* out, int M, int x_rows, int 
   }
   const int grid = static_cast<int>(items < sm_count ? items : sm_count);
   LRM_LAUNCH(kernel, dim3(grid), kUmmaThreads, smem, stream, map_x, map_w, out, M, N, K, mode, kb_per_split, real_splits,
-             status, qkv, group_cols, group_rows);
+             status, qkv, parts, group_cols, group_rows);
   return 0;
 }
 
@@ -282,6 +282,27 @@ LRM_API int lrm_gemm_bf16_umma_rows(const void* X, const void* W, void* out, int
   if (tile == 2) return launch_umma<256, 3, 2>(X, W, out, M, x_rows, N, K, mode, splits, status, stream);
   if (tile == 1) return launch_umma<256, 4>(X, W, out, M, x_rows, N, K, mode, splits, status, stream);
   return launch_umma<128, 6>(X, W, out, M, x_rows, N, K, mode, splits, status, stream);
+}
+
+// Epilogue 6: columns below `split` in float32 to out [M, split], the gate and up columns behind it gated to
+// `gated` (bfloat16, rows `pitch` elements apart). split a multiple of 32, the columns behind it and the pitch
+// multiples of 16 and 8.
+LRM_API int lrm_gemm_bf16_umma_split(const void* X, const void* W, void* out, int split, void* gated, long long pitch,
+                                     int M, int x_rows, int N, int K, int tile, int* status, cudaStream_t stream) {
+  if (M <= 0 || N <= 0) return 0;
+  if (!lrm_gemm_bf16_umma_supports(M, N, K)) return LRM_UNSUPPORTED;
+  if (split <= 0 || split % 32 || split >= N || (N - split) % 16 || pitch % 8 || pitch < (N - split) / 2 || x_rows < M ||
+      out == nullptr || gated == nullptr || status == nullptr || tile < 0 || tile > 3)
+    return LRM_BAD_ARGUMENT;
+  if ((reinterpret_cast<uintptr_t>(X) | reinterpret_cast<uintptr_t>(W) | reinterpret_cast<uintptr_t>(out) |
+       reinterpret_cast<uintptr_t>(gated)) % 16)
+    return LRM_UNSUPPORTED;
+  const QkvArgs none{};
+  const SplitArgs parts{static_cast<__nv_bfloat16*>(gated), pitch, split};
+  if (tile == 3) return launch_umma<192, 5>(X, W, out, M, x_rows, N, K, 6, 1, status, stream, none, 0, 0, parts);
+  if (tile == 2) return launch_umma<256, 3, 2>(X, W, out, M, x_rows, N, K, 6, 1, status, stream, none, 0, 0, parts);
+  if (tile == 1) return launch_umma<256, 4>(X, W, out, M, x_rows, N, K, 6, 1, status, stream, none, 0, 0, parts);
+  return launch_umma<128, 6>(X, W, out, M, x_rows, N, K, 6, 1, status, stream, none, 0, 0, parts);
 }
 
 // Several inputs of M rows each in one launch (mode 0 or 1): input i begins i * group_rows rows into X

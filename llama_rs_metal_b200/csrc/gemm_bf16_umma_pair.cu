@@ -95,7 +95,7 @@ template <int BN, int STAGES>
 __global__ __launch_bounds__(kPairThreads, 1) void gemm_bf16_umma_pair_kernel(
     const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
     void* __restrict__ out, int M, int N, int K, int mode, int* __restrict__ status, const QkvArgs qkv,
-    int group_cols, int group_rows) {
+    const SplitArgs parts, int group_cols, int group_rows) {
   constexpr uint32_t A_BYTES = PM * PK * 2, B_BYTES = (BN / 2) * PK * 2, STAGE_BYTES = A_BYTES + B_BYTES;
   constexpr uint32_t ALLOC = 512, SET = 256;  // two sets of accumulators, 256 columns apart
   static_assert(BN % 32 == 0 && BN >= 64 && BN <= 256, "BN / 2 rows of W per CTA, a multiple of 16");
@@ -222,7 +222,7 @@ __global__ __launch_bounds__(kPairThreads, 1) void gemm_bf16_umma_pair_kernel(
         for (int c = side * (BN / 64); c < (side + 1) * (BN / 64); ++c) {
           uint32_t r[32];
           tmem_load32(tmem_base + acc * SET + (static_cast<uint32_t>(quarter * 32) << 16) + c * 32, r);
-          store_piece(r, out, m0 + quarter * 32 + lane, n0 + c * 32, M, N, mode);
+          store_piece(r, out, m0 + quarter * 32 + lane, n0 + c * 32, M, N, mode, parts);
         }
       }
       tc_fence_before();
@@ -282,7 +282,7 @@ template <int BN, int STAGES> int resident_pairs() {
 template <int BN, int STAGES>
 int launch_pair(const void* X, const void* W, void* out, int M, int N, int K, int mode, int* status,
                 cudaStream_t stream, const QkvArgs& qkv = QkvArgs{}, int x_rows = 0, int group_cols = 0,
-                int group_rows = 0) {
+                int group_rows = 0, const SplitArgs& parts = SplitArgs{}) {
   const int room = resident_pairs<BN, STAGES>();
   if (room <= 0) return LRM_UNSUPPORTED;
   CUtensorMap map_x, map_w;
@@ -294,7 +294,7 @@ int launch_pair(const void* X, const void* W, void* out, int M, int N, int K, in
   int code = pair_config<BN, STAGES>(config, attributes, 2 * pairs, stream);
   if (code != 0) return code;
   cudaError_t e = cudaLaunchKernelEx(&config, gemm_bf16_umma_pair_kernel<BN, STAGES>, map_x, map_w, out, M, N, K,
-                                     mode, status, qkv, group_cols, group_rows);
+                                     mode, status, qkv, parts, group_cols, group_rows);
   return e == cudaSuccess ? 0 : static_cast<int>(e);
 }
 
@@ -318,6 +318,21 @@ LRM_API int lrm_gemm_bf16_umma_pair(const void* X, const void* W, void* out, int
   if (mode < 0 || mode > 3 || (mode == 3 && N % 16 != 0) || status == nullptr) return LRM_BAD_ARGUMENT;
   if (reinterpret_cast<uintptr_t>(X) % 16 || reinterpret_cast<uintptr_t>(W) % 16) return LRM_UNSUPPORTED;
   return launch_pair<256, 6>(X, W, out, M, N, K, mode, status, stream);
+}
+
+// Epilogue 6 on pairs of SMs, as lrm_gemm_bf16_umma_split.
+LRM_API int lrm_gemm_bf16_umma_pair_split(const void* X, const void* W, void* out, int split, void* gated, long long pitch,
+                                          int M, int N, int K, int* status, cudaStream_t stream) {
+  if (M <= 0 || N <= 0) return 0;
+  if (K < 8 || K % 8 != 0 || encode_tiled() == nullptr) return LRM_UNSUPPORTED;
+  if (split <= 0 || split % 32 || split >= N || (N - split) % 16 || pitch % 8 || pitch < (N - split) / 2 || out == nullptr ||
+      gated == nullptr || status == nullptr)
+    return LRM_BAD_ARGUMENT;
+  if ((reinterpret_cast<uintptr_t>(X) | reinterpret_cast<uintptr_t>(W) | reinterpret_cast<uintptr_t>(out) |
+       reinterpret_cast<uintptr_t>(gated)) % 16)
+    return LRM_UNSUPPORTED;
+  return launch_pair<256, 6>(X, W, out, M, N, K, 6, status, stream, QkvArgs{}, 0, 0, 0,
+                             SplitArgs{static_cast<__nv_bfloat16*>(gated), pitch, split});
 }
 
 // Several inputs in one launch, as lrm_gemm_bf16_umma_grouped; group_cols a multiple of 256.

@@ -2,6 +2,7 @@
 // (shared by the single-CTA kernel and the kernel that runs pairs of CTAs):
 //   0 store bfloat16, 1 store float32, 2 add into float32 in place (residual stream),
 //   3 SiLU gate over alternating blocks of 8 gate / 8 up columns, 4 store float32 (a K slice's plane),
+//   6 columns below a split as 1, the columns from it on as 3, each into a tensor of its own (SplitArgs),
 // and epilogue 5, which works on whole heads of a fused q|k|v projection (store_heads).
 #pragma once
 #include "umma.cuh"
@@ -10,14 +11,36 @@ namespace {
 
 __device__ __forceinline__ float silu_f32(float g) { return g / (1.0f + expf(-g)); }
 
+// What epilogue 6 needs: two products with the same input in one launch. Columns [0, split) are stored in
+// float32 to `out` [M, split]; columns from `split` (a multiple of 32) on are gate and up rows, and the
+// gated values go to `gated`, whose rows are `pitch` elements apart.
+struct SplitArgs {
+  __nv_bfloat16* gated;
+  long long pitch;
+  int split;
+};
+
 // The epilogue of one 32-column piece of an accumulator row held in registers.
 __device__ __forceinline__ void store_piece(const uint32_t (&r)[32], void* __restrict__ out, int m, int n,
-                                            int M, int N, int mode) {
+                                            int M, int N, int mode, const SplitArgs& parts) {
   if (m >= M || n >= N) return;
+  size_t pitch = N >> 1;  // of the gated values
+  if (mode == 6) {
+    if (n < parts.split) {
+      mode = 1;
+      N = parts.split;
+    } else {
+      mode = 3;
+      n -= parts.split;
+      N -= parts.split;
+      out = parts.gated;
+      pitch = parts.pitch;
+    }
+  }
   const bool whole = n + 32 <= N;
   if (mode == 3) {
     // [8 gate | 8 up | 8 gate | 8 up] -> 16 gated values
-    __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(out) + static_cast<size_t>(m) * (N >> 1) + (n >> 1);
+    __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(out) + static_cast<size_t>(m) * pitch + (n >> 1);
     uint32_t packed[8];
 #pragma unroll
     for (int i = 0; i < 16; i += 2) {

@@ -39,6 +39,7 @@ force_unfused_decode = False  # tests keep decode steps on the separate rotation
 force_cluster_size = None  # tests fix the CTAs per cluster of the fused decode kernel
 force_shared_key_splits = None  # tests fix the splits of the shared-key kernel's decode step
 force_sigmoid_ranks = None  # tests fix the CTAs per cluster of the sigmoid decode kernel
+force_gated_split = False  # tests keep decode steps of that kernel behind a split of the projection in its own launch
 force_gated_ranks = None  # tests fix the CTAs per cluster of the gated softmax kernel's decode step
 prefill_kernel = None  # tests pin the tcgen05 prompt kernel: "pingpong" or "single" (None: the rule in prefill())
 
@@ -329,6 +330,23 @@ def sigmoid(q, k, v, kv, kv_heads: int, dv: int, out, out_stride: int, offset, g
                                             kv_heads, d, dv, page_size, *tail, _stream()), "attention_sigmoid_rowwise")
 
 
+def gated_ranks(seqs: int, kv_heads: int, group: int, max_kv_len: int, window: int, keep_first: int) -> int:
+    """CTAs of a cluster that share a sequence's pages: about two CTAs per SM, no CTA without a page."""
+    if force_gated_ranks is not None:
+        return force_gated_ranks
+    seen = min(max_kv_len, abs(window) + 63 + keep_first) if window else max_kv_len
+    return max(1, min(8, -(-seen // 64), -(-2 * SM_COUNT // (seqs * kv_heads * -(-group // 16)))))
+
+
+def gated_decode_fused_supported(dtype, d: int, dv: int, kv, shaping: Shaping) -> bool:
+    """True when the decode kernel can begin at the float32 projection: biases and a split-half rotation are
+    all that stands between it and the attention."""
+    return (not force_rowwise and not force_gated_split and dtype == torch.bfloat16 and kv is not None
+            and shaping.taps is None and shaping.row_norm is None and shaping.head_weights is None
+            and shaping.head_norm_eps is None and not shaping.adjacent_pairs
+            and bool(library.load().lrm_attention_gated_supports(d, dv, kv.page_size)))
+
+
 def gated(q, k, v, kv, kv_heads: int, dv: int, out, out_stride: int, form, gate, gate_stride: int, scale: float,
           window: int, out_scale: float, max_seq_len: int, max_kv_len: int, cu_seqlens, seq_of_token, positions, slots,
           kv_lens) -> None:
@@ -348,12 +366,7 @@ def gated(q, k, v, kv, kv_heads: int, dv: int, out, out_stride: int, form, gate,
             and out_stride % 2 == 0 and all(t.data_ptr() % 16 == 0 for t in (q, keys, values)) and out.value % 4 == 0):
         ranks = 0
         if one_each:
-            # the CTAs of a cluster share a sequence's pages; about two CTAs per SM, no CTA without a page
-            seen = min(max_kv_len, abs(window) + 63 + form.keep_first) if window else max_kv_len
-            clusters = T * kv_heads * -(-(Hq // kv_heads) // 16)
-            ranks = max(1, min(8, -(-seen // 64), -(-2 * SM_COUNT // clusters)))
-            if force_gated_ranks is not None:
-                ranks = force_gated_ranks
+            ranks = gated_ranks(T, kv_heads, Hq // kv_heads, max_kv_len, window, form.keep_first)
         _done(lib.lrm_attention_gated(_ptr(q), _ptr(keys), _ptr(values), _ptr(None if one_each else cu_seqlens), *pages,
                                       T if one_each else cu_seqlens.numel() - 1, max_seq_len, Hq, kv_heads, d, dv, *tail,
                                       ranks, _stream()), "attention_gated_decode" if one_each else "attention_gated")
@@ -501,11 +514,17 @@ def attend(projected, *, q_heads: int, kv_heads: int, head_dim: int, rotary, ctx
         if shaping is not None:
             s = shaping
             table = None
+            in_one = (form is not None and phase == "decode" and writes_cache and projected.dtype == torch.float32
+                      and gated_decode_fused_supported(ctx.runtime.dtype, head_dim, dv, cache, s))
             if s.inv_freq is not None:  # one table of angles per step and set of frequencies
                 key = ("rope_table64", s.inv_freq.data_ptr(), s.magnitude)
                 table = ctx.scratch.get(key)
                 if table is None:
                     table = ctx.scratch[key] = ops.rope_table64(ctx.positions, s.inv_freq, s.magnitude)
+            if in_one:  # biases, rotation, cache write and attention in one launch
+                return ops.attention_gated_decode_fused(
+                    projected, bias, table, s.rotary, q_heads, dv, form, cache, ctx.dest_rows[cache.group], ctx.slots,
+                    ctx.kv_lens, ctx.max_kv_len, scale, window, out_scale)
             q, k, v = ops.shaped_qkv_store(
                 projected, q_heads, kv_heads if writes_cache else 0, head_dim, dv, ctx.positions, ctx.runtime.dtype,
                 bias=bias, taps=s.taps, tails=s.tails.state if s.tails is not None else None,

@@ -15,6 +15,7 @@
 """
 from __future__ import annotations
 
+import ctypes
 from typing import Dict, Optional
 
 import torch
@@ -305,6 +306,36 @@ def gemm_bf16(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, mode: in
         return
     _done(lib.lrm_gemm_bf16_mma(_ptr(x), _ptr(weight), _ptr(out), M, N, K, mode, _stream()),
           "gemm_bf16_mma")
+
+
+def gemm_bf16_split(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gated: torch.Tensor) -> None:
+    """Two products with one input: out (float32 [M, split]) = x . weight[:split]^T, and the SiLU gate of the gate
+    and up rows behind it into the first columns of `gated` (bfloat16 [M, W]). One launch of the kernels of
+    gemm_bf16; two where only the warp-level kernel takes the shape."""
+    M, K = x.shape
+    N, split, pitch = weight.shape[0], out.shape[1], gated.shape[1]
+    lib = library.load()
+    stream_ok, umma_ok = _fast_kernels(x, weight, lib)
+    if stream_ok and umma_ok and M > STREAM_ROWS and not force_stream:
+        stream_ok = not _few_rows_plan(M, N, K, 6)[0]
+    where = (_ptr(x), _ptr(weight), _ptr(out), split, _ptr(gated), ctypes.c_longlong(pitch), M)
+    if stream_ok:
+        _done(lib.lrm_gemm_bf16_stream_split(*where, N, K, _stream()), "gemm_bf16_stream_split")
+        return
+    if umma_ok and pitch % 8 == 0:
+        tile = tile_choice(M, N, K, 1, pair_room() if M > 64 else 0)
+        mark_status_dirty()
+        if tile == PAIR:
+            _done(lib.lrm_gemm_bf16_umma_pair_split(*where, N, K, _ptr(_status_word(x.device)), _stream()),
+                  "gemm_bf16_umma_pair_split")
+            return
+        held = (x.untyped_storage().nbytes() // x.element_size() - x.storage_offset()) // K
+        _done(lib.lrm_gemm_bf16_umma_split(*where, min(max(M, 32), max(M, held)), N, K, tile, _ptr(_status_word(x.device)),
+                                           _stream()), "gemm_bf16_umma_split")
+        return
+    _done(lib.lrm_gemm_bf16_mma(_ptr(x), _ptr(weight), _ptr(out), M, split, K, 1, _stream()), "gemm_bf16_mma")
+    _done(lib.lrm_gemm_bf16_mma_gate(_ptr(x), _ptr(weight[split:]), _ptr(gated), ctypes.c_longlong(pitch), M, N - split, K,
+                                     _stream()), "gemm_bf16_mma_gate")
 
 
 def gemm_bf16_grouped(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, group_cols: int) -> None:

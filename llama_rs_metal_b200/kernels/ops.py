@@ -326,6 +326,28 @@ def linear(x: torch.Tensor, weight: torch.Tensor, epilogue: str = STORE,
     return out
 
 
+SPLIT_MULTIPLE = 32  # where the columns of linear_split divide: whole pieces of a product's epilogue
+
+
+def linear_split(x: torch.Tensor, weight: torch.Tensor, split: int, gated: torch.Tensor) -> torch.Tensor:
+    """Two products with one bfloat16 input x [M, K] in one launch. Rows 0 .. split - 1 of weight (a multiple of
+    SPLIT_MULTIPLE) give the result, float32 [M, split]; the rows behind them alternate in blocks of 8 gate / 8 up
+    rows, and silu(gate) * up goes to the first columns of `gated` (bfloat16 [M, W])."""
+    _check(x, "x", torch.bfloat16, 2)
+    _check(weight, "weight", torch.bfloat16, 2)
+    _check(gated, "gated", torch.bfloat16, 2)
+    M, K = x.shape
+    N = weight.shape[0]
+    if weight.shape[1] != K or gated.shape[0] != M:
+        raise InvalidError("linear_split: shapes do not agree")
+    if not 0 < split < N or split % SPLIT_MULTIPLE or (N - split) % 16 or (N - split) // 2 > gated.shape[1]:
+        raise InvalidError("linear_split: the columns do not divide there, or the gated ones do not fit")
+    out = torch.empty((M, split), dtype=torch.float32, device=x.device)
+    from . import gemm_dispatch
+    gemm_dispatch.gemm_bf16_split(x, weight, out, gated)
+    return out
+
+
 GROUP_MULTIPLE = 128  # a grouped product's columns per input are a multiple of this: whole tiles of one input
 
 
@@ -1786,6 +1808,15 @@ class SoftmaxForm:
     out: Optional[Tuple[torch.Tensor, int]] = None
 
 
+def _check_form(what: str, form: SoftmaxForm, heads: int) -> None:
+    if form.sinks is not None:
+        _check(form.sinks, "sinks", torch.float32, 1)
+        if form.sinks.numel() != heads:
+            raise InvalidError(f"{what}: one sink per query head")
+    if (form.cap is not None and form.cap <= 0) or form.keep_first < 0:
+        raise InvalidError(f"{what}: a cap is positive, and so is the number of kept keys")
+
+
 def attention_gated(q: torch.Tensor, form: SoftmaxForm, scale: float, window: Optional[int], out_scale: float,
                     max_seq_len: int, k: Optional[torch.Tensor] = None, v: Optional[torch.Tensor] = None, kv=None,
                     cu_seqlens: Optional[torch.Tensor] = None, seq_of_token: Optional[torch.Tensor] = None,
@@ -1795,18 +1826,59 @@ def attention_gated(q: torch.Tensor, form: SoftmaxForm, scale: float, window: Op
     come from is told as for attention_sigmoid; `window` > 0 a window, < 0 a chunk."""
     what = "attention_gated"
     T, Hq, d, heads, dv = _attention_geometry(what, q, k, v, kv, cu_seqlens, seq_of_token, slots, kv_lens)
-    if form.sinks is not None:
-        _check(form.sinks, "sinks", torch.float32, 1)
-        if form.sinks.numel() != Hq:
-            raise InvalidError(f"{what}: one sink per query head")
-    if (form.cap is not None and form.cap <= 0) or form.keep_first < 0:
-        raise InvalidError(f"{what}: a cap is positive, and so are kept keys")
+    _check_form(what, form, Hq)
     gate, gate_stride = _gate_columns(what, form.gate, T, Hq if form.gate_per_head else Hq * dv)
     given, column = form.out if form.out is not None else (None, 0)
     out, out_ptr = _output_columns(given, column, T, Hq * dv, q.dtype, q.device)
     from . import attention_dispatch
     attention_dispatch.gated(q, k, v, kv, heads, dv, out_ptr, out.shape[1], form, gate, gate_stride, scale, window or 0,
                              out_scale, max_seq_len, max_kv_len, cu_seqlens, seq_of_token, positions, slots, kv_lens)
+    return out
+
+
+def attention_gated_decode_fused(projected: torch.Tensor, bias: Optional[torch.Tensor], table: Optional[torch.Tensor],
+                                 rotary: int, q_heads: int, value_dim: int, form: SoftmaxForm, kv, dest_rows: torch.Tensor,
+                                 slots: torch.Tensor, kv_lens: torch.Tensor, max_kv_len: int, scale: float,
+                                 window: Optional[int], out_scale: float = 1.0) -> torch.Tensor:
+    """A bfloat16 decode step's attention of the form `form` from the float32 projection [B, Hq*d + Hk*d + Hk*dv
+    (+ more)] on, in one launch: `bias` (float32 [row]), the split-half rotation by `table` (rope_table64 of the
+    step, [B, rotary/2, 2]), the new key and value into the cache view, attention. -> [B, Hq*dv]."""
+    what = "attention_gated_decode_fused"
+    _check(projected, "projected", torch.float32, 2)
+    B, d, heads = projected.shape[0], kv.head_dim, kv.kv_heads
+    row = q_heads * d + heads * (d + value_dim)
+    if projected.shape[1] < row or q_heads % heads or _value_dim(kv) != value_dim:
+        raise InvalidError(f"{what}: the projection does not match the head geometry")
+    _check(kv.k, "k pages", torch.bfloat16, 4)
+    _check(kv.v, "v pages", torch.bfloat16, 4)
+    _check(kv.page_table, "page table", torch.int32, 2)
+    if tuple(kv.k.shape[1:]) != (heads, kv.page_size, d) or tuple(kv.v.shape[1:]) != (heads, kv.page_size, value_dim):
+        raise InvalidError(f"{what}: cache pages do not match the head geometry")
+    for name, t in (("dest_rows", dest_rows), ("slots", slots), ("kv_lens", kv_lens)):
+        _check(t, name, torch.int32, 1)
+        if t.numel() != B:
+            raise InvalidError(f"{what}: one token per sequence")
+    if bias is not None:
+        _check(bias, "bias", torch.float32, 1)
+        if bias.numel() != row:
+            raise InvalidError(f"{what}: one bias per projected column")
+    if rotary:
+        _check(table, "table", torch.float32, 3)
+        if tuple(table.shape) != (B, rotary // 2, 2):
+            raise InvalidError(f"{what}: the table has one angle per sequence and rotated pair")
+    _check_form(what, form, q_heads)
+    gate, gate_stride = _gate_columns(what, form.gate, B, q_heads if form.gate_per_head else q_heads * value_dim)
+    given, column = form.out if form.out is not None else (None, 0)
+    out, out_ptr = _output_columns(given, column, B, q_heads * value_dim, torch.bfloat16, projected.device)
+    from . import attention_dispatch
+    window = window or 0
+    ranks = attention_dispatch.gated_ranks(B, heads, q_heads // heads, max_kv_len, window, form.keep_first)
+    _done(_lib().lrm_attention_gated_decode_fused(
+        _ptr(projected), ctypes.c_longlong(projected.shape[1]), _ptr(bias), _ptr(table if rotary else None), rotary,
+        _ptr(kv.k), _ptr(kv.v), _ptr(dest_rows), _ptr(kv.page_table), kv.page_table.shape[1], _ptr(slots), _ptr(kv_lens), B,
+        q_heads, heads, d, value_dim, ctypes.c_float(scale), ctypes.c_float(form.cap or 0.0), window, form.keep_first,
+        _ptr(form.sinks), gate, ctypes.c_longlong(gate_stride), int(form.gate_per_head), out_ptr,
+        ctypes.c_longlong(out.shape[1]), ctypes.c_float(out_scale), ranks, _stream()), what)
     return out
 
 

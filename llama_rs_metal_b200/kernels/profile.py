@@ -47,6 +47,32 @@ def _out_elem(mode) -> int:
     return {0: 2, 1: 4, 2: 8, 3: 1, 4: 4}.get(int(mode), 4)  # add: read and write; gate: half the columns
 
 
+def _split_gemm(a, N, K):
+    M, split = _v(a[6]), _v(a[3])
+    return 2.0 * (M * K + N * K) + 4.0 * M * split + 1.0 * M * (N - split), 2.0 * M * N * K
+
+
+def _visible(position: int, window: int, keep: int) -> int:
+    """Keys that the query at `position` sees under a window (> 0) or chunk (< 0) beside the first `keep`."""
+    if window == 0:
+        return position + 1
+    first = max(0, position - window + 1) if window > 0 else position - position % -window
+    return position + 1 - first + min(keep, first)
+
+
+def _visible_keys(window, keep) -> float:
+    """Cached keys a step's sequences read, all of a sequence's queries together."""
+    total = 0
+    for before, n in hints["sequences"]:
+        newest = _visible(before + n - 1, int(window), int(keep))
+        total += min(before + n, newest + n - 1) if n > 1 else newest
+    return float(total)
+
+
+def _visible_pairs(window, keep) -> float:
+    return float(sum(_visible(p, int(window), int(keep)) for before, n in hints["sequences"] for p in range(before, before + n)))
+
+
 # entry point -> (bytes, flops) from its positional arguments
 WORK: Dict[str, Callable[..., Tuple[float, float]]] = {
     "lrm_embed_rows": lambda a: (_v(a[4]) * _v(a[5]) * (_ELEM[_v(a[1])] + 4), 0),
@@ -154,9 +180,9 @@ WORK: Dict[str, Callable[..., Tuple[float, float]]] = {
         _v(a[18]) * _v(a[19]) * ((3 * _v(a[20]) + _v(a[21])) * _ELEM[_v(a[1])] + 4.0 * (6 * _v(a[20]) + _v(a[21]))), 0),
     # the shaped split: the projection row read (taps times, from cache), q, k, v written, k and v again into the cache
     "lrm_shaped_qkv_store": lambda a: (
-        _v(a[30]) * ((_v(a[31]) * _v(a[33]) + _v(a[32]) * (_v(a[33]) + _v(a[34]))) * (_ELEM[_v(a[1])] + _ELEM[_v(a[29])])
-                     + _v(a[32]) * (_v(a[33]) + _v(a[34])) * _ELEM[_v(a[29])]),
-        2.0 * _v(a[30]) * (_v(a[31]) * _v(a[33]) + _v(a[32]) * (_v(a[33]) + _v(a[34]))) * max(1, _v(a[5]))),
+        _v(a[31]) * ((_v(a[32]) * _v(a[34]) + _v(a[33]) * (_v(a[34]) + _v(a[35]))) * (_ELEM[_v(a[1])] + _ELEM[_v(a[30])])
+                     + _v(a[33]) * (_v(a[34]) + _v(a[35])) * _ELEM[_v(a[30])]),
+        2.0 * _v(a[31]) * (_v(a[32]) * _v(a[34]) + _v(a[33]) * (_v(a[34]) + _v(a[35]))) * max(1, _v(a[5]))),
     "lrm_token_shift": lambda a: (_v(a[8]) * _v(a[9]) * 2.0 * _ELEM[_v(a[1])], 0),
     "lrm_scaled_add": lambda a: (12.0 * _v(a[3]) * _v(a[4]), 0),
     "lrm_row_gate": lambda a: (_v(a[4]) * (_v(a[5]) * _ELEM[_v(a[2])] + (8.0 + 4.0 * _v(a[8])) * _v(a[6])), 0),
@@ -193,6 +219,22 @@ WORK: Dict[str, Callable[..., Tuple[float, float]]] = {
     "lrm_attention_sigmoid_decode": lambda a: (2.0 * hints["kv_tokens"] * _v(a[11]) * _v(a[12]) * 2, 0),
     "lrm_attention_sigmoid_rowwise": lambda a: (
         (2.0 * hints["kv_tokens"] * _v(a[15]) * _v(a[16]) * _ELEM[_v(a[4])], 0) if a[9] else (0, 4.0 * hints["pairs"] * _v(a[14]) * _v(a[16]))),
+    # two products with one input: the plain columns stored in float32, the gated half of the others in bfloat16
+    "lrm_gemm_bf16_stream_split": lambda a: _split_gemm(a, _v(a[7]), _v(a[8])),
+    "lrm_gemm_bf16_umma_split": lambda a: _split_gemm(a, _v(a[8]), _v(a[9])),
+    "lrm_gemm_bf16_umma_pair_split": lambda a: _split_gemm(a, _v(a[7]), _v(a[8])),
+    "lrm_gemm_bf16_mma_gate": lambda a: _gemm(_v(a[4]), _v(a[5]), _v(a[6]), 1),
+    # gated softmax attention, by the (query, key) pairs and the cached keys that its window or chunk shows:
+    # prompts q, k, v, the gate and the result once; portions and decode steps the visible keys and values
+    "lrm_attention_gated": lambda a: (
+        (_visible_keys(_v(a[16]), _v(a[17])) * _v(a[11]) * (_v(a[12]) + _v(a[13])) * 2.0 if a[4] and a[4].value
+         else 2.0 * hints["tokens"] * (_v(a[10]) + _v(a[11])) * (_v(a[12]) + _v(a[13]))),
+        2.0 * _visible_pairs(_v(a[16]), _v(a[17])) * _v(a[10]) * (_v(a[12]) + _v(a[13]))),
+    "lrm_attention_gated_decode_fused": lambda a: (
+        _visible_keys(_v(a[19]), _v(a[20])) * _v(a[14]) * (_v(a[15]) + _v(a[16])) * 2.0,
+        2.0 * _visible_pairs(_v(a[19]), _v(a[20])) * _v(a[13]) * (_v(a[15]) + _v(a[16]))),
+    "lrm_attention_gated_rowwise": lambda a: (
+        0, 2.0 * _visible_pairs(_v(a[18]), _v(a[19])) * _v(a[12]) * (_v(a[14]) + _v(a[15]))),
     "lrm_tanh_columns": lambda a: (_v(a[5]) * _v(a[6]) * (_ELEM[_v(a[1])] + _ELEM[_v(a[4])]), 0),
 }
 # entry points that only answer questions and launch nothing

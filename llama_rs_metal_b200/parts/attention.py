@@ -226,6 +226,9 @@ class Attention(Mixer):
     def projection(self) -> Optional[LinearWeight]:
         return self.qkv if self.shaped else None
 
+    def give_up_products(self) -> None:
+        self.qkv = self.q_only = self.out = None
+
     def mix(self, x, ctx, cache, out=None, column=0):
         """Projection in float32, then bias, convolution, norms and rotation in one kernel that also
         splits and stores, then attention under the window or the chunk."""

@@ -269,6 +269,10 @@ class Mixer(Part):
         """mix() from columns 0 .. of `projected`, float32 [T, at least projection.out_features]."""
         raise NotImplementedError
 
+    def give_up_products(self) -> None:
+        """Whoever joined this mixer's projection and output product with others makes them from now on:
+        only mix_projected() is called, and the mixer may let go of its matrices."""
+
     def cache_request(self):
         """KeyValueRequest, StateRequest, CompositeRequest or None."""
         return None

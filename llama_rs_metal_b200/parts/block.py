@@ -10,6 +10,8 @@ from ..kernels import ops
 from ..registry import register_block
 from ..weights.loader import TensorSpec
 from .base import Block, CompositeRequest, StateRequest
+from .linear import LinearWeight, SplitLinear
+from .mlp import GatedMLP
 from .norm import StreamCast
 
 STREAM_ITSELF = StreamCast()  # what a block whose sublayers read the stream itself has for an entry norm
@@ -99,7 +101,11 @@ class PreNormMixerBlock(_PreNormBlock):
 class _ParallelBlock(Block):
     """One norm whose output every sublayer reads: hidden += mixer(x) + feed_forward(x), x = norm(hidden).
 
-    A bias of the mixer's output rides in the norm's pass over the stream (Norm.forward_add)."""
+    Where the mixer can make its mixed heads from one product of its input (Mixer.projection, mix_projected), the
+    sublayers are joined under bfloat16: one product makes the mixer's projection and the gated values of the
+    feed-forward, the latter into the row that the mixed heads are then written beside, and one product with
+    [W_down | W_out] makes both outputs and their sum. A bias of the mixer's output then rides in the norm's pass
+    over the stream (Norm.forward_add)."""
 
     graph_safe = True
 
@@ -114,8 +120,44 @@ class ParallelBlock(_ParallelBlock):
 
     roles = {"mixer": "mixer", "feed_forward": "feed_forward", "norm": "norm"}
 
+    def __init__(self, **parts):
+        super().__init__(**parts)
+        self.into: Optional[SplitLinear] = None  # [projection | gate and up]
+        self.out: Optional[LinearWeight] = None  # [down | mixer's output]
+        self.inner = 0                           # columns of gated values in the joined row
+
+    def bind(self, weights, runtime) -> None:
+        # (a block is bound behind its parts)
+        mixer, ff = self.mixer, self.feed_forward
+        if runtime.dtype != torch.bfloat16 or mixer.projection is None or mixer.mixed_width is None \
+                or not isinstance(ff, GatedMLP) or not ff.gates_in_product:
+            return
+        four = (mixer.projection.weight, mixer.out.weight, ff.gate_up.weight, ff.down.weight)
+        if any(w.dtype != torch.bfloat16 for w in four) or any(n % 8 for n in (four[0].shape[1], mixer.mixed_width)):
+            return  # the products' kernels want rows of whole 16-byte pieces
+        self.inner = ff.intermediate_size
+        self.into = SplitLinear(four[0], four[2])
+        self.out = LinearWeight(torch.cat([four[3], four[1]], dim=1))
+        mixer.give_up_products()
+        ff.gate_up = ff.down = None
+
+    def _joined(self, hidden, ctx, cache, after: bool):
+        if self.mixer.output_bias is not None:
+            x = self.norm.forward_add(hidden, ctx, self.mixer.output_bias)
+        else:
+            x = self.norm.forward(hidden, ctx)
+        row = ops._activation(x.shape[0], self.inner + self.mixer.mixed_width, x.dtype, x.device)
+        projected = self.into(x, row)
+        self.mixer.mix_projected(projected, ctx, cache, row, self.inner)
+        ctx.may_defer = after
+        hidden = self.out(row, epilogue=ops.ADD, out=hidden, ctx=ctx)
+        ctx.may_defer = False
+        return hidden
+
     def forward(self, hidden, ctx, cache):
         after = ctx.next_folds_pending
+        if self.into is not None:
+            return self._joined(hidden, ctx, cache, after)
         x = self.norm.forward(hidden, ctx)
         hidden = self.mixer.forward(x, ctx, cache, residual=hidden)
         ctx.may_defer = after

@@ -71,6 +71,22 @@ class LinearWeight:
         return ops.linear(x, ops.cast(w, x.dtype), epilogue, out, out_dtype)
 
 
+class SplitLinear:
+    """Two products with one input as one launch (ops.linear_split): `plain` [n, in], whose result comes back in
+    float32, and `gate_up` [2 f, in] in alternating blocks of 8 gate / 8 up rows, whose gated values go to the
+    first f columns of a given tensor. `plain` is filled up with rows of zeros to whole pieces: the result has
+    `columns` >= n columns."""
+
+    def __init__(self, plain: torch.Tensor, gate_up: torch.Tensor):
+        multiple = ops.SPLIT_MULTIPLE
+        self.columns = -(-plain.shape[0] // multiple) * multiple
+        pad = torch.zeros((self.columns - plain.shape[0], plain.shape[1]), dtype=plain.dtype, device=plain.device)
+        self.weight = torch.cat([plain, pad, gate_up], dim=0).contiguous()
+
+    def __call__(self, x: torch.Tensor, gated: torch.Tensor) -> torch.Tensor:
+        return ops.linear_split(x, self.weight, self.columns, gated)
+
+
 class GroupedLinear:
     """Several matrices [out_i, in], one input each, as one stacked weight whose products are one launch
     (ops.linear_grouped): every matrix but the last is filled up with rows of zeros to `group_cols`

@@ -51,6 +51,11 @@ class GatedMLP(FeedForward):
         self.gate_up = LinearWeight(fused)
         self.down = LinearWeight(weights["down_proj.weight"])
 
+    @property
+    def gates_in_product(self) -> bool:
+        """True when the gate can be an epilogue of the fused gate and up product (bfloat16)."""
+        return self.activation == "silu" and self.block == GATE_BLOCK
+
     def forward(self, x, ctx, residual):
         if self.activation == "clamped_gate":
             both = self.gate_up(x, out_dtype=torch.float32)
@@ -59,7 +64,7 @@ class GatedMLP(FeedForward):
         if self.activation == "gelu_tanh":
             gated = ops.gelu_tanh_mul(self.gate_up(x, out_dtype=torch.float32), self.block, out_dtype=x.dtype)
             return self.down(gated, epilogue=ops.ADD, out=residual, ctx=ctx)
-        if self.block == GATE_BLOCK and self.gate_up.supports_fused_gate(x.dtype):
+        if self.gates_in_product and self.gate_up.supports_fused_gate(x.dtype):
             gated = self.gate_up(x, epilogue=ops.SILU_GATE)
         else:
             gated = ops.silu_mul(self.gate_up(x), self.block)
