@@ -311,13 +311,13 @@ def tolurax_shape(width, heads, kv_heads, ff, window, layers, vocab=32768):
 
 def munupel_shape(width, heads, kv_heads, ff, window, layers, vocab=32768):
     """A Munupel configuration with layers of a real model's widths (head size 128, values as wide): chunked attention
-    with capped scores (chunks of `window`, half of each head rotated with stretched frequencies) and windowed
+    with capped scores (chunks of 3/2 `window`, half of each head rotated with stretched frequencies) and windowed
     attention with sinks and 64 kept first keys in turn, a dense feed-forward beside each."""
     d = 128
     mlp = dict(kind="dense", ff=ff)
     sizes = dict(heads=heads, kv_heads=kv_heads, dim=d, vdim=d, scale=d ** -0.5)
     kinds = [
-        dict(type="attention", mlp=mlp, mixer=dict(sizes, softcap=30.0, mask=dict(size=window), rot=dict(
+        dict(type="attention", mlp=mlp, mixer=dict(sizes, softcap=30.0, mask=dict(size=3 * window // 2), rot=dict(
             dims=64, base=500000.0, scaling=dict(factor=8.0, original=4096, fast=32.0, slow=1.0)))),
         dict(type="attention_2", mlp=mlp, mixer=dict(sizes, rot=dict(dims=d, base=500000.0),
                                                      mask=dict(size=window, keep_first=64))),
@@ -326,7 +326,7 @@ def munupel_shape(width, heads, kv_heads, ff, window, layers, vocab=32768):
                 layers=[dict(kinds[i % 2]) for i in range(layers)])
 
 
-MUNUPEL_SIZES = {   # width, heads, kv heads, feed-forward width, window and chunk, layers
+MUNUPEL_SIZES = {   # width, heads, kv heads, feed-forward width, window, layers
     "1k": (1024, 8, 2, 4096, 512, 4),
     "2k": (2048, 16, 4, 8192, 1024, 4),
     "4k": (4096, 32, 8, 14336, 2048, 4),

@@ -15,7 +15,8 @@
 //  * tiled (bfloat16, d and dv multiples of 8 up to 128, filled up with zeros to 32, 64, 96 or 128 in shared
 //    memory): 64 queries of one head per CTA over 64-key tiles on mma.sync, double buffered by cp.async, from
 //    packed keys (prompts) or the cache's pages (portions). The tiles of the kept keys come first, then those
-//    of the window; tiles that every query sees whole take no test per score.
+//    of the window; tiles that every query sees whole take no test per score. (Prompts mostly run
+//    attention_gated_umma.cu.)
 //  * decode (same sizes): one query per sequence over the cache; the CTAs of a thread-block cluster take runs
 //    of the visible pages, and their sums, maxima and masses meet in distributed shared memory in rank order:
 //    one launch, no partial rows in memory. It can begin at the float32 projection (Fresh): it then adds the
@@ -25,25 +26,14 @@
 // reach a product.
 #include <cooperative_groups.h>
 
+#include "attention_gated.cuh"
 #include "attention_mma.cuh"
 
 namespace {
 
 namespace cg = cooperative_groups;
 
-constexpr float kLog2e = 1.4426950408889634f;
-
-struct Form {
-  float scale, cap;            // cap <= 0: none
-  int window, keep;            // see first_visible_key; keep: first keys visible to everyone behind them
-  const float* sinks;          // [q_heads] or null
-  const float* gate;           // null, or pre-activations: gate[t * gate_stride + (per head ? h : h * dv + j)]
-  long long gate_stride;
-  int gate_per_head;
-  void* out;
-  long long out_stride;
-  float out_scale;
-};
+static_assert(kTile == kKeyTile, "a tile of keys is a page");
 
 // Where keys come from: packed rows of the step (table null) or the cache's pages.
 struct Source {
@@ -65,16 +55,6 @@ struct Fresh {
   int rotary;
   const int* dest_rows;     // [seqs]: page * 64 + row of the new token in the cache
 };
-
-__device__ __forceinline__ float gate_at(const Form& f, size_t t, int h, int dv, int j) {
-  if (f.gate == nullptr) return f.out_scale;
-  const float z = f.gate[t * f.gate_stride + (f.gate_per_head ? h : h * dv + j)];
-  return f.out_scale / (1.0f + expf(-z));
-}
-
-__device__ __forceinline__ bool sees(const Form& f, int key, int query, int first) {
-  return key <= query && (key >= first || key < f.keep);
-}
 
 // --------------------------------------------------------------------------- row-wise
 template <typename A, int PER, bool PAGED>
@@ -143,25 +123,6 @@ __global__ void gated_rowwise_kernel(const A* q, Source src, Form f, const int* 
 }
 
 // --------------------------------------------------------------------------- tiles
-__device__ __forceinline__ float rcp_fast(float x) {  // 1 / x on the special-function unit, 0 for infinity
-  float y;
-  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-
-// From q . k to the capped score in the log2 domain: tanh(x) = 1 - 2 / (1 + e^2x), whose error is a rounding
-// of the cap wherever x lies. Without a cap a product.
-struct ScoreMap {
-  float mul, cap_log2;
-  bool capped;
-  __device__ __forceinline__ explicit ScoreMap(const Form& f)
-      : mul(f.cap > 0.f ? 2.f * f.scale / f.cap * kLog2e : f.scale * kLog2e), cap_log2(f.cap * kLog2e), capped(f.cap > 0.f) {}
-  __device__ __forceinline__ float plain(float dot) const { return dot * mul; }
-  __device__ __forceinline__ float cap(float dot) const {
-    return fmaf(-2.f * cap_log2, rcp_fast(1.0f + exp2_fast(dot * mul)), cap_log2);
-  }
-};
-
 template <int N>
 __device__ __forceinline__ void to_scores(float (&s)[N][4], const ScoreMap& map) {
   if (map.capped) {
@@ -205,16 +166,6 @@ __device__ __forceinline__ void load_queries(uint32_t (&qa)[D / 16][4], const __
         qa[ks][half + 2 * hi] = r < valid_rows && c < width ? *reinterpret_cast<const uint32_t*>(base + r * pitch + c) : 0u;
       }
 }
-
-// The tiles a range of queries visits: those of the kept keys that lie before the window's, then the window's.
-struct Tiles {
-  int kept, first, count;
-  __device__ __forceinline__ Tiles(int first_key, int last_key, int keep) : first(first_key / kTile) {
-    kept = min((keep + kTile - 1) / kTile, first);
-    count = kept + last_key / kTile - first + 1;
-  }
-  __device__ __forceinline__ int at(int i) const { return i < kept ? i : first + i - kept; }
-};
 
 template <int D, int DV>
 __global__ __launch_bounds__(kThreads) void gated_tiled_kernel(const __nv_bfloat16* q, Source src, Form f,
@@ -559,18 +510,6 @@ int launch_decode(const void* q, const Source& src, const Form& f, const int*, c
   e = cudaLaunchKernelEx(&config, kernel, static_cast<const __nv_bfloat16*>(q), src, f, g.fresh, g.q_heads, g.kv_heads,
                          row_groups, g.d, g.dv);
   return e == cudaSuccess ? 0 : static_cast<int>(e);
-}
-
-bool bad_form(const Form& f, int q_heads, int kv_heads, int d, int dv) {
-  return q_heads <= 0 || kv_heads <= 0 || q_heads % kv_heads != 0 || d <= 0 || dv <= 0 || f.keep < 0 || f.out == nullptr ||
-         f.out_stride < static_cast<long long>(q_heads) * dv ||
-         (f.gate != nullptr && f.gate_stride < (f.gate_per_head ? q_heads : static_cast<long long>(q_heads) * dv));
-}
-
-Form make_form(float scale, float cap, int window, int keep, const float* sinks, const float* gate, long long gate_stride,
-               int gate_per_head, void* out, long long out_stride, float out_scale) {
-  // without a window or a chunk every earlier key is visible: kept keys say nothing
-  return Form{scale, cap, window, window == 0 ? 0 : keep, sinks, gate, gate_stride, gate_per_head, out, out_stride, out_scale};
 }
 
 }  // namespace

@@ -21,8 +21,10 @@
 // projection and the rounding at the end is float32. Reads of the projection go through plain
 // pointers: it is the output of the kernel before.
 //
+// Layers with biases and a split-half rotation at most (steps 1 and 5, from a table) take four columns per
+// thread, all loads and stores 16 or 8 bytes wide, wherever sizes and addresses allow (split_rotate_kernel).
 // Layers without a convolution, a row norm and a division behind the rotation (steps 1, 4 and 5 at
-// most) run a second kernel: a warp takes a head from its projection to its stores in registers,
+// most) otherwise run a kernel of their own: a warp takes a head from its projection to its stores in registers,
 // with no barrier after the table of cosines and sines.
 #include "common.cuh"
 
@@ -274,6 +276,67 @@ __global__ void shaped_heads_kernel(const S* proj, long long stride, const float
   }
 }
 
+template <typename A> __device__ __forceinline__ void store4(A* dst, const float (&y)[4]);
+template <> __device__ __forceinline__ void store4<float>(float* dst, const float (&y)[4]) {
+  *reinterpret_cast<float4*>(dst) = make_float4(y[0], y[1], y[2], y[3]);
+}
+template <> __device__ __forceinline__ void store4<__nv_bfloat16>(__nv_bfloat16* dst, const float (&y)[4]) {
+  __nv_bfloat162 lo = __floats2bfloat162_rn(y[0], y[1]), hi = __floats2bfloat162_rn(y[2], y[3]);
+  *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
+}
+
+// A thread takes four consecutive columns of one token's row; `quads` of them make a row.
+template <typename A>
+__global__ __launch_bounds__(256) void split_rotate_kernel(const float* proj, long long stride, const float* __restrict__ bias,
+                                                           const float2* table, int rotary, A* __restrict__ q_out,
+                                                           A* __restrict__ k_out, A* __restrict__ v_out,
+                                                           A* __restrict__ k_pages, A* __restrict__ v_pages,
+                                                           const int* __restrict__ dest_rows, long long items, int quads,
+                                                           int q_heads, int kv_heads, int d, int dv, int page_size) {
+  pdl_trigger();
+  const long long item = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
+  if (item >= items) return;
+  const int t = static_cast<int>(item / quads), col = static_cast<int>(item - static_cast<long long>(t) * quads) * 4;
+  const int nqk = (q_heads + kv_heads) * d, half = rotary / 2;
+  const bool is_v = col >= nqk;
+  const int hd = is_v ? (col - nqk) / dv : col / d, c = is_v ? col - nqk - hd * dv : col - hd * d;
+  const bool is_q = !is_v && hd < q_heads;
+  const int kh = is_v ? hd : hd - q_heads;
+  const int dest = !is_q && k_pages != nullptr ? dest_rows[t] : -1;
+  const bool turned = !is_v && c < rotary, leads = c < half;
+  const int other = leads ? col + half : col - half;  // the partners of a turned quad
+  float4 add = make_float4(0.f, 0.f, 0.f, 0.f), add_other = add;
+  if (bias != nullptr) {
+    add = *reinterpret_cast<const float4*>(bias + col);
+    if (turned) add_other = *reinterpret_cast<const float4*>(bias + other);
+  }
+  pdl_wait();
+  const float* row = proj + static_cast<size_t>(t) * stride;
+  const float4 x = *reinterpret_cast<const float4*>(row + col);
+  float y[4] = {x.x + add.x, x.y + add.y, x.z + add.z, x.w + add.w};
+  if (turned) {
+    const float4 p = *reinterpret_cast<const float4*>(row + other);
+    const float4* turns = reinterpret_cast<const float4*>(table + static_cast<size_t>(t) * half + (leads ? c : c - half));
+    const float4 a = turns[0], b = turns[1];  // (cos, sin) of two pairs each
+    const float co[4] = {a.x, a.z, b.x, b.z}, sn[4] = {a.y, a.w, b.y, b.w};
+    const float q[4] = {p.x + add_other.x, p.y + add_other.y, p.z + add_other.z, p.w + add_other.w};
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+      y[e] = leads ? fmaf(y[e], co[e], -__fmul_rn(q[e], sn[e])) : fmaf(y[e], co[e], __fmul_rn(q[e], sn[e]));
+  }
+  if (is_q) {
+    store4(q_out + (static_cast<size_t>(t) * q_heads + hd) * d + c, y);
+    return;
+  }
+  const int n = is_v ? dv : d;
+  A* packed = is_v ? v_out : k_out;
+  if (packed != nullptr) store4(packed + (static_cast<size_t>(t) * kv_heads + kh) * n + c, y);
+  if (dest >= 0) {
+    const size_t at = (static_cast<size_t>(dest / page_size) * kv_heads + kh) * page_size + dest % page_size;
+    store4((is_v ? v_pages : k_pages) + at * n + c, y);
+  }
+}
+
 }  // namespace
 
 // proj: [tokens, stride], of whose columns the first q_heads * d + kv_heads * (d + dv) are the row;
@@ -301,6 +364,24 @@ LRM_API int lrm_shaped_qkv_store(const void* proj, int in_dtype, long long strid
   if ((q_head_w == nullptr) != (k_head_w == nullptr)) return LRM_BAD_ARGUMENT;
   const int width = q_heads * d + kv_heads * (d + dv);
   if (stride < width) return LRM_BAD_ARGUMENT;
+  const uintptr_t all = reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(bias) | reinterpret_cast<uintptr_t>(table) |
+                        reinterpret_cast<uintptr_t>(q_out) | reinterpret_cast<uintptr_t>(k_out) | reinterpret_cast<uintptr_t>(v_out) |
+                        reinterpret_cast<uintptr_t>(k_pages) | reinterpret_cast<uintptr_t>(v_pages);
+  if (taps == nullptr && q_norm == nullptr && q_head_w == nullptr && !head_norm && pairing == 0 && in_dtype == LRM_F32 &&
+      (rotary == 0 || table != nullptr) && rotary % 8 == 0 && d % 4 == 0 && dv % 4 == 0 && stride % 4 == 0 && all % 16 == 0) {
+    const int quads = width / 4;
+    const long long items = static_cast<long long>(tokens) * quads;
+#define LRM_SPLIT_ROTATE(AT)                                                                                          \
+  LRM_LAUNCH((split_rotate_kernel<AT>), dim3(static_cast<unsigned>((items + 255) / 256)), 256, 0, stream,             \
+             static_cast<const float*>(proj), stride, bias, turns, rotary, static_cast<AT*>(q_out), static_cast<AT*>(k_out), \
+             static_cast<AT*>(v_out), static_cast<AT*>(k_pages), static_cast<AT*>(v_pages), dest_rows, items, quads, q_heads, \
+             kv_heads, d, dv, page_size)
+    if (out_dtype == LRM_F32) LRM_SPLIT_ROTATE(float);
+    else if (out_dtype == LRM_BF16) LRM_SPLIT_ROTATE(__nv_bfloat16);
+    else return LRM_BAD_ARGUMENT;
+#undef LRM_SPLIT_ROTATE
+    return 0;
+  }
   if (taps == nullptr && q_norm == nullptr && !head_norm && d <= 32 * kHeadPer && dv <= 32 * kHeadPer) {
     const int heads = q_heads + 2 * kv_heads;
     const int threads = 32 * (heads < 4 ? heads : heads >= 16 ? 8 : 4);

@@ -15,7 +15,7 @@ Attention without a softmax (a key's weight is the sigmoid of its score) has ker
 csrc/attention_sigmoid.cu: tiled in bfloat16 for head sizes 32, 64, 96 and 128, row-wise otherwise.
 Softmax attention with a cap on its scores, kept first keys or an output gate (and then also with sinks and
 values of another width) runs csrc/attention_gated.cu: tiled in bfloat16 for head sizes that are multiples of
-8 up to 128, row-wise otherwise.
+8 up to 128 (prompts on tcgen05, csrc/attention_gated_umma.cu), row-wise otherwise.
 
 `attend` is the one call a mixer makes: it takes the step's projection and picks
 rotation, cache write and attention kernels for the step's phase and geometry.
@@ -330,6 +330,9 @@ def sigmoid(q, k, v, kv, kv_heads: int, dv: int, out, out_stride: int, offset, g
                                             kv_heads, d, dv, page_size, *tail, _stream()), "attention_sigmoid_rowwise")
 
 
+GATED_UMMA_TOKENS = 65  # prompts from this length on go to the tcgen05 kernel
+
+
 def gated_ranks(seqs: int, kv_heads: int, group: int, max_kv_len: int, window: int, keep_first: int) -> int:
     """CTAs of a cluster that share a sequence's pages: about two CTAs per SM, no CTA without a page."""
     if force_gated_ranks is not None:
@@ -365,6 +368,14 @@ def gated(q, k, v, kv, kv_heads: int, dv: int, out, out_stride: int, form, gate,
     if (not force_rowwise and q.dtype == torch.bfloat16 and lib.lrm_attention_gated_supports(d, dv, page_size)
             and out_stride % 2 == 0 and all(t.data_ptr() % 16 == 0 for t in (q, keys, values)) and out.value % 4 == 0):
         ranks = 0
+        if (not paged and not force_warp_level and max_seq_len >= GATED_UMMA_TOKENS and scale > 0 and out_stride % 8 == 0
+                and out.value % 16 == 0 and lib.lrm_attention_gated_umma_supports(d, dv)):
+            from . import gemm_dispatch
+            gemm_dispatch.mark_status_dirty()
+            _done(lib.lrm_attention_gated_umma(_ptr(q), _ptr(k), _ptr(v), _ptr(cu_seqlens), T, cu_seqlens.numel() - 1,
+                                               max_seq_len, Hq, kv_heads, d, dv, *tail,
+                                               _ptr(gemm_dispatch._status_word(q.device)), _stream()), "attention_gated_umma")
+            return
         if one_each:
             ranks = gated_ranks(T, kv_heads, Hq // kv_heads, max_kv_len, window, form.keep_first)
         _done(lib.lrm_attention_gated(_ptr(q), _ptr(keys), _ptr(values), _ptr(None if one_each else cu_seqlens), *pages,

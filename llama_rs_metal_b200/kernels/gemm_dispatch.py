@@ -69,7 +69,9 @@ def check_status() -> None:
                      24: "probabilities", 25: "the output", 26: "a free key/value stage", 27: "aligned shared memory"}
             names.update({31: "a free stage", 32: "operand tiles", 33: "the accumulator", 34: "copies in flight",
                           35: "a free accumulator"})
-            kernel = "gemm_bf16_umma_pair" if code >= 31 else "attention_prefill_pingpong" if code >= 21 else \
+            names.update({41: "the query tile", 42: "a key/value tile", 43: "scores", 44: "probabilities", 45: "the output",
+                          46: "a free key/value stage", 47: "aligned shared memory"})
+            kernel = "attention_gated_umma" if code >= 41 else "gemm_bf16_umma_pair" if code >= 31 else "attention_prefill_pingpong" if code >= 21 else \
                 "attention_prefill_umma" if code >= 11 else "gemm_bf16_umma"
             raise LlamaError(f"{kernel} gave up waiting for {names.get(code, code)}; its result is invalid")
 

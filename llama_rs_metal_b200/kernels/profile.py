@@ -233,6 +233,9 @@ WORK: Dict[str, Callable[..., Tuple[float, float]]] = {
     "lrm_attention_gated_decode_fused": lambda a: (
         _visible_keys(_v(a[19]), _v(a[20])) * _v(a[14]) * (_v(a[15]) + _v(a[16])) * 2.0,
         2.0 * _visible_pairs(_v(a[19]), _v(a[20])) * _v(a[13]) * (_v(a[15]) + _v(a[16]))),
+    "lrm_attention_gated_umma": lambda a: (
+        2.0 * _v(a[4]) * (_v(a[7]) + _v(a[8])) * (_v(a[9]) + _v(a[10])),
+        2.0 * _visible_pairs(_v(a[13]), _v(a[14])) * _v(a[7]) * (_v(a[9]) + _v(a[10]))),
     "lrm_attention_gated_rowwise": lambda a: (
         0, 2.0 * _visible_pairs(_v(a[18]), _v(a[19])) * _v(a[12]) * (_v(a[14]) + _v(a[15]))),
     "lrm_tanh_columns": lambda a: (_v(a[5]) * _v(a[6]) * (_ELEM[_v(a[1])] + _ELEM[_v(a[4])]), 0),

@@ -518,6 +518,104 @@ def make_tolurax_dir(path, name, dtype=torch.bfloat16, edit=None):
     return write_model_folder(path, config.to_dict(), tensors, spec["seed"])
 
 
+def _scaled_rotation(dims, base, scaling=None):
+    out = dict(dims=dims, base=base)
+    if scaling is not None:
+        out["scaling"] = dict(zip(("factor", "original", "fast", "slow"), scaling))
+    return out
+
+
+def _gated(heads, kv_heads, dim, vdim, scale, size=None, rot=None, softcap=None, keep_first=None):
+    out = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, scale=scale)
+    if size is not None:
+        out["mask"] = dict(size=size)
+        if keep_first is not None:
+            out["mask"]["keep_first"] = keep_first
+    if rot is not None:
+        out["rot"] = rot
+    if softcap is not None:
+        out["softcap"] = softcap
+    return out
+
+
+def _chunk_layer(mixer, ff=None):
+    return dict(type="attention", mixer=mixer, mlp=None if ff is None else dict(kind="dense", ff=ff))
+
+
+def _window_layer(mixer, ff=None):
+    return dict(type="attention_2", mixer=mixer, mlp=None if ff is None else dict(kind="dense", ff=ff))
+
+
+_M1_SHARED = _gated(4, 2, 12, 20, 0.35, 7, _scaled_rotation(6, 50.0, (8.0, 64, 4.0, 0.5)), 3.0)
+_M2_SHARED = _gated(4, 2, 64, 96, 0.12, 65, _scaled_rotation(32, 10000.0), keep_first=70)
+
+# Three tiny Munupel configurations. Between them: sizes that are multiples of nothing and sizes whose sublayers
+# are joined and whose attention runs on the tensor cores (M2: query sizes 64, 40, 128 and 96, values wider and
+# narrower); key heads fewer than, and as many as, query heads, a group of 20; chunks and windows of one token,
+# shorter than a page, of one page, and longer; kept first keys that end inside a page, on a page's border and
+# behind it, one, and none; rotation of a part of the head, of all of it, and none, with frequencies kept,
+# stretched and blended; low caps and none; layers with and without a feed-forward; layers that run another
+# layer's tensors, also one whose owner comes later, and one that names such a layer.
+MUNUPEL = {
+    "M1": dict(
+        config=dict(architecture="Munupel", vocab=211, width=72, norm=dict(eps=1e-6), layers=[
+            _chunk_layer(_M1_SHARED, 56),
+            _window_layer(_gated(3, 3, 10, 6, 0.4, 9, _scaled_rotation(10, 100.0), keep_first=3)),
+            _window_layer(_gated(6, 2, 16, 10, 0.3, 40, keep_first=1), 40),
+            dict(_chunk_layer(_M1_SHARED, 56), weights_of=0),
+            _chunk_layer(_gated(2, 1, 18, 18, 0.3, 70)),
+        ]), seed=71, std=0.12),
+    "M2": dict(
+        config=dict(architecture="Munupel", vocab=512, width=192, norm=dict(eps=2e-5), layers=[
+            _window_layer(_M2_SHARED, 448),
+            _chunk_layer(_gated(20, 1, 40, 56, 0.2, 64, _scaled_rotation(24, 500.0, (4.0, 256, 16.0, 1.0)), 4.0), 256),
+            dict(_window_layer(_M2_SHARED, 448), weights_of=0),
+            _chunk_layer(_gated(4, 4, 128, 64, 0.1, 100, _scaled_rotation(128, 1000.0, (2.0, 100, 8.0, 2.0)), 6.0)),
+            _window_layer(_gated(6, 3, 96, 128, 0.11, 64, _scaled_rotation(64, 20000.0), keep_first=64), 320),
+        ]), seed=72, std=0.06),
+    "M3": dict(
+        config=dict(architecture="Munupel", vocab=300, width=64, norm=dict(eps=1e-5), layers=[
+            _chunk_layer(_gated(2, 2, 16, 24, 0.3)),
+            dict(_window_layer(_gated(1, 1, 8, 8, 0.5), 40), weights_of=3),
+            _window_layer(_gated(3, 1, 16, 32, 0.4, 1), 24),
+            _window_layer(_gated(1, 1, 8, 8, 0.5), 40),
+            dict(_window_layer(_gated(1, 1, 8, 8, 0.5), 40), weights_of=1),
+            _chunk_layer(_gated(2, 1, 8, 8, 0.4, 1, _scaled_rotation(2, 30.0), 2.0), 32),
+        ]), seed=73, std=0.15),
+}
+
+
+def make_munupel_dir(path, name, dtype=torch.bfloat16, edit=None):
+    """A model folder of a tiny Munupel configuration (a name of MUNUPEL, or a spec of the caller's own) with
+    seeded random weights; `edit` (a function of the name -> tensor dict) may change them before they are
+    written. Norm weights are N(1, 0.2), biases N(0, 0.5) (so that one left out shows), sinks N(1, 1) (about as
+    much mass as a handful of keys), queries and keys larger than the rest (scores of several units, so that
+    caps bite and single keys stand out), gates likewise (far from all alike)."""
+    from llama_rs_metal_b200.engine.model import DecoderModel
+    from llama_rs_metal_b200.registry import find_architecture
+    from llama_rs_metal_b200.runtime import Runtime
+    from llama_rs_metal_b200.weights.random_init import random_tensors, write_model_folder
+    spec = MUNUPEL[name] if isinstance(name, str) else name
+    arch = find_architecture(spec["config"])
+    config = arch.config_class.from_dict(spec["config"])
+    model = DecoderModel(arch.plan(config), Runtime(torch.device("cpu"), torch.float32))
+    tensors = random_tensors(model.tensor_specs(), spec["seed"], std=spec["std"], vector_mean=0.0, vector_std=0.5,
+                             dtype=dtype)
+    for name_, t in tensors.items():
+        last = name_.rsplit(".", 1)[-1]
+        if last in ("norm", "norm1"):
+            t.mul_(0.4).add_(1.0)
+        elif last == "sink":
+            t.mul_(2.0).add_(1.0)
+        elif last in ("q", "k", "g"):
+            t.mul_(1.6)
+        elif name_ == "embed":
+            t.mul_(1.0 / spec["std"])
+    if edit is not None:
+        edit(tensors)
+    return write_model_folder(path, config.to_dict(), tensors, spec["seed"])
+
+
 def random_tokens(seed, length, vocab):
     rng = np.random.default_rng(seed)
     return [int(t) for t in rng.integers(0, vocab, size=length)]

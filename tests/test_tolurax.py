@@ -151,7 +151,7 @@ def test_stretched_frequencies_agree_with_the_position_encoding():
 def test_attention_options_that_exclude_each_other():
     from llama_rs_metal_b200.parts.attention import Attention
     with pytest.raises(InvalidError, match="gate"):
-        Attention(64, 2, 1, 16, gate=True)
+        Attention(64, 2, 1, 16, gate="head", weights="sigmoid")
     with pytest.raises(UnsupportedError, match="weights"):
         Attention(64, 2, 1, 16, weights="relu")
     assert Attention(64, 2, 1, 16).mixed_width is None
