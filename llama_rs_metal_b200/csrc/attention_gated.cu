@@ -272,8 +272,9 @@ __global__ __launch_bounds__(kThreads) void gated_tiled_kernel(const __nv_bfloat
       if (c >= dv) continue;
       float a = head_gate, e = head_gate;
       if (by_element) {
-        a *= gate_at(f, tok, h, dv, c);
-        e *= gate_at(f, tok, h, dv, c + 1);
+        const float* z = f.gate + tok * f.gate_stride + h * dv + c;
+        a *= f.out_scale * unit_sigmoid(z[0]);
+        e *= f.out_scale * unit_sigmoid(z[1]);
       }
       *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16(o[dn][2 * half] * a, o[dn][2 * half + 1] * e);
     }

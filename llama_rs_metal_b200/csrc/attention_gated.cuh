@@ -51,6 +51,8 @@ __device__ __forceinline__ float unit_rcp(float x) {  // 1 / x likewise, 0 for i
   return y;
 }
 
+__device__ __forceinline__ float unit_sigmoid(float z) { return unit_rcp(1.0f + unit_exp2(-kLog2e * z)); }
+
 // From q . k to the capped score in the log2 domain: tanh(x) = 1 - 2 / (1 + e^2x), whose error is a rounding
 // of the cap wherever x lies. Without a cap a product. Both rise with q . k (where the scale is positive).
 struct ScoreMap {

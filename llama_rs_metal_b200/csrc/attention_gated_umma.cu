@@ -199,6 +199,12 @@ __global__ __launch_bounds__(kGatedThreads, CTAS) void gated_umma_kernel(
     const int row_first = first_visible_key(row, f.window);
     const int whole_from = first_visible_key(q0 + BQ - 1, f.window);
     const float sink_log2 = f.sinks != nullptr ? f.sinks[h] * kLog2e : -INFINITY;
+    // the row's gates are wanted at the end: have them in L2 by then
+    const size_t tok = static_cast<size_t>(start + min(row, len - 1));
+    const bool by_element = f.gate != nullptr && !f.gate_per_head;
+    const float* gates = by_element ? f.gate + tok * f.gate_stride + h * dv : nullptr;
+    if (by_element)
+      for (int c = 0; c < dv; c += 32) asm volatile("prefetch.global.L2 [%0];" ::"l"(gates + c));
     float m_run = sink_log2;   // the row's true running maximum (log2 domain)
     float m_ref = -INFINITY;   // the maximum O and the mass are scaled by
     float l = 0.f;
@@ -284,6 +290,24 @@ __global__ __launch_bounds__(kGatedThreads, CTAS) void gated_umma_kernel(
       __syncwarp();
       if (lane == 0) mbar_arrive(p_ready);
     }
+    // 32 gates at a time on the way into registers, the first ones while the last product runs
+    const bool fours = by_element && f.gate_stride % 4 == 0 && (reinterpret_cast<uintptr_t>(f.gate) & 15) == 0 && dv % 4 == 0;
+    float z[32];
+    auto load_gates = [&](int c) {
+      if (!by_element) return;
+#pragma unroll
+      for (int e = 0; e < 32; e += 4) {
+        if (c + e >= dv) break;  // (dv is a multiple of 8)
+        if (fours) {
+          const float4 four = *reinterpret_cast<const float4*>(gates + c + e);
+          z[e] = four.x, z[e + 1] = four.y, z[e + 2] = four.z, z[e + 3] = four.w;
+        } else {
+#pragma unroll
+          for (int u = 0; u < 4; ++u) z[e + u] = gates[c + e + u];
+        }
+      }
+    };
+    load_gates(0);
     if (ok && !__all_sync(0xffffffffu, mbar_wait(o_done, 0, status, kStuckOutput))) {
       *bail = 1;
       ok = false;
@@ -291,10 +315,7 @@ __global__ __launch_bounds__(kGatedThreads, CTAS) void gated_umma_kernel(
     tc_fence_after();
     if (ok) {
       // the mass belongs to m_ref, and so does O: their quotient is the row's attention
-      const size_t tok = static_cast<size_t>(start + min(row, len - 1));
-      const bool by_element = f.gate != nullptr && !f.gate_per_head;
       const float factor = (by_element ? f.out_scale : gate_at(f, tok, h, dv, 0)) / l;
-      const float* gates = by_element ? f.gate + tok * f.gate_stride + h * dv : nullptr;
       __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(f.out) + tok * f.out_stride + h * dv;
 #pragma unroll 1
       for (int c = 0; c < dv; c += 32) {
@@ -309,14 +330,15 @@ __global__ __launch_bounds__(kGatedThreads, CTAS) void gated_umma_kernel(
             for (int u = 0; u < 8; u += 2) {
               float x = __uint_as_float(r[e + u]) * factor, y = __uint_as_float(r[e + u + 1]) * factor;
               if (by_element) {
-                x *= unit_rcp(1.0f + unit_exp2(-kLog2e * gates[c + e + u]));
-                y *= unit_rcp(1.0f + unit_exp2(-kLog2e * gates[c + e + u + 1]));
+                x *= unit_sigmoid(z[e + u]);
+                y *= unit_sigmoid(z[e + u + 1]);
               }
               packed[u >> 1] = pack_bf16(x, y);
             }
             *reinterpret_cast<uint4*>(dst + c + e) = make_uint4(packed[0], packed[1], packed[2], packed[3]);
           }
         }
+        load_gates(c + 32);
       }
     }
   }

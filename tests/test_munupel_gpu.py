@@ -287,11 +287,10 @@ def test_sublayers_are_joined_under_bfloat16_only(engine, folders, tmp_path):
     odd = dict(config=dict(architecture="Munupel", vocab=50, width=60, norm=dict(eps=1e-5), layers=[
         helpers._window_layer(helpers._gated(2, 1, 8, 12, 0.3, 5, keep_first=1), 32)]), seed=1, std=0.1)
     folder = helpers.make_munupel_dir(str(tmp_path), odd)
-    for path, dtype, joined in ((folders["M2"], "bfloat16", True), (folders["M1"], "bfloat16", True), (folders["M2"], "float32", False),
-                                (folder, "bfloat16", False)):
+    for path, dtype, joined in ((folders["M2"], "bfloat16", [True] * 3), (folders["M1"], "bfloat16", [True, False]),
+                                (folders["M2"], "float32", [False] * 3), (folder, "bfloat16", [False])):
         _, _, model = open_runner(engine, path, dtype)
-        blocks = [b for b in model.blocks if b.kind == "parallel"]
-        assert blocks and all((b.into is not None) == joined for b in blocks), (path, dtype)
+        assert [b.into is not None for b in model.blocks if b.kind == "parallel"] == joined, (path, dtype)
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
