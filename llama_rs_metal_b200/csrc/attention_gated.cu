@@ -33,6 +33,8 @@ namespace {
 
 namespace cg = cooperative_groups;
 
+constexpr int kMaxRanks = 8;  // CTAs that share a sequence's keys in a decode step, at most
+
 static_assert(kTile == kKeyTile, "a tile of keys is a page");
 
 // Where keys come from: packed rows of the step (table null) or the cache's pages.
@@ -330,35 +332,52 @@ __global__ __launch_bounds__(kThreads) void gated_decode_kernel(const __nv_bfloa
   __nv_bfloat16* new_value = new_key + D;
   const bool has_newest = split && end == count && begin < end;
   if (split) {
+    // columns of this CTA's query heads, then of the new key and of the new value, kItems at a time so that their
+    // loads are all under way before the first is used
+    constexpr int kItems = 4;
     const float* row = fresh.proj + static_cast<size_t>(b) * fresh.stride;
     const int half = fresh.rotary / 2;
     const float2* turns = fresh.table + static_cast<size_t>(b) * half;
-    auto shaped = [&](int first, int c) {  // column c of the head that begins at column `first`
-      auto at = [&](int i) { return row[first + i] + (fresh.bias != nullptr ? fresh.bias[first + i] : 0.f); };
-      const float x = at(c);
-      if (c >= 2 * half) return x;
-      const bool leads = c < half;
-      const float2 turn = turns[leads ? c : c - half];
-      const float p = at(leads ? c + half : c - half);
-      return leads ? fmaf(x, turn.x, -__fmul_rn(p, turn.y)) : fmaf(x, turn.x, __fmul_rn(p, turn.y));
-    };
-    for (int i = threadIdx.x; i < 16 * D; i += kThreads) {
-      const int r = i / D, c = i % D;
-      Qs[r * KSTRIDE + c] = __float2bfloat16_rn(r < rows && c < d ? shaped((head0 + r) * d, c) : 0.f);
-    }
-    if (has_newest) {
-      const int dest = rg == 0 ? fresh.dest_rows[b] : -1;  // one of the groups of query heads stores the row
-      const size_t cached = dest >= 0 ? (static_cast<size_t>(dest / kTile) * kv_heads + kh) * kTile + dest % kTile : 0;
-      for (int c = threadIdx.x; c < d + dv; c += kThreads) {
-        if (c < d) {
-          const __nv_bfloat16 x = __float2bfloat16_rn(shaped((q_heads + kh) * d, c));
-          new_key[c] = x;
-          if (dest >= 0) const_cast<__nv_bfloat16*>(static_cast<const __nv_bfloat16*>(src.k))[cached * d + c] = x;
+    const int nq = rows * d, items = nq + (has_newest ? d + dv : 0);
+    const int dest = has_newest && rg == 0 ? fresh.dest_rows[b] : -1;  // one of the groups of query heads stores the row
+    const size_t cached = dest >= 0 ? (static_cast<size_t>(dest / kTile) * kv_heads + kh) * kTile + dest % kTile : 0;
+    __nv_bfloat16* k_row = const_cast<__nv_bfloat16*>(static_cast<const __nv_bfloat16*>(src.k)) + cached * d;
+    __nv_bfloat16* v_row = const_cast<__nv_bfloat16*>(static_cast<const __nv_bfloat16*>(src.v)) + cached * dv;
+    for (int i0 = threadIdx.x; i0 < items; i0 += kItems * kThreads) {
+      float x[kItems], partner[kItems];
+      float2 turn[kItems];
+      int place[kItems];  // column within its head
+#pragma unroll
+      for (int u = 0; u < kItems; ++u) {
+        const int i = i0 + u * kThreads;
+        const bool is_v = i >= nq + d;
+        const int col = i < nq ? head0 * d + i : is_v ? (q_heads + kv_heads) * d + kh * dv + i - nq - d : (q_heads + kh) * d + i - nq;
+        const int c = i < nq ? i % d : is_v ? i - nq - d : i - nq;
+        place[u] = c;
+        x[u] = partner[u] = 0.f;
+        turn[u] = make_float2(1.f, 0.f);
+        if (i >= items) continue;
+        x[u] = row[col] + (fresh.bias != nullptr ? fresh.bias[col] : 0.f);
+        if (!is_v && c < 2 * half) {
+          const int other = c < half ? col + half : col - half;
+          partner[u] = row[other] + (fresh.bias != nullptr ? fresh.bias[other] : 0.f);
+          turn[u] = turns[c < half ? c : c - half];
+        }
+      }
+#pragma unroll
+      for (int u = 0; u < kItems; ++u) {
+        const int i = i0 + u * kThreads, c = place[u];
+        if (i >= items) continue;
+        const float cross = __fmul_rn(partner[u], turn[u].y);
+        const __nv_bfloat16 y = __float2bfloat16_rn(i >= nq + d || c >= 2 * half ? x[u] : fmaf(x[u], turn[u].x, c < half ? -cross : cross));
+        if (i < nq) {
+          Qs[(i / d) * KSTRIDE + c] = y;
+        } else if (i < nq + d) {
+          new_key[c] = y;
+          if (dest >= 0) k_row[c] = y;
         } else {
-          const int first = (q_heads + kv_heads) * d + kh * dv + c - d;
-          const __nv_bfloat16 x = __float2bfloat16_rn(row[first] + (fresh.bias != nullptr ? fresh.bias[first] : 0.f));
-          new_value[c - d] = x;
-          if (dest >= 0) const_cast<__nv_bfloat16*>(static_cast<const __nv_bfloat16*>(src.v))[cached * dv + c - d] = x;
+          new_value[c] = y;
+          if (dest >= 0) v_row[c] = y;
         }
       }
     }
@@ -366,8 +385,10 @@ __global__ __launch_bounds__(kThreads) void gated_decode_kernel(const __nv_bfloa
 #pragma unroll
     for (int ks = 0; ks < D / 16; ++ks)
 #pragma unroll
-      for (int e = 0; e < 4; ++e)
-        qa[ks][e] = *reinterpret_cast<const uint32_t*>(Qs + (g + 8 * (e & 1)) * KSTRIDE + 16 * ks + 8 * (e >> 1) + 2 * t);
+      for (int e = 0; e < 4; ++e) {
+        const int r = g + 8 * (e & 1), c = 16 * ks + 8 * (e >> 1) + 2 * t;
+        qa[ks][e] = r < rows && c < d ? *reinterpret_cast<const uint32_t*>(Qs + r * KSTRIDE + c) : 0u;
+      }
   } else {
     load_queries<D>(qa, q + (static_cast<size_t>(b) * q_heads + head0) * d, d, d, rows);
   }
@@ -439,26 +460,36 @@ __global__ __launch_bounds__(kThreads) void gated_decode_kernel(const __nv_bfloa
     joined[i] = c == DV ? top : value;
   }
   cg::cluster_group cluster = cg::this_cluster();
+  const int outputs = rows * dv, share = (outputs + ranks - 1) / ranks, to = min(outputs, (rank + 1) * share);
+  const int mine = rank * share + threadIdx.x;  // the first of this thread's outputs: its gate comes while the others arrive
+  float gate = mine < to ? gate_at(f, b, head0 + mine / dv, dv, mine % dv) : 0.f;
   if (ranks > 1) cluster.sync();  // every CTA's parts are complete
   else __syncthreads();
   __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(f.out) + static_cast<size_t>(b) * f.out_stride + head0 * dv;
-  const int items = rows * dv, share = (items + ranks - 1) / ranks, to = min(items, (rank + 1) * share);
-  for (int i = rank * share + threadIdx.x; i < to; i += kThreads) {
+  for (int i = mine; i < to; i += kThreads) {
     const int r = i / dv, c = i % dv;
+    if (i != mine) gate = gate_at(f, b, head0 + r, dv, c);
     const float sink_log2 = f.sinks != nullptr ? f.sinks[head0 + r] * kLog2e : -INFINITY;
-    float top = sink_log2, value = 0.f;
-    for (int k = 0; k < ranks; ++k) top = fmaxf(top, cluster.map_shared_rank(joined, k)[r * PART + DV]);
-    float mass = f.sinks != nullptr ? exp2f(sink_log2 - top) : 0.f;
-    for (int k = 0; k < ranks; ++k) {
-      const float* part = cluster.map_shared_rank(joined, k) + r * PART;
-      const float mk = part[DV];
-      if (mk > -INFINITY) {
-        const float w = exp2f(mk - top);
-        value = fmaf(part[c], w, value);
-        mass = fmaf(part[DV + 1], w, mass);
-      }
+    float mk[kMaxRanks], lk[kMaxRanks], vk[kMaxRanks];  // all of the peers' values under way together
+#pragma unroll
+    for (int k = 0; k < kMaxRanks; ++k) {
+      const float* part = cluster.map_shared_rank(joined, k < ranks ? k : 0) + r * PART;
+      mk[k] = k < ranks ? part[DV] : -INFINITY;
+      lk[k] = k < ranks ? part[DV + 1] : 0.f;
+      vk[k] = k < ranks ? part[c] : 0.f;
     }
-    dst[i] = __float2bfloat16_rn(value / mass * gate_at(f, b, head0 + r, dv, c));
+    float top = sink_log2, value = 0.f;
+#pragma unroll
+    for (int k = 0; k < kMaxRanks; ++k) top = fmaxf(top, mk[k]);
+    float mass = f.sinks != nullptr ? exp2f(sink_log2 - top) : 0.f;
+#pragma unroll
+    for (int k = 0; k < kMaxRanks; ++k)
+      if (mk[k] > -INFINITY) {  // (a CTA that saw no key has nothing to add)
+        const float w = exp2f(mk[k] - top);
+        value = fmaf(vk[k], w, value);
+        mass = fmaf(lk[k], w, mass);
+      }
+    dst[i] = __float2bfloat16_rn(value / mass * gate);
   }
   if (ranks > 1) cluster.sync();  // nobody leaves while a peer may still read its parts
 }
@@ -589,7 +620,7 @@ LRM_API int lrm_attention_gated(const void* q, const void* k, const void* v, con
                                 float out_scale, int ranks, cudaStream_t stream) {
   if (seqs <= 0 || (ranks == 0 && max_seq_len <= 0)) return 0;
   const Form f = make_form(scale, cap, window, keep, sinks, gate, gate_stride, gate_per_head, out, out_stride, out_scale);
-  if (bad_form(f, q_heads, kv_heads, d, dv) || ranks < 0 || ranks > 8 || (ranks == 0 && cu_seqlens == nullptr) ||
+  if (bad_form(f, q_heads, kv_heads, d, dv) || ranks < 0 || ranks > kMaxRanks || (ranks == 0 && cu_seqlens == nullptr) ||
       (ranks > 0 && page_table == nullptr) || (page_table != nullptr && (slots == nullptr || kv_lens == nullptr)))
     return LRM_BAD_ARGUMENT;
   if (!lrm_attention_gated_supports(d, dv, kTile) || out_stride % 2 != 0 || reinterpret_cast<uintptr_t>(out) % 4 != 0 ||
@@ -613,7 +644,7 @@ LRM_API int lrm_attention_gated_decode_fused(const float* proj, long long stride
                                              float out_scale, int ranks, cudaStream_t stream) {
   if (seqs <= 0) return 0;
   const Form f = make_form(scale, cap, window, keep, sinks, gate, gate_stride, gate_per_head, out, out_stride, out_scale);
-  if (bad_form(f, q_heads, kv_heads, d, dv) || ranks < 1 || ranks > 8 || proj == nullptr || dest_rows == nullptr ||
+  if (bad_form(f, q_heads, kv_heads, d, dv) || ranks < 1 || ranks > kMaxRanks || proj == nullptr || dest_rows == nullptr ||
       page_table == nullptr || slots == nullptr || kv_lens == nullptr || rotary < 0 || rotary % 2 || rotary > d ||
       (rotary > 0 && table == nullptr) || stride < q_heads * d + static_cast<long long>(kv_heads) * (d + dv))
     return LRM_BAD_ARGUMENT;
