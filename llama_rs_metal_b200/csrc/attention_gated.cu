@@ -33,6 +33,7 @@ namespace {
 
 namespace cg = cooperative_groups;
 
+constexpr int kStages = 3;    // pages of a decode step's ring
 constexpr int kMaxRanks = 8;  // CTAs that share a sequence's keys in a decode step, at most
 
 static_assert(kTile == kKeyTile, "a tile of keys is a page");
@@ -292,8 +293,8 @@ __global__ __launch_bounds__(kThreads) void gated_decode_kernel(const __nv_bfloa
   constexpr int KSTRIDE = D + 8, VSTRIDE = DV + 8, KTILE = kTile * KSTRIDE, VTILE = kTile * VSTRIDE;
   constexpr int PART = DV + 2;  // a row's sums, maximum (log2 domain) and mass
   extern __shared__ __align__(16) unsigned char smem_raw[];
-  __nv_bfloat16* Ks = reinterpret_cast<__nv_bfloat16*>(smem_raw);
-  __nv_bfloat16* Vs = Ks + 2 * KTILE;
+  __nv_bfloat16* Ks = reinterpret_cast<__nv_bfloat16*>(smem_raw);  // [kStages][64][D + 8]
+  __nv_bfloat16* Vs = Ks + kStages * KTILE;                        // [kStages][64][DV + 8]
   const int ranks = gridDim.x, rank = blockIdx.x;
   const int rg = blockIdx.y % row_groups, kh = (blockIdx.y / row_groups) % kv_heads;
   const int b = blockIdx.y / (row_groups * kv_heads);
@@ -309,7 +310,12 @@ __global__ __launch_bounds__(kThreads) void gated_decode_kernel(const __nv_bfloa
   const int* table = src.page_table + static_cast<size_t>(src.slots[b]) * src.table_stride;
   const ScoreMap map(f);
 
-  auto issue = [&](int i, int stage) {
+  auto issue = [&](int i) {  // page i of the list into its stage; one group of copies per call, empty beyond the end
+    if (i >= end) {
+      cp_async_commit();
+      return;
+    }
+    const int stage = (i - begin) % kStages;
     const int page_index = tiles.at(i), k0 = page_index * kTile, page = table[page_index];
     const int lo = k0 < f.keep ? 0 : first_key - k0;
     const int hi = page < 0 ? 0 : i < tiles.kept ? f.keep - k0 : len - k0;
@@ -321,13 +327,13 @@ __global__ __launch_bounds__(kThreads) void gated_decode_kernel(const __nv_bfloa
   // only q and the newest key and value row (in the last page) come from the kernel before this one; where
   // this kernel splits the projection it puts the newest row there itself
   const bool split = fresh.proj != nullptr;
-  const bool early = begin < end && (split || begin != count - 1);
-  if (early) issue(begin, 0);
+  int issued = begin;
+  while (issued < begin + kStages - 1 && (split || issued < count - 1)) issue(issued++);
   pdl_wait();
-  if (!early && begin < end) issue(begin, 0);
+  while (issued < begin + kStages - 1) issue(issued++);
 
   uint32_t qa[D / 16][4];
-  __nv_bfloat16* Qs = Vs + 2 * VTILE;      // [16][D + 8], behind it the new key [D] and the new value [DV]
+  __nv_bfloat16* Qs = Vs + kStages * VTILE;  // [16][D + 8], behind it the new key [D] and the new value [DV]
   __nv_bfloat16* new_key = Qs + 16 * KSTRIDE;
   __nv_bfloat16* new_value = new_key + D;
   const bool has_newest = split && end == count && begin < end;
@@ -399,10 +405,10 @@ __global__ __launch_bounds__(kThreads) void gated_decode_kernel(const __nv_bfloa
     for (int e = 0; e < 4; ++e) o[dn][e] = 0.f;
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
   for (int i = begin; i < end; ++i) {
-    const int stage = (i - begin) & 1, k0 = tiles.at(i) * kTile + 16 * warp;
-    cp_async_wait<0>();  // page i is here
-    __syncthreads();     // ... for every thread, and everyone is done with page i - 1
-    if (i + 1 < end) issue(i + 1, stage ^ 1);
+    const int stage = (i - begin) % kStages, k0 = tiles.at(i) * kTile + 16 * warp;
+    cp_async_wait<kStages - 2>();  // page i is here
+    __syncthreads();               // ... for every thread, and everyone is done with page i - 1
+    issue(i + kStages - 1);
     if (has_newest && i == count - 1) {  // the page's copy of the newest row is older than the row
       const int r = query % kTile;
       for (int c = threadIdx.x; c < d + dv; c += kThreads) {
@@ -518,7 +524,7 @@ int launch_tiled(const void* q, const Source& src, const Form& f, const int* cu_
 template <int D, int DV>
 int launch_decode(const void* q, const Source& src, const Form& f, const int*, const Geometry& g, cudaStream_t stream) {
   auto kernel = gated_decode_kernel<D, DV>;
-  const int held = tiles_bytes<D, DV>() + (g.fresh.proj != nullptr ? fresh_bytes<D, DV>() : 0);
+  const int held = tiles_bytes<D, DV>() / 2 * kStages + (g.fresh.proj != nullptr ? fresh_bytes<D, DV>() : 0);
   const int bytes = held > parts_bytes<DV>() ? held : parts_bytes<DV>();
   cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
   if (e != cudaSuccess) return static_cast<int>(e);
@@ -538,7 +544,9 @@ int launch_decode(const void* q, const Source& src, const Form& f, const int*, c
   attributes[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
   attributes[1].val.programmaticStreamSerializationAllowed = 1;
   config.attrs = attributes;
-  config.numAttrs = g_lrm_pdl ? 2 : 1;
+  // a cluster of several CTAs does not start ahead of its predecessor's end: let in early, its CTAs take the places
+  // that come free one by one and hold them while the others still wait for theirs (2 to 20 us per decode step)
+  config.numAttrs = g_lrm_pdl && g.ranks == 1 ? 2 : 1;
   e = cudaLaunchKernelEx(&config, kernel, static_cast<const __nv_bfloat16*>(q), src, f, g.fresh, g.q_heads, g.kv_heads,
                          row_groups, g.d, g.dv);
   return e == cudaSuccess ? 0 : static_cast<int>(e);

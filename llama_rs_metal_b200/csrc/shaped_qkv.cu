@@ -285,18 +285,17 @@ template <> __device__ __forceinline__ void store4<__nv_bfloat16>(__nv_bfloat16*
   *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
 }
 
-// A thread takes four consecutive columns of one token's row; `quads` of them make a row.
+// A thread takes four consecutive columns of the row of token blockIdx.x; `quads` of them make a row.
 template <typename A>
 __global__ __launch_bounds__(256) void split_rotate_kernel(const float* proj, long long stride, const float* __restrict__ bias,
                                                            const float2* table, int rotary, A* __restrict__ q_out,
                                                            A* __restrict__ k_out, A* __restrict__ v_out,
                                                            A* __restrict__ k_pages, A* __restrict__ v_pages,
-                                                           const int* __restrict__ dest_rows, long long items, int quads,
-                                                           int q_heads, int kv_heads, int d, int dv, int page_size) {
+                                                           const int* __restrict__ dest_rows, int quads, int q_heads,
+                                                           int kv_heads, int d, int dv, int page_size) {
   pdl_trigger();
-  const long long item = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
-  if (item >= items) return;
-  const int t = static_cast<int>(item / quads), col = static_cast<int>(item - static_cast<long long>(t) * quads) * 4;
+  const int t = blockIdx.x, col = (blockIdx.y * blockDim.x + threadIdx.x) * 4;
+  if (col >= quads * 4) return;
   const int nqk = (q_heads + kv_heads) * d, half = rotary / 2;
   const bool is_v = col >= nqk;
   const int hd = is_v ? (col - nqk) / dv : col / d, c = is_v ? col - nqk - hd * dv : col - hd * d;
@@ -370,11 +369,11 @@ LRM_API int lrm_shaped_qkv_store(const void* proj, int in_dtype, long long strid
   if (taps == nullptr && q_norm == nullptr && q_head_w == nullptr && !head_norm && pairing == 0 && in_dtype == LRM_F32 &&
       (rotary == 0 || table != nullptr) && rotary % 8 == 0 && d % 4 == 0 && dv % 4 == 0 && stride % 4 == 0 && all % 16 == 0) {
     const int quads = width / 4;
-    const long long items = static_cast<long long>(tokens) * quads;
+    const int threads = quads >= 256 ? 256 : (quads + 31) / 32 * 32;
 #define LRM_SPLIT_ROTATE(AT)                                                                                          \
-  LRM_LAUNCH((split_rotate_kernel<AT>), dim3(static_cast<unsigned>((items + 255) / 256)), 256, 0, stream,             \
+  LRM_LAUNCH((split_rotate_kernel<AT>), dim3(tokens, (quads + threads - 1) / threads), threads, 0, stream,            \
              static_cast<const float*>(proj), stride, bias, turns, rotary, static_cast<AT*>(q_out), static_cast<AT*>(k_out), \
-             static_cast<AT*>(v_out), static_cast<AT*>(k_pages), static_cast<AT*>(v_pages), dest_rows, items, quads, q_heads, \
+             static_cast<AT*>(v_out), static_cast<AT*>(k_pages), static_cast<AT*>(v_pages), dest_rows, quads, q_heads, \
              kv_heads, d, dv, page_size)
     if (out_dtype == LRM_F32) LRM_SPLIT_ROTATE(float);
     else if (out_dtype == LRM_BF16) LRM_SPLIT_ROTATE(__nv_bfloat16);
