@@ -322,7 +322,7 @@ def drawn_configuration(seed):
 
     def pick(*values):
         return values[int(rng.integers(len(values)))]
-    width = int(pick(40, 64, 88, 136, 256))
+    width = int(pick(40, 64, 88, 136, 232))
     layers = []
     for _ in range(int(rng.integers(2, 6))):
         kv = int(pick(1, 2, 3))
@@ -330,14 +330,14 @@ def drawn_configuration(seed):
         rot = None
         if pick(True, True, True, False):
             scaling = pick(None, (8.0, 128, 32.0, 1.0), (2.0, 40, 3.0, 0.5), (4.0, 1000, 16.0, 2.0))
-            rot = helpers._scaled_rotation(int(pick(*[r for r in (2, 4, 16, 24, 64, 96) if r <= dim])), float(pick(30.0, 10000.0, 250000.0)), scaling)
+            rot = helpers._scaled_rotation(int(pick(*[r for r in (2, 4, 16, 24, 64, 96) if r <= dim])), float(pick(30.0, 10000.0, 200000.0)), scaling)
         sizes = (heads, kv, dim, int(pick(dim, 8, 12, 32, 96)), float(pick(0.1, 0.3)))
         ff = int(pick(24, 64, 100)) if rng.integers(3) else None
         if pick(True, False):
-            layers.append(helpers._chunk_layer(helpers._gated(*sizes, pick(None, 1, 2, 33, 64, 96, 200), rot, pick(None, 2.0, 5.0)), ff))
+            layers.append(helpers._chunk_layer(helpers._gated(*sizes, pick(None, 1, 2, 33, 64, 90, 200), rot, pick(None, 2.0, 5.0)), ff))
         else:
-            size = pick(None, 1, 2, 40, 64, 65, 136)
-            layers.append(helpers._window_layer(helpers._gated(*sizes, size, rot, keep_first=pick(None, 1, 20, 64, 70) if size else None), ff))
+            size = pick(None, 1, 2, 40, 64, 65, 130)
+            layers.append(helpers._window_layer(helpers._gated(*sizes, size, rot, keep_first=pick(None, 1, 17, 64, 70) if size else None), ff))
     if rng.integers(3):
         of = int(rng.integers(len(layers)))
         layers.insert(int(rng.integers(of + 1, len(layers) + 1)), dict(layers[of], weights_of=of))
